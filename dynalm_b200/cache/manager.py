@@ -41,7 +41,7 @@ DEFAULT_PAGE_SIZE = 16      # tokens per page, the reference's block size (dynal
 def _torch_dtype(name: Optional[str], default: torch.dtype) -> torch.dtype:
     if name is None:
         return default
-    return {"float32": torch.float32, "bfloat16": torch.bfloat16}[name]
+    return {"float32": torch.float32, "bfloat16": torch.bfloat16, "int32": torch.int32}[name]
 
 
 @dataclass

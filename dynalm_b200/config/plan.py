@@ -35,9 +35,12 @@ class Spec:
     """kind, width, named parameters, file tensors (local name -> name in the model file)."""
 
     registry = ""          # which registry of dynalm_b200.parts builds it: "mixer", "feed_forward", "norm", "position", "connection"
-    __slots__ = ("kind", "width", "params", "tensors", "_key")
+    __slots__ = ("kind", "width", "params", "tensors", "index", "_key")
 
-    def __init__(self, kind: str, width: int = 0, tensors: Optional[Mapping[str, str]] = None, **params: Any):
+    def __init__(self, kind: str, width: int = 0, tensors: Optional[Mapping[str, str]] = None, index: int = 0, **params: Any):
+        # which piece of a file tensor that several layers share is this part's; like the names, it does not count when
+        # specs are compared
+        object.__setattr__(self, "index", int(index))
         object.__setattr__(self, "kind", kind)
         object.__setattr__(self, "width", int(width))
         object.__setattr__(self, "params", {k: _frozen(v) for k, v in params.items()})
@@ -113,7 +116,8 @@ class FeedForwardSpec(Spec):
 class ConnectionSpec(Spec):
     """How a sublayer sits on the residual stream when that is more than one running sum. kind "hyper" (parameter
     streams = n, tensors in [n], out [n], mix [n, n]): the sublayer reads sum_s in[s] x_s and every stream becomes
-    x_t <- sum_s mix[s, t] x_s + out[t] * result."""
+    x_t <- sum_s mix[s, t] x_s + out[t] * result. kind "sigmoid_gate" (tensors weight [W, W], bias [W]): one stream, x <- x +
+    sigmoid(weight h + bias) * result, h the sublayer's input."""
 
     registry = "connection"
     __slots__ = ()
@@ -187,6 +191,11 @@ class EmbeddingSpec:
     width: int
     scale: float = 1.0
     tensors: Dict[str, str] = field(default_factory=dict, hash=False, compare=False)
+    # pair_rows = n > 0: a row of a second table (tensor "pairs", [n + 1, width]) is added, row (pair_previous * previous
+    # token + pair_current * token) mod n, the last row for a sequence's first token
+    pair_rows: int = 0
+    pair_previous: int = 0
+    pair_current: int = 0
 
 
 @dataclass(frozen=True)

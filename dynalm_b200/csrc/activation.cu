@@ -83,7 +83,44 @@ __global__ void gelu_tanh_vec_kernel(const T* __restrict__ x, T* __restrict__ ou
   reinterpret_cast<Vec16*>(out)[i] = pack<T>(f);
 }
 
+// xIELU with coefficients c = (c0, c1) from memory: c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 at and below it.
+template <typename T>
+__global__ void xielu_kernel(const T* __restrict__ x, T* __restrict__ out, const float* __restrict__ c, size_t n) {
+  const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  out[i] = from_float<T>(xielu_f(to_float(x[i]), c[0], c[1]));
+}
+
+// 16 bytes per access; n counts vectors.
+template <typename T>
+__global__ void xielu_vec_kernel(const T* __restrict__ x, T* __restrict__ out, const float* __restrict__ c, size_t n) {
+  constexpr int V = PerVec<T>::n;
+  const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float c0 = c[0], c1 = c[1];
+  float f[V];
+  unpack<T>(reinterpret_cast<const Vec16*>(x)[i], f);
+#pragma unroll
+  for (int j = 0; j < V; ++j) f[j] = xielu_f(f[j], c0, c1);
+  reinterpret_cast<Vec16*>(out)[i] = pack<T>(f);
+}
+
 }  // namespace dl
+
+// out[i] = xIELU(x[i]) over n contiguous elements (out may be x); coeffs: two float32 on the device.
+DL_EXPORT int dl_xielu(int dtype, const void* x, void* out, const float* coeffs, long long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if ((dtype != 0 && dtype != 1) || coeffs == nullptr) return DL_ERR_UNSUPPORTED;
+  const int vec = dtype == 0 ? 4 : 8;
+  const bool wide = n % vec == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
+  const size_t count = static_cast<size_t>(wide ? n / vec : n);
+  const unsigned blocks = static_cast<unsigned>((count + 255) / 256);
+#define DL_XI(K, T) dl::K<T><<<blocks, 256, 0, stream>>>(static_cast<const T*>(x), static_cast<T*>(out), coeffs, count)
+  if (dtype == 0) { if (wide) DL_XI(xielu_vec_kernel, float); else DL_XI(xielu_kernel, float); }
+  else { if (wide) DL_XI(xielu_vec_kernel, dl::bf16); else DL_XI(xielu_kernel, dl::bf16); }
+#undef DL_XI
+  return dl::launch_status();
+}
 
 // out[i] = gelu_tanh(x[i]) over n contiguous elements (out may be x).
 DL_EXPORT int dl_gelu_tanh(int dtype, const void* x, void* out, long long n, cudaStream_t stream) {

@@ -10,6 +10,9 @@
 //   * a row at position p sees key j <= p if p - j < window (window 0: all) or j < keep_first: the key tiles that hold
 //     kept tokens are walked first, then the tiles of the window;
 //   * with `sink` the denominator of a row's softmax holds one more term exp(0), which carries no value;
+//   * with (rate, step) per head a distance bias rate_h ln(1 + step_h (p - j)) comes off every score; its values for the
+//     127 distances of a 64 x 64 tile of rows and keys are worked out once per tile, in shared memory;
+//   * with a gate the output is multiplied by sigmoid(gate[row, head * VD + column]) on the way out;
 //   * warps whose 16 rows lie past the end of the tile (a one-row tile leaves three of four) skip the arithmetic;
 //   * in a step whose tiles are all single tokens the rows of a tile are the query heads that share a KV head, so the
 //     keys and values of a token are read once for the group.
@@ -58,13 +61,22 @@ __device__ __forceinline__ uint32_t mf_pack(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&p);
 }
 
+__device__ __forceinline__ float mf_log2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float mf_sigmoid(bf16 g) { return 1.0f / (1.0f + mf_exp2(-1.4426950408889634f * to_float(g))); }
+
 // tiles[i] = (request, first row of the step, rows, first position)
 template <int KD, int VD>
 __global__ void __launch_bounds__(MF_THREADS)
 masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ k_cache, size_t k_row,
                     const bf16* __restrict__ v_cache, size_t v_row, const int* __restrict__ block_table, int max_blocks,
                     const int4* __restrict__ tiles, bf16* __restrict__ out, int out_stride, int n_heads, int n_kv_heads,
-                    int page_shift, float scale_log2, int window, int keep_first, int sink, int grp, float* __restrict__ partial) {
+                    int page_shift, float scale_log2, int window, int keep_first, int sink, int grp, float* __restrict__ partial,
+                    const float* __restrict__ rate, const float* __restrict__ dstep, const bf16* __restrict__ gate, int gate_stride) {
+  __shared__ float bias_tab[2][2 * MF_BN];
   constexpr int SUB = MF_TILE / MF_BM;    // blocks per query tile
   constexpr int LDK = KD + 8;             // row strides in elements: 16 bytes of padding keep ldmatrix conflict-free
   constexpr int LDV = VD + 8;
@@ -141,12 +153,26 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
     lo_r[h] = window > 0 ? max(0, pos_r[h] - window + 1) : 0;
   }
   uint32_t qf[KS][4];
+  // with a distance bias the scores are scaled before it comes off (base-2 units), else on the way into the exponential
+  const bool biased = rate != nullptr;
+  const float sl = biased ? 1.0f : scale_log2;
+  float rate_r[2] = {0.0f, 0.0f}, step_r[2] = {0.0f, 0.0f};      // of the lane's rows' heads
+  if (biased) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int hd = grp > 0 ? head + min(warp * 16 + g + h * 8, grp - 1) : head;
+      rate_r[h] = rate[hd];
+      step_r[h] = dstep[hd];
+    }
+  }
 
   for (int it = it_begin; it < it_end; ++it) {
     const int j = tile_of(it);
     const int stage = (it - it_begin) & 1;
     if (it + 1 < it_end) load_kv(tile_of(it + 1), stage ^ 1);
     mf_commit();
+    if (biased && grp == 0)          // entry n: distance pos0 - (last key of the tile) + n
+      bias_tab[stage][tid] = rate_r[0] * mf_log2(fmaf(step_r[0], static_cast<float>(max(0, pos0 - j * MF_BN - (MF_BN - 1) + tid)), 1.0f));
     mf_wait<1>();
     __syncthreads();
     if (warp_live) {
@@ -179,6 +205,19 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
       // scale, mask by position, online softmax; P as bf16 A fragments
       const int key0 = j * MF_BN;
       uint32_t pf[MF_BN / 16][4];
+      if (biased) {
+#pragma unroll
+        for (int i = 0; i < MF_BN / 8; ++i) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int c = i * 8 + 2 * t + (e & 1);                       // the key's place in the tile
+            float b;
+            if (grp == 0) b = bias_tab[stage][warp * 16 + g + (e >> 1) * 8 - c + (MF_BN - 1)];
+            else b = rate_r[e >> 1] * mf_log2(fmaf(step_r[e >> 1], static_cast<float>(max(0, pos0 - key0 - c)), 1.0f));
+            s[i][e] = fmaf(s[i][e], scale_log2, -b);
+          }
+        }
+      }
       const bool edge = it < n_kept || key0 + MF_BN - 1 > (grp > 0 ? pos0 : pos0 + warp * 16) ||
                         (window > 0 && key0 < max(lo_r[0], lo_r[1]));
       float mx[2] = {-INFINITY, -INFINITY};
@@ -200,7 +239,7 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
       for (int h = 0; h < 2; ++h) {
         mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
         mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-        const float m_new = fmaxf(m_run[h], mx[h] * scale_log2);     // the scale is positive
+        const float m_new = fmaxf(m_run[h], mx[h] * sl);     // the scale is positive
         corr[h] = m_new == -INFINITY ? 1.0f : mf_exp2(m_run[h] - m_new);
         m_run[h] = m_new;
         neg_m[h] = m_new == -INFINITY ? 0.0f : -m_new;
@@ -208,8 +247,8 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
       float ls[2] = {0.0f, 0.0f};
 #pragma unroll
       for (int i = 0; i < MF_BN / 8; ++i) {
-        const float p0 = mf_exp2(fmaf(s[i][0], scale_log2, neg_m[0])), p1 = mf_exp2(fmaf(s[i][1], scale_log2, neg_m[0]));
-        const float p2 = mf_exp2(fmaf(s[i][2], scale_log2, neg_m[1])), p3 = mf_exp2(fmaf(s[i][3], scale_log2, neg_m[1]));
+        const float p0 = mf_exp2(fmaf(s[i][0], sl, neg_m[0])), p1 = mf_exp2(fmaf(s[i][1], sl, neg_m[0]));
+        const float p2 = mf_exp2(fmaf(s[i][2], sl, neg_m[1])), p3 = mf_exp2(fmaf(s[i][3], sl, neg_m[1]));
         ls[0] += p0 + p1;
         ls[1] += p2 + p3;
         pf[i >> 1][(i & 1) * 2] = mf_pack(p0, p1);
@@ -285,15 +324,22 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
     // row r of a tile is row row0 + r of the step, or (grp > 0) head `head + r` of row row0
     bf16* dst_a = grp > 0 ? out + static_cast<size_t>(row0) * out_stride + col + r_a * VD : out + static_cast<size_t>(row0 + r_a) * out_stride + col;
     bf16* dst_b = grp > 0 ? out + static_cast<size_t>(row0) * out_stride + col + r_b * VD : out + static_cast<size_t>(row0 + r_b) * out_stride + col;
-    if (r_a < nrows) *reinterpret_cast<uint32_t*>(dst_a) = mf_pack(o[i][0] * inv[0], o[i][1] * inv[0]);
-    if (r_b < nrows) *reinterpret_cast<uint32_t*>(dst_b) = mf_pack(o[i][2] * inv[1], o[i][3] * inv[1]);
+    float f[4] = {inv[0], inv[0], inv[1], inv[1]};
+    if (gate != nullptr) {
+      const bf16* g_a = grp > 0 ? gate + static_cast<size_t>(row0) * gate_stride + col + r_a * VD : gate + static_cast<size_t>(row0 + r_a) * gate_stride + col;
+      const bf16* g_b = grp > 0 ? gate + static_cast<size_t>(row0) * gate_stride + col + r_b * VD : gate + static_cast<size_t>(row0 + r_b) * gate_stride + col;
+      if (r_a < nrows) { f[0] *= mf_sigmoid(g_a[0]); f[1] *= mf_sigmoid(g_a[1]); }
+      if (r_b < nrows) { f[2] *= mf_sigmoid(g_b[0]); f[3] *= mf_sigmoid(g_b[1]); }
+    }
+    if (r_a < nrows) *reinterpret_cast<uint32_t*>(dst_a) = mf_pack(o[i][0] * f[0], o[i][1] * f[1]);
+    if (r_b < nrows) *reinterpret_cast<uint32_t*>(dst_b) = mf_pack(o[i][2] * f[2], o[i][3] * f[3]);
   }
 }
 
 // out[row][head] = sum_p o_p 2^(m_p - M) / (sum_p l_p 2^(m_p - M) + [sink] 2^(-M)), M = max_p m_p (and 0 with the sink):
 // the parts of a row and head that masked_flash_kernel left, in the order of the parts.
 __global__ void masked_flash_merge_kernel(const float* __restrict__ partial, int n_parts, int VD, int n_heads, int sink,
-                                          bf16* __restrict__ out, int out_stride) {
+                                          bf16* __restrict__ out, int out_stride, const bf16* __restrict__ gate, int gate_stride) {
   const int row = blockIdx.x, head = blockIdx.y;
   const float* rec = partial + (static_cast<size_t>(row) * n_heads + head) * n_parts * (VD + 2);
   float M = sink ? 0.0f : -INFINITY;
@@ -310,6 +356,7 @@ __global__ void masked_flash_merge_kernel(const float* __restrict__ partial, int
       const float m = rec[p * (VD + 2)];
       if (m != -INFINITY) acc = fmaf(rec[p * (VD + 2) + 2 + v], mf_exp2(m - M), acc);
     }
+    if (gate != nullptr) acc *= mf_sigmoid(gate[static_cast<size_t>(row) * gate_stride + head * VD + v]);
     out[static_cast<size_t>(row) * out_stride + head * VD + v] = __float2bfloat16_rn(acc * inv);
   }
 }
@@ -318,7 +365,8 @@ template <int KD, int VD>
 int launch_masked_flash(const void* q, int q_stride, const void* kc, long long k_row, const void* vc, long long v_row,
                         const int* block_table, int max_blocks, const int* tiles, int n_tiles, void* out, int out_stride,
                         int n_heads, int n_kv_heads, int page_shift, float scale, int window, int keep_first, int sink,
-                        int grp, int parts, float* partial, int rows, cudaStream_t stream) {
+                        int grp, int parts, float* partial, int rows, const float* rate, const float* dstep, const void* gate,
+                        int gate_stride, cudaStream_t stream) {
   constexpr size_t smem = (static_cast<size_t>(MF_BM + 2 * MF_BN) * (KD + 8) + static_cast<size_t>(2 * MF_BN) * (VD + 8)) * sizeof(bf16);
   static bool configured = false;
   if (!configured) {
@@ -332,11 +380,11 @@ int launch_masked_flash(const void* q, int q_stride, const void* kc, long long k
       static_cast<const bf16*>(q), q_stride, static_cast<const bf16*>(kc), static_cast<size_t>(k_row),
       static_cast<const bf16*>(vc), static_cast<size_t>(v_row), block_table, max_blocks, reinterpret_cast<const int4*>(tiles),
       static_cast<bf16*>(out), out_stride, n_heads, n_kv_heads, page_shift, scale * 1.4426950408889634f, window, keep_first,
-      sink, grp, parts > 1 ? partial : nullptr);
+      sink, grp, parts > 1 ? partial : nullptr, rate, dstep, static_cast<const bf16*>(gate), gate_stride);
   if (parts > 1) {
     dim3 mgrid(rows, n_heads);
     masked_flash_merge_kernel<<<mgrid, VD < 64 ? 32 : 64, 0, stream>>>(partial, parts, VD, n_heads, sink, static_cast<bf16*>(out),
-                                                                      out_stride);
+                                                                      out_stride, static_cast<const bf16*>(gate), gate_stride);
   }
   return launch_status();
 }
@@ -346,13 +394,16 @@ int launch_masked_flash(const void* q, int q_stride, const void* kc, long long k
 // bfloat16 only. tiles: int32 [n_tiles, 4] = (request, first row, rows <= 128, first position), 16-byte aligned.
 // q rows have head h at column h * key_dim, out rows at column h * value_dim. k_cache / v_cache point at the first
 // token's keys / values (KV head j at j * key_dim / j * value_dim); k_row / v_row elements lie between two tokens.
+// rate, dstep: float32 [n_heads] of the distance bias, or both null. gate: rows of gate_stride elements, head h's gate at
+// column h * value_dim, or null.
 // one_token_tiles: every tile is a single token, tile i being row i of the step; parts > 1 then deals a row's key tiles
 // over that many blocks and merges them (partial: scratch). Sizes it takes: key_dim == value_dim in steps of 16 up to 128, and the pairs listed below; others are refused.
 DL_EXPORT int dl_masked_flash_attention(const void* q, int q_stride, const void* k_cache, long long k_row, const void* v_cache,
                                         long long v_row, const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                                         void* out, int out_stride, int n_heads, int n_kv_heads, int key_dim, int value_dim,
                                         int page_size, float scale, int window, int keep_first, int sink, int one_token_tiles,
-                                        int parts, float* partial, cudaStream_t stream) {
+                                        int parts, float* partial, const float* rate, const float* dstep, const void* gate,
+                                        int gate_stride, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   int page_shift = 0;
   while ((1 << page_shift) < page_size) ++page_shift;
@@ -360,6 +411,7 @@ DL_EXPORT int dl_masked_flash_attention(const void* q, int q_stride, const void*
       (out_stride & 1) || !(scale > 0.0f) || (k_row & 7) || (v_row & 7) || window < 0 || keep_first < 0 ||
       (reinterpret_cast<uintptr_t>(k_cache) & 15) || (reinterpret_cast<uintptr_t>(v_cache) & 15))
     return DL_ERR_UNSUPPORTED;
+  if ((rate != nullptr) != (dstep != nullptr)) return DL_ERR_UNSUPPORTED;
   // every tile one token (the caller says so) and heads that share keys: the heads of a KV head are the rows of a tile
   const int group = n_heads / n_kv_heads;
   const int grp = (one_token_tiles && group > 1 && group <= dl::MF_BM) ? group : 0;
@@ -370,7 +422,7 @@ DL_EXPORT int dl_masked_flash_attention(const void* q, int q_stride, const void*
   if (key_dim == K && value_dim == V)                                                                                   \
     return dl::launch_masked_flash<K, V>(q, q_stride, k_cache, k_row, v_cache, v_row, block_table, max_blocks, tiles,   \
                                          n_tiles, out, out_stride, n_heads, n_kv_heads, page_shift, scale, window,      \
-                                         keep_first, sink, grp, parts, partial, n_tiles, stream)
+                                         keep_first, sink, grp, parts, partial, n_tiles, rate, dstep, gate, gate_stride, stream)
   DL_CASE(16, 16); DL_CASE(32, 32); DL_CASE(48, 48); DL_CASE(64, 64); DL_CASE(80, 80); DL_CASE(96, 96); DL_CASE(112, 112);
   DL_CASE(128, 128);
   DL_CASE(32, 16); DL_CASE(48, 32); DL_CASE(64, 32); DL_CASE(96, 48); DL_CASE(96, 64); DL_CASE(128, 64); DL_CASE(64, 128);

@@ -127,6 +127,11 @@ __device__ __forceinline__ float gelu_tanh_bf16(float z) {
   return 0.5f * z * (1.0f + t);
 }
 
+// xIELU: c0 z^2 + z / 2 above zero, c1 (e^z - 1 - z) + z / 2 at and below it.
+__device__ __forceinline__ float xielu_f(float z, float c0, float c1) {
+  return 0.5f * z + (z > 0.0f ? c0 * z * z : c1 * (expm1f(z) - z));
+}
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // Programmatic dependent launch. A kernel launched with the attribute may begin while the kernel before it on

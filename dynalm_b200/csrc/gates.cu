@@ -3,6 +3,7 @@
 //   dl_gelu_mul       out[t, j] = gelu_tanh(gu[t, j]) * gu[t, inner + j]      (a gated feed-forward's activation)
 //   dl_sigmoid_gate   x[t, j] <- x[t, j] * sigmoid(gate[t, j])                (an output gate on concatenated heads)
 //   dl_scaled_sum     out[i] = sa * sum_p a[p][i] + sb * sum_p b[p][i]        (two mixers side by side; float32 out)
+//   dl_token_gate     out[t, j] = gelu_tanh(z[t, j]) * table[id_t, j]         (a small input that depends on the token)
 //   dl_softcap        x[i] <- cap * tanh(x[i] / cap)                          (float32 logits)
 #include "common.cuh"
 
@@ -49,6 +50,36 @@ __global__ void sigmoid_gate_kernel(T* __restrict__ x, int x_stride, const T* __
   *p = from_float<T>(to_float(*p) / (1.0f + expf(-g)));
 }
 
+// 16 bytes per access: n, both pitches and both bases multiples of the vector width.
+template <typename T>
+__global__ void sigmoid_gate_vec_kernel(T* __restrict__ x, int x_stride, const T* __restrict__ gate, int gate_stride, int rows,
+                                        int n) {
+  constexpr int V = PerVec<T>::n;
+  const int per_row = n / V;
+  const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= static_cast<size_t>(rows) * per_row) return;
+  const size_t t = idx / per_row, j = (idx % per_row) * V;
+  float a[V], g[V];
+  Vec16* p = reinterpret_cast<Vec16*>(x + t * x_stride + j);
+  unpack<T>(*p, a);
+  unpack<T>(*reinterpret_cast<const Vec16*>(gate + t * gate_stride + j), g);
+#pragma unroll
+  for (int k = 0; k < V; ++k) a[k] /= 1.0f + expf(-g[k]);
+  *p = pack<T>(a);
+}
+
+template <typename T>
+__global__ void token_gate_kernel(const T* __restrict__ z, const T* __restrict__ table, long long table_stride,
+                                  const int* __restrict__ ids, T* __restrict__ out, int rows, int n, int vocab) {
+  const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= static_cast<size_t>(rows) * n) return;
+  const size_t t = idx / n;
+  const int j = static_cast<int>(idx % n);
+  int id = ck_token(ids[t], vocab);
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  out[idx] = from_float<T>(gelu_tanh_full(to_float(z[idx])) * to_float(table[static_cast<size_t>(id) * table_stride + j]));
+}
+
 template <typename TA, typename TB>
 __global__ void scaled_sum_kernel(const TA* __restrict__ a, int parts_a, size_t stride_a, float sa, const TB* __restrict__ b,
                                   int parts_b, size_t stride_b, float sb, float* __restrict__ out, size_t n) {
@@ -90,9 +121,28 @@ DL_EXPORT int dl_gelu_mul(int dtype, const void* gu, void* out, int rows, int in
 DL_EXPORT int dl_sigmoid_gate(int dtype, void* x, int x_stride, const void* gate, int gate_stride, int rows, int n,
                               cudaStream_t stream) {
   if (rows <= 0 || n <= 0) return 0;
+  const int vec = dtype == 0 ? 4 : 8;
+  if ((dtype == 0 || dtype == 1) && n % vec == 0 && x_stride % vec == 0 && gate_stride % vec == 0 &&
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate)) & 15) == 0) {
+    const unsigned blocks = dl::blocks_for(static_cast<size_t>(rows) * (n / vec));
+    if (dtype == 0) dl::sigmoid_gate_vec_kernel<float><<<blocks, 256, 0, stream>>>(static_cast<float*>(x), x_stride, static_cast<const float*>(gate), gate_stride, rows, n);
+    else dl::sigmoid_gate_vec_kernel<dl::bf16><<<blocks, 256, 0, stream>>>(static_cast<dl::bf16*>(x), x_stride, static_cast<const dl::bf16*>(gate), gate_stride, rows, n);
+    return dl::launch_status();
+  }
   const size_t total = static_cast<size_t>(rows) * n;
   if (dtype == 0) dl::sigmoid_gate_kernel<float><<<dl::blocks_for(total), 256, 0, stream>>>(static_cast<float*>(x), x_stride, static_cast<const float*>(gate), gate_stride, rows, n);
   else if (dtype == 1) dl::sigmoid_gate_kernel<dl::bf16><<<dl::blocks_for(total), 256, 0, stream>>>(static_cast<dl::bf16*>(x), x_stride, static_cast<const dl::bf16*>(gate), gate_stride, rows, n);
+  else return DL_ERR_UNSUPPORTED;
+  return dl::launch_status();
+}
+
+// z, out: contiguous [rows, n] (out may be z); table: rows of table_stride elements, one per token id.
+DL_EXPORT int dl_token_gate(int dtype, const void* z, const void* table, long long table_stride, const int* ids, void* out,
+                            int rows, int n, int vocab, cudaStream_t stream) {
+  if (rows <= 0 || n <= 0) return 0;
+  const unsigned blocks = dl::blocks_for(static_cast<size_t>(rows) * n);
+  if (dtype == 0) dl::token_gate_kernel<float><<<blocks, 256, 0, stream>>>(static_cast<const float*>(z), static_cast<const float*>(table), table_stride, ids, static_cast<float*>(out), rows, n, vocab);
+  else if (dtype == 1) dl::token_gate_kernel<dl::bf16><<<blocks, 256, 0, stream>>>(static_cast<const dl::bf16*>(z), static_cast<const dl::bf16*>(table), table_stride, ids, static_cast<dl::bf16*>(out), rows, n, vocab);
   else return DL_ERR_UNSUPPORTED;
   return dl::launch_status();
 }

@@ -55,7 +55,8 @@ DL_EXPORT int dl_gemm_tcgen05(const void* x, int ldx, const void* w, void* y, in
 
 // A grouped product on the same kernel: runs of a's rows, listed on the device as row tiles (matrix, first row, rows <=
 // 128; n_tiles[0] of them, at most max_row_tiles), each run times its own matrix of w [matrices, N, K]. mode 0: y bf16,
-// 1: y fp32, 4: y bf16 = max(., 0)^2. The experts of a mixture-of-experts feed-forward (csrc/moe.cu writes the list).
+// 1: y fp32, 4: y bf16 = max(., 0)^2, 6: rows 2j and 2j + 1 of a matrix are gate and up row j, y bf16 [rows, N / 2] =
+// silu(gate) * up. The experts of a mixture-of-experts feed-forward (csrc/moe.cu writes the list).
 DL_EXPORT int dl_gemm_tcgen05_grouped(const void* a, int lda, int rows, const void* w, int matrices, int N, int K, void* y,
                                       int ldy, int mode, const int* tiles, const int* n_tiles, int max_row_tiles, int* status,
                                       cudaStream_t stream) {

@@ -23,7 +23,7 @@ template <int BN> struct T5 {
   static constexpr size_t SMEM = static_cast<size_t>(STAGES) * STAGE_BYTES + T5_STORE_BYTES + 1024 /* alignment */ + 256 /* barriers */;
 };
 
-enum { T5_OUT_BF16 = 0, T5_OUT_F32 = 1, T5_OUT_SWIGLU = 2, T5_OUT_QKV_ROPE = 3, T5_OUT_RELU2 = 4, T5_OUT_GELU = 5 };
+enum { T5_OUT_BF16 = 0, T5_OUT_F32 = 1, T5_OUT_SWIGLU = 2, T5_OUT_QKV_ROPE = 3, T5_OUT_RELU2 = 4, T5_OUT_GELU = 5, T5_OUT_PAIRS = 6 };
 enum { T5_ERR_PRODUCER = 1, T5_ERR_MMA = 2, T5_ERR_EPILOGUE = 3 };
 
 // Which output tile a tile number stands for. Tiles are numbered in groups of `group_m` row blocks: inside a
@@ -346,6 +346,26 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
             store_rows_pieces(wlo, whi, my_stage, lane, dst, piece * 32, hd / 2 + piece * 32);
           }
         }
+      } else if (mode == T5_OUT_PAIRS) {
+        // rows 2j and 2j + 1 of W are the gate and up rows of feature j: 128 columns of the tile give 64 of the output
+        for (int c0 = 0; c0 < T5_BN; c0 += 128) {
+          uint4 w[8];
+#pragma unroll
+          for (int hh = 0; hh < 4; ++hh) {
+            uint32_t v[32];
+            tmem_ld32(lane_addr + c0 + hh * 32, v);
+            tmem_ld_wait();
+            auto fin = [&](int j) {
+              const float g = __uint_as_float(v[j]);
+              return __fdividef(g, 1.0f + __expf(-g)) * __uint_as_float(v[j + 1]);
+            };
+#pragma unroll
+            for (int j = 0; j < 32; j += 16)
+              w[hh * 2 + j / 16] = make_uint4(pack2_bf16(fin(j), fin(j + 2)), pack2_bf16(fin(j + 4), fin(j + 6)),
+                                              pack2_bf16(fin(j + 8), fin(j + 10)), pack2_bf16(fin(j + 12), fin(j + 14)));
+          }
+          store_rows_bf16(w, my_stage, lane, static_cast<bf16*>(y), ldy, row0, M, (n0 + c0) / 2, N / 2);   // N / 2 is a multiple of 8
+        }
       } else {
         for (int c0 = 0; c0 < T5_BN; c0 += 64) {
           uint32_t va[32], vb[32];
@@ -548,7 +568,8 @@ static int t5_launch(const void* x, int ldx, const void* w, void* y, int ldy, in
 }
 
 // A grouped product (see T5Groups): a bf16 [rows, K] whose runs of rows are listed in `tiles`, w bf16 [matrices, N, K]
-// contiguous, y [rows, N] bf16 (mode 0, or 4 with the squared ReLU) or fp32 (mode 1). max_row_tiles: the most row tiles
+// contiguous, y [rows, N] bf16 (mode 0, or 4 with the squared ReLU) or fp32 (mode 1), or with mode 6 (gate and up rows of w
+// in turn, N a multiple of 16) y [rows, N / 2] bf16. max_row_tiles: the most row tiles
 // the list can hold; the grid is sized for it and blocks past the list's end do nothing.
 template <class P>
 static int t5_launch_grouped(const void* a, int lda, int rows, const void* w, int matrices, int N, int K, void* y, int ldy,
@@ -558,7 +579,8 @@ static int t5_launch_grouped(const void* a, int lda, int rows, const void* w, in
   if (rows <= 0 || N <= 0 || max_row_tiles <= 0) return 0;
   if (K <= 0 || (K & 7) || (lda & 7) || (reinterpret_cast<uintptr_t>(a) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) ||
       (reinterpret_cast<uintptr_t>(y) & 15) || status == nullptr || tiles == nullptr || n_tiles == nullptr || matrices <= 0 ||
-      (mode != dl::T5_OUT_BF16 && mode != dl::T5_OUT_F32 && mode != dl::T5_OUT_RELU2) ||
+      (mode != dl::T5_OUT_BF16 && mode != dl::T5_OUT_F32 && mode != dl::T5_OUT_RELU2 && mode != dl::T5_OUT_PAIRS) ||
+      (mode == dl::T5_OUT_PAIRS && (N & 15)) ||
       (mode == dl::T5_OUT_F32 ? (N & 3) || (ldy & 3) : (N & 7) || (ldy & 7)) ||
       static_cast<long long>(matrices) * N > (1ll << 30))
     return DL_ERR_UNSUPPORTED;

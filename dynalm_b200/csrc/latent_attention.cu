@@ -14,7 +14,8 @@
 //   dl_latent_attention   one block per (row, head): softmax over the window's records with a sink in the denominator
 //
 // Rotation: interleaved pairs (2i, 2i+1) of the first `rot` of the r numbers turn by position * freq[i]; the angle is
-// formed in double precision from a double frequency table, so that it is exact to float32 at any position.
+// formed in double precision from a double frequency table, so that it is exact to float32 at any position; the turned
+// numbers are multiplied by `mag`. Without a query latent (q_rank 0) dl_latent_prep makes the record alone.
 // Norms, angles, scores, softmax and the weighted sum are float32.
 #include "common.cuh"
 
@@ -22,10 +23,10 @@ namespace dl {
 
 constexpr int LAT_THREADS = 256;
 
-__device__ __forceinline__ void turn(float a, float b, int pos, double freq, float& oa, float& ob) {
+__device__ __forceinline__ void turn(float a, float b, int pos, double freq, float mag, float& oa, float& ob) {
   double s, c;
   sincos(static_cast<double>(pos) * freq, &s, &c);
-  const float cf = static_cast<float>(c), sf = static_cast<float>(s);
+  const float cf = static_cast<float>(c) * mag, sf = static_cast<float>(s) * mag;
   oa = a * cf - b * sf;
   ob = b * cf + a * sf;
 }
@@ -35,21 +36,23 @@ template <typename T>
 __global__ void __launch_bounds__(LAT_THREADS)
 latent_prep_kernel(const T* __restrict__ proj, int proj_stride, int q_rank, int R, int r, int rot,
                    const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
-                   const double* __restrict__ freq, const int* __restrict__ positions,
+                   const double* __restrict__ freq, float mag, const int* __restrict__ positions,
                    const int* __restrict__ row_slot, const int* __restrict__ block_table, int max_blocks,
                    int page_size, T* __restrict__ cq, T* __restrict__ cache) {
   __shared__ float red[33];
   const int row = blockIdx.x, tid = threadIdx.x;
   const T* pr = proj + static_cast<size_t>(row) * proj_stride;
-  float ss = 0.0f;
-  for (int i = tid; i < q_rank; i += LAT_THREADS) {
-    const float v = to_float(pr[i]);
-    ss = fmaf(v, v, ss);
+  float ss = 0.0f, inv;
+  if (q_rank > 0) {
+    for (int i = tid; i < q_rank; i += LAT_THREADS) {
+      const float v = to_float(pr[i]);
+      ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, red);
+    inv = 1.0f / sqrtf(ss / static_cast<float>(q_rank) + eps);
+    for (int i = tid; i < q_rank; i += LAT_THREADS)
+      cq[static_cast<size_t>(row) * q_rank + i] = from_float<T>(to_float(pr[i]) * inv * wq[i]);
   }
-  ss = block_sum(ss, red);
-  float inv = 1.0f / sqrtf(ss / static_cast<float>(q_rank) + eps);
-  for (int i = tid; i < q_rank; i += LAT_THREADS)
-    cq[static_cast<size_t>(row) * q_rank + i] = from_float<T>(to_float(pr[i]) * inv * wq[i]);
   ss = 0.0f;
   for (int i = tid; i < R; i += LAT_THREADS) {
     const float v = to_float(pr[q_rank + i]);
@@ -66,7 +69,7 @@ latent_prep_kernel(const T* __restrict__ proj, int proj_stride, int q_rank, int 
   const T* kr = pr + q_rank + R;
   for (int i = tid; i < rot / 2; i += LAT_THREADS) {
     float a, b;
-    turn(to_float(kr[2 * i]), to_float(kr[2 * i + 1]), pos, freq[i], a, b);
+    turn(to_float(kr[2 * i]), to_float(kr[2 * i + 1]), pos, freq[i], mag, a, b);
     rec[R + 2 * i] = from_float<T>(a);
     rec[R + 2 * i + 1] = from_float<T>(b);
   }
@@ -78,7 +81,7 @@ latent_prep_kernel(const T* __restrict__ proj, int proj_stride, int q_rank, int 
 template <typename T>
 __global__ void rotate_pairs_kernel(const T* __restrict__ q, int q_stride, int head_in, int in_off, T* __restrict__ out,
                                     int out_stride, int head_out, int out_off, int r, int rot,
-                                    const double* __restrict__ freq, const int* __restrict__ positions, int rows, int H) {
+                                    const double* __restrict__ freq, float mag, const int* __restrict__ positions, int rows, int H) {
   const int per = rot / 2 + (r - rot);
   const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (idx >= static_cast<size_t>(rows) * H * per) return;
@@ -87,7 +90,7 @@ __global__ void rotate_pairs_kernel(const T* __restrict__ q, int q_stride, int h
   T* dst = out + static_cast<size_t>(row) * out_stride + static_cast<size_t>(h) * head_out + out_off;
   if (e < rot / 2) {
     float a, b;
-    turn(to_float(src[2 * e]), to_float(src[2 * e + 1]), positions[row], freq[e], a, b);
+    turn(to_float(src[2 * e]), to_float(src[2 * e + 1]), positions[row], freq[e], mag, a, b);
     dst[2 * e] = from_float<T>(a);
     dst[2 * e + 1] = from_float<T>(b);
   } else {
@@ -226,14 +229,14 @@ latent_attention_kernel(const T* __restrict__ qw, int q_stride, const T* __restr
 }  // namespace dl
 
 DL_EXPORT int dl_latent_prep(int dtype, const void* proj, int proj_stride, int q_rank, int R, int r, int rot, const float* wq,
-                             const float* wkv, float eps, const double* freq, const int* positions, const int* row_slot,
+                             const float* wkv, float eps, const double* freq, float mag, const int* positions, const int* row_slot,
                              const int* block_table, int max_blocks, int page_size, void* cq, void* cache, int rows,
                              cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (q_rank <= 0 || R <= 0 || r < 0 || rot < 0 || rot > r || rot % 2 != 0 || page_size <= 0) return DL_ERR_UNSUPPORTED;
+  if (q_rank < 0 || R <= 0 || r < 0 || rot < 0 || rot > r || rot % 2 != 0 || page_size <= 0) return DL_ERR_UNSUPPORTED;
 #define DL_LAUNCH(T)                                                                                                   \
   dl::latent_prep_kernel<T><<<rows, dl::LAT_THREADS, 0, stream>>>(static_cast<const T*>(proj), proj_stride, q_rank, R, r, rot, \
-                                                                  wq, wkv, eps, freq, positions, row_slot, block_table, \
+                                                                  wq, wkv, eps, freq, mag, positions, row_slot, block_table, \
                                                                   max_blocks, page_size, static_cast<T*>(cq), static_cast<T*>(cache))
   if (dtype == 0) DL_LAUNCH(float);
   else if (dtype == 1) DL_LAUNCH(dl::bf16);
@@ -243,7 +246,7 @@ DL_EXPORT int dl_latent_prep(int dtype, const void* proj, int proj_stride, int q
 }
 
 DL_EXPORT int dl_rotate_pairs(int dtype, const void* q, int q_stride, int head_in, int in_off, void* out, int out_stride,
-                              int head_out, int out_off, int r, int rot, const double* freq, const int* positions, int rows,
+                              int head_out, int out_off, int r, int rot, const double* freq, float mag, const int* positions, int rows,
                               int H, cudaStream_t stream) {
   if (rows <= 0 || H <= 0 || r <= 0) return 0;
   if (rot < 0 || rot > r || rot % 2 != 0) return DL_ERR_UNSUPPORTED;
@@ -253,7 +256,7 @@ DL_EXPORT int dl_rotate_pairs(int dtype, const void* q, int q_stride, int head_i
 #define DL_LAUNCH(T)                                                                                                  \
   dl::rotate_pairs_kernel<T><<<blocks, threads, 0, stream>>>(static_cast<const T*>(q), q_stride, head_in, in_off,     \
                                                              static_cast<T*>(out), out_stride, head_out, out_off, r, rot, \
-                                                             freq, positions, rows, H)
+                                                             freq, mag, positions, rows, H)
   if (dtype == 0) DL_LAUNCH(float);
   else if (dtype == 1) DL_LAUNCH(dl::bf16);
   else return DL_ERR_UNSUPPORTED;

@@ -1,17 +1,21 @@
 // Mixture of experts: routing, the grouping of (token, expert) pairs by expert, the experts' products over those
 // groups, and the weighted sum of a token's experts.
 //
-//   dl_moe_route     scores = softmax(router logits) over all experts, float32. Experts form `groups` equal groups of
-//                    neighbours; a group's score is its largest score and only experts of the `keep` best groups can be
-//                    chosen. The `top` allowed experts with the largest scores are chosen (equal scores: the lower
-//                    index), their weights are their scores divided by their sum (+ 1e-20), times `scale`.
+//   dl_moe_route     scores = softmax(router logits) over all experts, or sigmoid of each, float32; choice scores = scores
+//                    (+ a correction per expert). Experts form `groups` equal groups of neighbours; a group's score is
+//                    its largest choice score, or the sum of its two largest, and only experts of the `keep` best groups
+//                    can be chosen. The `top` allowed experts with the largest choice scores are chosen (equal ones: the
+//                    lower index), their weights are their scores, divided by their sum (+ 1e-20) or not, times `scale`.
 //   dl_moe_group     a counting sort of the tokens' pairs by expert: where every pair stands in that order, which pair
 //                    stands at every place, and the list of row tiles (expert, first place, places) for the products.
 //   dl_moe_linear    C[place] = act(A[row of place] W_e^T) for every place of every tile, W_e the matrix of the tile's
 //                    expert: a plain tiled product with float32 accumulation in a fixed order of k (any dtype), and one on
 //                    the tensor cores for bfloat16 (mma.sync m16n8k16, float32 accumulation), with tiles of 32 places for
 //                    steps that bring an expert few and of 128 for steps that bring it many.
-//   dl_moe_combine   y[t] = sum_k weight[t, k] * C[place of pair (t, k)], float32, in the order of k.
+//                    act "pairs": rows 2j and 2j + 1 of a matrix are the gate and up rows of feature j, and the result is
+//                    silu(gate) * up, half as many columns.
+//   dl_moe_combine   y[t] = sum_k weight[t, k] * C[place of pair (t, k)], float32, in the order of k; then, with a shared
+//                    expert's output and its gate logit, + sigmoid(z[t]) * S[t].
 #include "common.cuh"
 
 namespace dl {
@@ -20,59 +24,133 @@ constexpr int MOE_MAX_EXPERTS = 256;
 constexpr int MOE_TM = 32;          // places a tile of the kernels for few places an expert
 constexpr int MOE_TM_WIDE = 128;    // places a tile of the kernel for many
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, int stride, int tokens, int E, int top, int groups,
-                                 int keep, float scale, int* __restrict__ ids, float* __restrict__ weights) {
-  const int t = blockIdx.x * blockDim.x + threadIdx.x;
-  if (t >= tokens) return;
-  float s[MOE_MAX_EXPERTS];
-  const float* z = logits + static_cast<size_t>(t) * stride;
-  float m = -INFINITY;
-  for (int i = 0; i < E; ++i) m = fmaxf(m, z[i]);
-  float sum = 0.0f;
-  for (int i = 0; i < E; ++i) {
-    s[i] = expf(z[i] - m);
-    sum += s[i];
+// One warp per token. Lane l holds the scores of experts l, l + 32, ...; every choice is a warp-wide maximum (equal scores:
+// the lower index).
+constexpr int MOE_PER_LANE = MOE_MAX_EXPERTS / 32;
+constexpr int MOE_ROUTE_WARPS = 4;
+
+__device__ __forceinline__ int moe_warp_best(float v, int index) {      // the index of the largest v, -1 when none is a number
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, index, o);
+    if (oi >= 0 && (index < 0 || ov > v || (ov == v && oi < index))) { v = ov; index = oi; }
   }
-  const float inv = 1.0f / sum;
-  for (int i = 0; i < E; ++i) s[i] *= inv;
-  const int per = E / groups;
-  unsigned long long allowed_lo[MOE_MAX_EXPERTS / 64];      // bit g: group g is kept (groups <= experts <= 256)
-  for (int w = 0; w < MOE_MAX_EXPERTS / 64; ++w) allowed_lo[w] = 0ull;
-  if (keep >= groups) {
-    for (int g = 0; g < groups; ++g) allowed_lo[g >> 6] |= 1ull << (g & 63);
+  return index;
+}
+
+__global__ void __launch_bounds__(MOE_ROUTE_WARPS * 32)
+moe_route_kernel(const float* __restrict__ logits, int stride, int tokens, int E, int top, int groups, int keep,
+                 const float* __restrict__ correction, int sigmoid_scores, int group_top2, int renormalize, float scale,
+                 int* __restrict__ ids, float* __restrict__ weights) {
+  __shared__ float choice_s[MOE_ROUTE_WARPS][MOE_MAX_EXPERTS];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * MOE_ROUTE_WARPS + warp;
+  if (t >= tokens) return;                                     // (no block barrier below: warps work alone)
+  const float* z = logits + static_cast<size_t>(t) * stride;
+  float s[MOE_PER_LANE], c[MOE_PER_LANE];                      // scores, choice scores
+  float m = -INFINITY;
+#pragma unroll
+  for (int k = 0; k < MOE_PER_LANE; ++k) {
+    const int i = lane + 32 * k;
+    s[k] = i < E ? z[i] : -INFINITY;
+    m = fmaxf(m, s[k]);
+  }
+  if (sigmoid_scores) {
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k) s[k] = 1.0f / (1.0f + expf(-s[k]));
   } else {
-    for (int r = 0; r < keep; ++r) {
-      int best = -1;
-      float bs = -INFINITY;
-      for (int g = 0; g < groups; ++g) {
-        if (allowed_lo[g >> 6] >> (g & 63) & 1ull) continue;
-        float gs = -INFINITY;
-        for (int i = g * per; i < (g + 1) * per; ++i) gs = fmaxf(gs, s[i]);
-        if (gs > bs) { bs = gs; best = g; }
+    m = warp_max(m);
+    float sum = 0.0f;
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k) {
+      s[k] = expf(s[k] - m);                                   // 0 past the last expert
+      sum += s[k];
+    }
+    const float inv = 1.0f / warp_sum(sum);
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k) s[k] *= inv;
+  }
+#pragma unroll
+  for (int k = 0; k < MOE_PER_LANE; ++k) {
+    const int i = lane + 32 * k;
+    c[k] = i < E ? s[k] + (correction != nullptr ? correction[i] : 0.0f) : -INFINITY;
+  }
+  const int per = E / groups;
+  if (keep < groups) {
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k)
+      if (lane + 32 * k < E) choice_s[warp][lane + 32 * k] = c[k];
+    __syncwarp();
+    float gs[MOE_PER_LANE];                                    // scores of groups lane, lane + 32, ...
+    bool kept[MOE_PER_LANE];
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k) {
+      const int g = lane + 32 * k;
+      gs[k] = -INFINITY;
+      kept[k] = false;
+      if (g < groups) {
+        float a = -INFINITY, b = -INFINITY;                    // the two largest
+        for (int i = g * per; i < (g + 1) * per; ++i) {
+          const float v = choice_s[warp][i];
+          if (v > a) { b = a; a = v; }
+          else if (v > b) b = v;
+        }
+        gs[k] = group_top2 && per > 1 ? a + b : a;
       }
-      if (best >= 0) allowed_lo[best >> 6] |= 1ull << (best & 63);
+    }
+    for (int r = 0; r < keep; ++r) {
+      float v = -INFINITY;
+      int who = -1;
+#pragma unroll
+      for (int k = 0; k < MOE_PER_LANE; ++k) {
+        const int g = lane + 32 * k;
+        if (g < groups && !kept[k] && (who < 0 || gs[k] > v)) { v = gs[k]; who = g; }
+      }
+      who = moe_warp_best(v, who);
+#pragma unroll
+      for (int k = 0; k < MOE_PER_LANE; ++k)
+        if (who == lane + 32 * k) kept[k] = true;
+    }
+    __syncwarp();                                              // the choice scores have been read: group marks take their place
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k)
+      if (lane + 32 * k < groups) choice_s[warp][lane + 32 * k] = kept[k] ? 1.0f : 0.0f;
+    __syncwarp();
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k) {
+      const int i = lane + 32 * k;
+      if (i < E && choice_s[warp][i / per] == 0.0f) c[k] = -INFINITY;
     }
   }
   float wsum = 0.0f;
   int* my_ids = ids + static_cast<size_t>(t) * top;
   float* my_w = weights + static_cast<size_t>(t) * top;
+  unsigned taken = 0;                                          // bit k: this lane's k-th expert has been chosen
   for (int r = 0; r < top; ++r) {
-    int best = -1;
-    float bs = -INFINITY;
-    for (int i = 0; i < E; ++i) {
-      const int g = i / per;
-      if (!(allowed_lo[g >> 6] >> (g & 63) & 1ull)) continue;
-      bool taken = false;
-      for (int q = 0; q < r; ++q) taken |= my_ids[q] == i;
-      if (!taken && s[i] > bs) { bs = s[i]; best = i; }
+    float v = -INFINITY;
+    int who = -1;
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k)
+      if (!(taken >> k & 1u) && c[k] > v) { v = c[k]; who = lane + 32 * k; }
+    who = moe_warp_best(v, who);
+    if (who < 0) who = 0;                                      // (scores that are not numbers: some expert all the same)
+    float w = 0.0f;
+#pragma unroll
+    for (int k = 0; k < MOE_PER_LANE; ++k)
+      if (who == lane + 32 * k) { taken |= 1u << k; w = s[k]; }
+    w = __shfl_sync(0xffffffffu, w, who & 31);
+    wsum += w;
+    if (lane == 0) {
+      my_ids[r] = who;
+      my_w[r] = renormalize ? w : w * scale;
     }
-    if (best < 0) best = 0;                                  // (scores that are not numbers: some expert all the same)
-    my_ids[r] = best;
-    my_w[r] = s[best];
-    wsum += s[best];
   }
-  const float f = scale / (wsum + 1e-20f);
-  for (int r = 0; r < top; ++r) my_w[r] *= f;
+  if (renormalize) {
+    __syncwarp();
+    const float f = scale / (wsum + 1e-20f);
+    for (int r = lane; r < top; r += 32) my_w[r] *= f;
+  }
 }
 
 // One block. pairs = tokens * top. Outputs: place_of[pair], pair_at[place], tiles[3 * i] = (expert, first place,
@@ -123,6 +201,8 @@ __device__ __forceinline__ float apply_act(float v, int act) {
   if (act == 1) { v = fmaxf(v, 0.0f); v = v * v; }
   return v;
 }
+constexpr int MOE_ACT_PAIRS = 2;
+__device__ __forceinline__ float silu_times(float g, float u) { return g / (1.0f + expf(-g)) * u; }
 
 // Plain tiled product: tile = 32 places x 64 features, 256 threads, 2 x 4 results a thread, k in steps of 16.
 // A row of place p: a[(rows_of ? rows_of[pair_at[p]] / div : p) * lda]; W of expert x: w + x * N * K, [N, K].
@@ -169,6 +249,14 @@ moe_linear_simt_kernel(const T* __restrict__ a, int lda, const int* __restrict__
   for (int i = 0; i < 2; ++i) {
     const int r = ty * 2 + i;
     if (r >= np) continue;
+    if (act == MOE_ACT_PAIRS) {
+#pragma unroll
+      for (int j = 0; j < 4; j += 2) {
+        const int n = n0 + tx * 4 + j;
+        if (n + 1 < N) c[static_cast<size_t>(p0 + r) * ldc + n / 2] = from_float<TO>(silu_times(acc[i][j], acc[i][j + 1]));
+      }
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
@@ -278,6 +366,11 @@ moe_linear_tc_kernel(const bf16* __restrict__ a, int lda, const int* __restrict_
         const int r = wm * (TM / WM) + mi * 16 + g + 8 * h;
         const int n = n0 + wn * (TN / WN) + ni * 8 + q * 2;
         if (r >= np) continue;
+        if (act == MOE_ACT_PAIRS) {
+          if (n + 1 < N)
+            c[static_cast<size_t>(p0 + r) * ldc + n / 2] = from_float<TO>(silu_times(acc[mi][ni][2 * h], acc[mi][ni][2 * h + 1]));
+          continue;
+        }
         TO* dst = c + static_cast<size_t>(p0 + r) * ldc + n;
         if (n < N) dst[0] = from_float<TO>(apply_act<bf16>(acc[mi][ni][2 * h], act));
         if (n + 1 < N) dst[1] = from_float<TO>(apply_act<bf16>(acc[mi][ni][2 * h + 1], act));
@@ -294,28 +387,56 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ a, int lda16, const 
   out[i] = a[static_cast<size_t>(pair_at[place] / top_div) * lda16 + c];
 }
 
-template <typename TO>
+// V columns a thread (4 where every row starts on a 16-byte boundary).
+template <typename TO, typename TS, int V>
 __global__ void moe_combine_kernel(const float* __restrict__ c, int width, const int* __restrict__ place_of,
-                                   const float* __restrict__ weights, int top, TO* __restrict__ y, size_t total) {
+                                   const float* __restrict__ weights, int top, const TS* __restrict__ shared, int parts,
+                                   size_t part_stride, const float* __restrict__ shared_z, int z_stride, TO* __restrict__ y,
+                                   size_t total) {
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= total) return;
-  const size_t t = i / width;
-  const int col = static_cast<int>(i % width);
-  float sum = 0.0f;
-  for (int k = 0; k < top; ++k)
-    sum = fmaf(weights[t * top + k], c[static_cast<size_t>(place_of[t * top + k]) * width + col], sum);
-  y[i] = from_float<TO>(sum);
+  const int per_row = width / V;
+  const size_t t = i / per_row;
+  const int col = static_cast<int>(i % per_row) * V;
+  float sum[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) sum[j] = 0.0f;
+  for (int k = 0; k < top; ++k) {
+    const float w = weights[t * top + k];
+    const float* row = c + static_cast<size_t>(place_of[t * top + k]) * width + col;
+    if constexpr (V == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(row);
+      sum[0] = fmaf(w, v.x, sum[0]); sum[1] = fmaf(w, v.y, sum[1]); sum[2] = fmaf(w, v.z, sum[2]); sum[3] = fmaf(w, v.w, sum[3]);
+    } else {
+      sum[0] = fmaf(w, row[0], sum[0]);
+    }
+  }
+  if (shared != nullptr) {
+    const float g = 1.0f / (1.0f + expf(-shared_z[t * z_stride]));
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      float v = 0.0f;
+      for (int p = 0; p < parts; ++p) v += to_float(shared[p * part_stride + t * width + col + j]);
+      sum[j] = fmaf(g, v, sum[j]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) y[t * width + col + j] = from_float<TO>(sum[j]);
 }
 
 }  // namespace dl
 
-DL_EXPORT int dl_moe_route(const float* logits, int stride, int tokens, int E, int top, int groups, int keep, float scale,
-                           int* ids, float* weights, cudaStream_t stream) {
+// correction: float32 [E] or null; sigmoid_scores 0: softmax over all experts; group_top2 0: a group's largest choice score.
+DL_EXPORT int dl_moe_route(const float* logits, int stride, int tokens, int E, int top, int groups, int keep,
+                           const float* correction, int sigmoid_scores, int group_top2, int renormalize, float scale, int* ids,
+                           float* weights, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (E <= 0 || E > dl::MOE_MAX_EXPERTS || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
       top > keep * (E / groups))
     return DL_ERR_UNSUPPORTED;
-  dl::moe_route_kernel<<<(tokens + 127) / 128, 128, 0, stream>>>(logits, stride, tokens, E, top, groups, keep, scale, ids, weights);
+  constexpr int WARPS = dl::MOE_ROUTE_WARPS;
+  dl::moe_route_kernel<<<(tokens + WARPS - 1) / WARPS, WARPS * 32, 0, stream>>>(logits, stride, tokens, E, top, groups, keep, correction,
+                                                                               sigmoid_scores, group_top2, renormalize, scale, ids, weights);
   return dl::launch_status();
 }
 
@@ -328,14 +449,15 @@ DL_EXPORT int dl_moe_group(const int* ids, int pairs, int E, int* place_of, int*
 }
 
 // dtype of a and w: 0 float32, 1 bfloat16; out_dtype of c likewise. pair_at null: the rows of a are the places
-// themselves; else the row of a place is pair_at[place] / top_div. act: 0 none, 1 squared ReLU. tensor_cores: use the
+// themselves; else the row of a place is pair_at[place] / top_div. act: 0 none, 1 squared ReLU, 2 pairs (N even; c has N / 2
+// columns). tensor_cores: use the
 // mma.sync kernels where they apply (bfloat16, K a multiple of 64, rows of a and w on 16-byte boundaries).
 // tile_rows: the places a tile as dl_moe_group was told: 32, or 128 for the wide tensor-core kernel (bfloat16 only).
 DL_EXPORT int dl_moe_linear(int dtype, int out_dtype, const void* a, int lda, const int* pair_at, int top_div, const void* w,
                             int N, int K, void* c, int ldc, const int* tiles, const int* n_tiles, int max_tiles, int act,
                             int tensor_cores, int tile_rows, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
-  if (N <= 0 || K <= 0 || top_div <= 0 || max_tiles > 65535) return DL_ERR_UNSUPPORTED;
+  if (N <= 0 || K <= 0 || top_div <= 0 || max_tiles > 65535 || act < 0 || act > 2 || (act == 2 && (N & 1))) return DL_ERR_UNSUPPORTED;
   const bool wide = tile_rows == dl::MOE_TM_WIDE;
   if (!wide && tile_rows != dl::MOE_TM) return DL_ERR_UNSUPPORTED;
   const bool tc_ok = dtype == 1 && tensor_cores && K % 64 == 0 && lda % 8 == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0 &&
@@ -395,13 +517,30 @@ DL_EXPORT int dl_moe_gather(const void* a, int lda, const int* pair_at, int top_
   return dl::launch_status();
 }
 
+// shared: the shared expert's output [parts][tokens, width] (part_stride elements apart; shared_dtype) with its gate's logits
+// at shared_z[t * z_stride] (float32), or null.
 DL_EXPORT int dl_moe_combine(int out_dtype, const float* c, int width, const int* place_of, const float* weights, int top,
-                             void* y, int tokens, cudaStream_t stream) {
+                             int shared_dtype, const void* shared, int parts, long long part_stride, const float* shared_z,
+                             int z_stride, void* y, int tokens, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  const size_t total = static_cast<size_t>(tokens) * width;
+  if (shared != nullptr && (parts <= 0 || shared_z == nullptr)) return DL_ERR_UNSUPPORTED;
+  const bool wide = width % 4 == 0 && (reinterpret_cast<uintptr_t>(c) & 15) == 0;
+  const size_t total = static_cast<size_t>(tokens) * (wide ? width / 4 : width);
   const unsigned blocks = static_cast<unsigned>((total + 255) / 256);
-  if (out_dtype == 0) dl::moe_combine_kernel<float><<<blocks, 256, 0, stream>>>(c, width, place_of, weights, top, static_cast<float*>(y), total);
-  else if (out_dtype == 1) dl::moe_combine_kernel<dl::bf16><<<blocks, 256, 0, stream>>>(c, width, place_of, weights, top, static_cast<dl::bf16*>(y), total);
+#define DL_MC(TO, TS, V)                                                                                              \
+  dl::moe_combine_kernel<TO, TS, V><<<blocks, 256, 0, stream>>>(c, width, place_of, weights, top, static_cast<const TS*>(shared), \
+                                                                parts, static_cast<size_t>(part_stride), shared_z, z_stride,     \
+                                                                static_cast<TO*>(y), total)
+#define DL_MCV(TO, TS)            \
+  do {                            \
+    if (wide) DL_MC(TO, TS, 4);   \
+    else DL_MC(TO, TS, 1);        \
+  } while (0)
+  if (out_dtype == 0 && shared_dtype == 0) DL_MCV(float, float);
+  else if (out_dtype == 1 && shared_dtype == 0) DL_MCV(dl::bf16, float);
+  else if (out_dtype == 1 && shared_dtype == 1) DL_MCV(dl::bf16, dl::bf16);
   else return DL_ERR_UNSUPPORTED;
+#undef DL_MCV
+#undef DL_MC
   return dl::launch_status();
 }

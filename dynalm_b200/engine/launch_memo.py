@@ -74,9 +74,9 @@ class _Layout:
 
 
 class _Record:
-    __slots__ = ("calls", "own", "library", "pending", "pending_scale", "pending2", "as_input", "streams", "parts")
+    __slots__ = ("calls", "own", "library", "pending", "pending_scale", "pending2", "as_input", "streams", "parts", "gate", "via")
 
-    def __init__(self, calls, pending, pending_scale, pending2=None, as_input=None, streams=None, parts=1):
+    def __init__(self, calls, pending, pending_scale, pending2=None, as_input=None, streams=None, parts=1, gate=None, via=False):
         # [(function, arguments, ((argument index, tensor index, offset or None for the tensor itself), ...))]
         self.calls = calls
         self.library = sum(1 for f, _, _ in calls if f is ops.library_mm_again)
@@ -87,6 +87,8 @@ class _Record:
         self.as_input = as_input
         self.streams = streams
         self.parts = parts
+        self.gate = gate
+        self.via = via              # the pending result joins through a part of the layer (its bias, its norm weight)
 
 
 def _patches(calls, layout: _Layout):
@@ -148,6 +150,8 @@ class LayerLaunchMemo:
                None if second is None else (second.data_ptr(), tuple(second.shape), second.dtype),
                None if stream.as_input is None else stream.as_input.data_ptr(),
                None if stream.streams is None else (stream.streams.data_ptr(), stream.parts, stream.link is not None),
+               None if stream.gate is None else (stream.gate.data_ptr(), stream.gate.stride(), stream.gate.dtype),
+               stream.via is not None,
                layout.signature)
         if key in self.records:
             record = self.records[key]
@@ -168,6 +172,8 @@ class LayerLaunchMemo:
             REPLAYED_LAYERS += 1
             stream.pending, stream.pending_scale, stream.pending2 = record.pending, record.pending_scale, record.pending2
             stream.as_input = record.as_input
+            stream.gate = record.gate
+            stream.via = block.last_via() if record.via else None      # this layer's own, not the recorded one
             if record.streams is not None:
                 # the pending result belongs to the last sublayer of THIS layer: its stream connection, not the recorded one
                 stream.streams, stream.parts, stream.link = record.streams, record.parts, block.last_link()
@@ -178,5 +184,6 @@ class LayerLaunchMemo:
             self.records[key] = None             # some work was not written down: this kind runs through its parts
         else:
             self.records[key] = _Record(_patches(recording.calls, layout), stream.pending, stream.pending_scale,
-                                        stream.pending2, stream.as_input, stream.streams, stream.parts)
+                                        stream.pending2, stream.as_input, stream.streams, stream.parts, stream.gate,
+                                        stream.via is not None)
         return stream

@@ -7,6 +7,7 @@ allocates its scratch through the runtime's workspace; `forward` looks nothing u
 
 from __future__ import annotations
 
+import dataclasses
 from typing import Dict, List, Optional
 
 import torch
@@ -71,8 +72,27 @@ class Decoder:
         return plans
 
     def cache_specs(self) -> List[Optional[CacheSpec]]:
-        """Per run-order entry: the cache it owns, or None when it owns none."""
-        return [None if run.cache_of is not None else self.blocks[run.layer].cache_spec() for run in self.order]
+        """Per run-order entry: the cache it owns, or None when it owns none (an entry that reads another's pages may still
+        keep a state row of its own). Behind the run order, when it keeps any, the state of the embedding."""
+        specs = []
+        for run in self.order:
+            block = self.blocks[run.layer]
+            if run.cache_of is None:
+                specs.append(block.cache_spec())
+            else:
+                own = getattr(block, "reader_state_spec", None)
+                specs.append(own() if own is not None else None)
+        embedding = self.embedding.cache_spec()
+        return specs + ([embedding] if embedding is not None else [])
+
+    def cache_views(self, cache, tables) -> list:
+        """The view every run-order entry is handed (`cache`: the manager, `tables`: its block tables on the device): its
+        own, or the pages of the entry it reads with its own state row beside them; behind them the embedding's."""
+        views = [cache.view(i, tables) for i in range(len(self.order))]
+        for i, run in enumerate(self.order):
+            if run.cache_of is not None:
+                views[i] = dataclasses.replace(views[run.cache_of], state=views[i])
+        return views + ([cache.view(len(self.order), tables)] if self.embedding.cache_spec() is not None else [])
 
     def weight_bytes(self) -> int:
         seen, n = set(), 0
@@ -84,17 +104,16 @@ class Decoder:
         return n
 
     def hidden(self, ctx, caches) -> ResidualStream:
-        """Run embedding and all blocks; `caches[i]` is the CacheView of run-order entry i (or None)."""
-        x = self.embedding.forward(ctx.token_ids, ctx.num_tokens)
+        """Run embedding and all blocks; `caches` as `cache_views` gives them."""
+        x = self.embedding.forward(ctx, caches[len(self.order)] if len(caches) > len(self.order) else None)
         stream = ResidualStream(x)
         memo = launch_memo.LayerLaunchMemo(self._run_layouts, self._run_kinds) if launch_memo.ENABLED else None
         for i, run in enumerate(self.order):
-            owner = i if run.cache_of is None else run.cache_of
             block = self.blocks[run.layer]
             if memo is None:
-                stream = block.forward(stream, ctx, caches[owner], run.cache_of is None)
+                stream = block.forward(stream, ctx, caches[i], run.cache_of is None)
             else:
-                stream = memo.run(i, block, stream, ctx, caches[owner], run.cache_of is None)
+                stream = memo.run(i, block, stream, ctx, caches[i], run.cache_of is None)
         return stream
 
     def logits(self, stream: ResidualStream, ctx, out: torch.Tensor) -> torch.Tensor:
@@ -106,6 +125,12 @@ class Decoder:
 
     def _final_norm(self, stream: ResidualStream, normed: torch.Tensor, ctx) -> None:
         """The final norm of the wanted rows, with what the last block left pending added on the way in."""
+        if stream.via is not None and hasattr(self.final_norm, "forward_update"):
+            # the last sublayer's result joins through a gate or a norm of its own
+            self.final_norm.forward_update(stream, normed, rows=ctx.logit_rows)
+            return
+        if stream.via is not None:
+            stream.flush()
         if stream.streams is not None and hasattr(self.final_norm, "forward_stream"):
             # a stream of several parts: the norm reads their plain sum, after the last sublayer's update
             self.final_norm.forward_stream(stream.streams, stream.parts, normed, delta=stream.pending, link=stream.link,

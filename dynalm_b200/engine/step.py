@@ -383,7 +383,7 @@ class StepFunction:
 
     def caches(self):
         if self._caches is None:
-            self._caches = [self.cache.view(i, self.batcher.tables) for i in range(len(self.model.order))]
+            self._caches = self.model.cache_views(self.cache, self.batcher.tables)
         return self._caches
 
     def step(self, entries: Sequence[StepEntry], reserve: bool = True, token_feedback=None,

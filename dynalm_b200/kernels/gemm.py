@@ -206,6 +206,14 @@ def linear_act(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int, activat
     return act
 
 
+def linear_xielu(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int, coeffs: torch.Tensor) -> torch.Tensor:
+    """xIELU(x W^T) with the coefficients `coeffs` (ops.xielu): the product followed by the activation kernel."""
+    act = runtime.buffer("ffn_act", (x.shape[0], inner))
+    linear(x, w_up, act)
+    ops.xielu(act, act, coeffs)
+    return act
+
+
 def linear_relu2(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int) -> torch.Tensor:
     """max(x W^T, 0)^2 (see linear_act)."""
     return linear_act(x, w_up, runtime, inner, "relu2")

@@ -22,14 +22,20 @@ _P, _I, _F, _L = c_void_p, c_int, c_float, c_longlong
 
 # library -> function -> argument types
 _SIGNATURES = {
-    "embedding": {"dl_embed": [_I, _P, _P, _P, _I, _I, _I, _F, _P]},
+    "embedding": {"dl_embed": [_I, _P, _P, _P, _I, _I, _I, _F, _P],
+                  "dl_embed_pairs": [_I, _P, _P, _P, _P, _P, _P, _P, _P, _L, _P, _I, _I, _I, _F, _I, _L, _L, _P]},
+    "residual_norm": {"dl_residual_norm": [_I, _I, _I, _P, _I, _P, _I, _L, _F, _P, _L, _P, _P, _F, _P, _I, _P, _P, _F, _P, _P,
+                                           _I, _I, _P, _L, _P]},
+    "conv_cache": {
+        "dl_conv_cache": [_I, _P, _L, _I, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _P, _L, _P, _L, _P, _L, _I, _P],
+        "dl_conv_keep_many": [_I, _P, _L, _I, _I, _P, _L, _P, _P, _I, _P]},
     "norm": {
         "dl_rmsnorm": [_I, _I, _P, _P, _F, _P, _F, _P, _P, _I, _I, _I, _I, _L, _P, _L, _P],
         "dl_residual_add": [_I, _P, _P, _F, _L, _I, _L, _P],
         "dl_rmsnorm_pair": [_I, _P, _P, _I, _I, _L, _P, _I, _I, _L, _P, _P, _F, _P, _P, _P, _I, _I, _I, _P],
     },
     "activation": {"dl_silu_mul": [_I, _P, _P, _I, _I, _P], "dl_relu2": [_I, _P, _P, _L, _P],
-                   "dl_gelu_tanh": [_I, _P, _P, _L, _P]},
+                   "dl_gelu_tanh": [_I, _P, _P, _L, _P], "dl_xielu": [_I, _P, _P, _P, _L, _P]},
     "norm_after_sum": {
         "dl_norm_after_sum": [_I, _I, _P, _P, _I, _L, _P, _F, _P, _F, _P, _I, _I, _P],
         "dl_cast_rows": [_I, _P, _P, _L, _P]},
@@ -41,8 +47,8 @@ _SIGNATURES = {
                         _P, _P],
         "dl_gated_group_norm": [_I, _P, _P, _I, _P, _F, _P, _I, _I, _I, _P]},
     "latent_attention": {
-        "dl_latent_prep": [_I, _P, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _P, _P, _I, _I, _P, _P, _I, _P],
-        "dl_rotate_pairs": [_I, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _P, _I, _I, _P],
+        "dl_latent_prep": [_I, _P, _I, _I, _I, _I, _I, _P, _P, _F, _P, _F, _P, _P, _P, _I, _I, _P, _P, _I, _P],
+        "dl_rotate_pairs": [_I, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _F, _P, _I, _I, _P],
         "dl_head_linear": [_I, _P, _I, _I, _I, _P, _I, _P, _I, _I, _P, _I, _I, _I, _I, _P],
         "dl_latent_attention": [_I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P]},
     "head_linear_tc": {
@@ -69,7 +75,7 @@ _SIGNATURES = {
         "dl_paged_attention_generic_kv": [_I, _P, _I, _P, _L, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I,
                                           _P],
         "dl_paged_attention_generic_masked": [_I, _P, _I, _P, _L, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F,
-                                              _I, _I, _I, _P]},
+                                              _I, _I, _I, _P, _P, _P]},
     "delta_rule": {
         "dl_delta_rule": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
         "dl_delta_rule_step": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
@@ -84,7 +90,7 @@ _SIGNATURES = {
                                       _P]},
     "attention_masked_flash": {
         "dl_masked_flash_attention": [_P, _I, _P, _L, _P, _L, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _I, _P,
-                                      _P]},
+                                      _P, _P, _P, _I, _P]},
     "layer_norm": {
         "dl_stream_layer_norm": [_I, _I, _P, _I, _I, _P, _P, _I, _L, _F, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _P],
         "dl_stream_sum": [_I, _P, _I, _I, _P, _I, _L, _F, _P, _P, _P, _I, _P]},
@@ -92,15 +98,16 @@ _SIGNATURES = {
         "dl_gla_decay": [_P, _I, _I, _I, _P, _F, _P],
         "dl_gla_scan": [_I, _P, _I, _I, _I, _I, _P, _I, _F, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P]},
     "moe": {
-        "dl_moe_route": [_P, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P],
+        "dl_moe_route": [_P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P],
         "dl_moe_group": [_P, _I, _I, _P, _P, _P, _P, _I, _P],
         "dl_moe_linear": [_I, _I, _P, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
         "dl_moe_gather": [_P, _I, _P, _I, _P, _I, _I, _P],
-        "dl_moe_combine": [_I, _P, _I, _P, _P, _I, _P, _I, _P]},
+        "dl_moe_combine": [_I, _P, _I, _P, _P, _I, _I, _P, _I, _L, _P, _I, _P, _I, _P]},
     "gates": {
         "dl_gelu_mul": [_I, _P, _P, _I, _I, _P],
         "dl_sigmoid_gate": [_I, _P, _I, _P, _I, _I, _I, _P],
         "dl_scaled_sum": [_I, _P, _I, _L, _F, _I, _P, _I, _L, _F, _P, _L, _P],
+        "dl_token_gate": [_I, _P, _P, _L, _P, _P, _I, _I, _I, _P],
         "dl_softcap": [_P, _L, _F, _P],
         "dl_add_bias": [_I, _P, _L, _P, _I, _I, _P]},
     "norm_sandwich": {
@@ -733,40 +740,41 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps
                                               rows, inner, parts, _stream()), "gated_group_norm")
 
 
-def latent_prep(proj: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, rot: int, q_weight: torch.Tensor,
+def latent_prep(proj: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, rot: int, q_weight: Optional[torch.Tensor],
                 kv_weight: torch.Tensor, eps: float, freq: Optional[torch.Tensor], positions: torch.Tensor,
                 row_slot: torch.Tensor, block_table: torch.Tensor, cache: torch.Tensor, page_size: int,
-                cq: torch.Tensor) -> None:
+                cq: Optional[torch.Tensor], mag: float = 1.0) -> None:
     """Per row of proj = [query latent | latent | key part | ...]: cq = rmsnorm(query latent) * q_weight, and the row's
     record [rmsnorm(latent) * kv_weight | key part with its first `rot` numbers turned by the position] into the paged
-    cache [pages, page_size, kv_rank + rot_dim]. freq: float64 [rot / 2]. See csrc/latent_attention.cu."""
+    cache [pages, page_size, kv_rank + rot_dim]. freq: float64 [rot / 2]; mag multiplies the turned numbers. q_rank 0: there
+    is no query latent (q_weight and cq None). See csrc/latent_attention.cu."""
     _cuda(proj, q_weight, kv_weight, freq, positions, row_slot, block_table, cache, cq)
     _rows_contiguous(proj, "proj")
     rows = proj.shape[0]
     if proj.shape[1] < q_rank + kv_rank + rot_dim:
         raise InvalidArgument("latent_prep: proj is narrower than its three pieces")
-    if q_weight.dtype != torch.float32 or q_weight.numel() != q_rank or kv_weight.dtype != torch.float32 or kv_weight.numel() != kv_rank:
+    if (q_rank and (q_weight.dtype != torch.float32 or q_weight.numel() != q_rank)) or kv_weight.dtype != torch.float32 or kv_weight.numel() != kv_rank:
         raise InvalidArgument("latent_prep: norm weights float32 [q_rank] and [kv_rank]")
     if rot and (freq is None or freq.dtype != torch.float64 or freq.numel() != rot // 2):
         raise InvalidArgument("latent_prep: freq float64 [rot / 2]")
     if cache.dtype != proj.dtype or not cache.is_contiguous() or cache.dim() != 3 or cache.shape[1] != page_size \
             or cache.shape[2] != kv_rank + rot_dim:
         raise InvalidArgument("latent_prep: the cache must be contiguous [pages, page_size, kv_rank + rot_dim] of proj's dtype")
-    if cq.dtype != proj.dtype or cq.shape != (rows, q_rank) or not cq.is_contiguous():
+    if q_rank and (cq.dtype != proj.dtype or cq.shape != (rows, q_rank) or not cq.is_contiguous()):
         raise InvalidArgument("latent_prep: cq contiguous [rows, q_rank] of proj's dtype")
     if block_table.dtype != torch.int32 or block_table.stride(-1) != 1:
         raise InvalidArgument("latent_prep: block_table must be int32 rows")
     check_limits("latent_attention", pages=cache.shape[0], requests=block_table.shape[0], rows=rows)
     _check(_fn("latent_attention", "dl_latent_prep")(
         dtype_code(proj.dtype), _p(proj), proj.stride(0), q_rank, kv_rank, rot_dim, rot, _p(q_weight), _p(kv_weight), eps,
-        _p(freq), _p(positions), _p(row_slot), _p(block_table), block_table.stride(0), page_size, _p(cq), _p(cache), rows,
+        _p(freq), mag, _p(positions), _p(row_slot), _p(block_table), block_table.stride(0), page_size, _p(cq), _p(cache), rows,
         _stream()), "latent_prep")
 
 
 def rotate_pairs(q: torch.Tensor, head_in: int, in_off: int, out: torch.Tensor, head_out: int, out_off: int, r: int,
-                 rot: int, freq: Optional[torch.Tensor], positions: torch.Tensor, heads: int) -> None:
+                 rot: int, freq: Optional[torch.Tensor], positions: torch.Tensor, heads: int, mag: float = 1.0) -> None:
     """out[row, h * head_out + out_off + i] = q[row, h * head_in + in_off + i] for i < r, the first `rot` of them
-    turned in interleaved pairs (2i, 2i + 1) by position * freq[i]."""
+    turned in interleaved pairs (2i, 2i + 1) by position * freq[i] and multiplied by mag."""
     _cuda(q, out, freq, positions)
     _rows_contiguous(q, "q")
     _rows_contiguous(out, "out")
@@ -777,7 +785,7 @@ def rotate_pairs(q: torch.Tensor, head_in: int, in_off: int, out: torch.Tensor, 
         raise InvalidArgument("rotate_pairs: freq float64 [rot / 2]")
     _check(_fn("latent_attention", "dl_rotate_pairs")(
         dtype_code(q.dtype), _p(q), q.stride(0), head_in, in_off, _p(out), out.stride(0), head_out, out_off, r, rot,
-        _p(freq), _p(positions), q.shape[0], heads, _stream()), "rotate_pairs")
+        _p(freq), mag, _p(positions), q.shape[0], heads, _stream()), "rotate_pairs")
 
 
 def head_linear(x: torch.Tensor, head_in: int, n_in: int, w: torch.Tensor, out: torch.Tensor, head_out: int,
@@ -1778,14 +1786,24 @@ def qk_proj_norm_cache(proj: torch.Tensor, wq: Optional[torch.Tensor], wk: Optio
         v_row, proj.shape[0], heads, kv_heads, dim, vdim, page_size, _stream()), "qk_proj_norm_cache")
 
 
+def _distance_bias(rate: Optional[torch.Tensor], step: Optional[torch.Tensor], heads: int) -> None:
+    if (rate is None) != (step is None) or (rate is not None and any(t.dtype != torch.float32 or t.numel() != heads
+                                                                     or not t.is_contiguous() for t in (rate, step))):
+        raise InvalidArgument("attention: the distance bias is float32 [heads] of rates and of steps, or neither")
+
+
 def paged_attention_generic_kv(q: torch.Tensor, k_cache: torch.Tensor, k_row: int, v_cache: torch.Tensor, v_row: int,
                                block_table: torch.Tensor, positions: torch.Tensor, row_request: torch.Tensor,
                                out: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, vdim: int, page_size: int,
-                               scale: float, window: int = 0, keep_first: int = 0, sink: bool = False) -> None:
+                               scale: float, window: int = 0, keep_first: int = 0, sink: bool = False,
+                               rate: Optional[torch.Tensor] = None, step: Optional[torch.Tensor] = None) -> None:
     """paged_attention_generic with keys of head_dim and values of vdim numbers: k_cache / v_cache point at the first
     token's keys / values (KV head j at j * head_dim / j * vdim), k_row / v_row elements lie between two tokens.
     out: rows with head h at column h * vdim. keep_first: keys at positions below it stay visible behind the window;
-    sink: the softmax's denominator holds one more term of score 0, which carries no value."""
+    sink: the softmax's denominator holds one more term of score 0, which carries no value; rate, step (float32 [n_heads],
+    both or neither): rate_h ln(1 + step_h * distance) comes off every score."""
+    _cuda(rate, step)
+    _distance_bias(rate, step, n_heads)
     _cuda(q, k_cache, v_cache, block_table, positions, row_request, out)
     _rows_contiguous(q, "q")
     _rows_contiguous(out, "out")
@@ -1799,7 +1817,8 @@ def paged_attention_generic_kv(q: torch.Tensor, k_cache: torch.Tensor, k_row: in
     _check(_fn("attention_generic", "dl_paged_attention_generic_masked")(
         dtype_code(q.dtype), _p(q), q.stride(0), _p(k_cache), k_row, _p(v_cache), v_row, _p(block_table),
         block_table.stride(0), _p(positions), _p(row_request), _p(out), out.stride(0), q.shape[0], n_heads, n_kv_heads,
-        head_dim, vdim, page_size, scale, window, int(keep_first), 1 if sink else 0, _stream()), "paged_attention_generic_kv")
+        head_dim, vdim, page_size, scale, window, int(keep_first), 1 if sink else 0, _p(rate), _p(step), _stream()),
+           "paged_attention_generic_kv")
 
 
 def gelu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
@@ -1983,6 +2002,7 @@ def gla_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, z: torch.Te
 
 
 MOE_MAX_EXPERTS = 256
+MOE_ACTS = {"none": 0, "relu2": 1, "pairs": 2}
 MOE_TILE_ROWS = 32          # places a tile of the kernels for few places an expert
 MOE_WIDE_TILE_ROWS = 128    # of the wide tensor-core kernel
 MOE_WIDE_FROM = int(os.environ.get("DYNALM_MOE_WIDE_FROM", "48"))     # places an expert on average from which tiles are wide
@@ -2003,21 +2023,29 @@ def moe_tile_rows(pairs: int, experts: int, a: torch.Tensor, widths) -> int:
 
 
 def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, scale: float, ids: torch.Tensor,
-              weights: torch.Tensor) -> None:
-    """Per row of float32 router logits [tokens, experts]: softmax over all experts, the `keep` best of `groups` equal
-    groups of neighbouring experts (a group's score: its largest), the `top` best experts of those groups (ids int32
-    [tokens, top]) and their scores over their sum, times `scale` (weights float32 [tokens, top])."""
-    _cuda(logits, ids, weights)
+              weights: torch.Tensor, correction: Optional[torch.Tensor] = None, scores: str = "softmax",
+              group_score: str = "max", renormalize: bool = True) -> None:
+    """Per row of float32 router logits [tokens, experts]: scores = softmax over all experts (or the sigmoid of each), choice
+    scores = scores + correction (float32 [experts], or None), the `keep` best of `groups` equal groups of neighbouring
+    experts (a group's score: its largest choice score, or with group_score "top2" the sum of its two largest), the `top`
+    experts of those groups with the largest choice scores (ids int32 [tokens, top]) and their scores, over their sum
+    (renormalize) or as they are, times `scale` (weights float32 [tokens, top])."""
+    _cuda(logits, ids, weights, correction)
     _rows_contiguous(logits, "logits")
     tokens, experts = logits.shape
     if logits.dtype != torch.float32 or ids.dtype != torch.int32 or weights.dtype != torch.float32 \
             or not ids.is_contiguous() or not weights.is_contiguous() or ids.numel() < tokens * top or weights.numel() < tokens * top:
         raise InvalidArgument("moe_route: logits float32, ids int32 [tokens, top], weights float32 [tokens, top]")
+    if scores not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
+        raise InvalidArgument(f"moe_route: no scores '{scores}' (softmax, sigmoid) or group score '{group_score}' (max, top2)")
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts):
+        raise InvalidArgument("moe_route: correction float32 [experts]")
     if experts > MOE_MAX_EXPERTS or top > experts or groups <= 0 or experts % groups or not 0 < keep <= groups \
             or top > keep * (experts // groups):
         raise Unsupported(f"moe_route: {experts} experts in {groups} groups, {keep} kept, {top} a token")
-    _check(_fn("moe", "dl_moe_route")(_p(logits), logits.stride(0), tokens, experts, top, groups, keep, scale, _p(ids),
-                                      _p(weights), _stream()), "moe_route")
+    _check(_fn("moe", "dl_moe_route")(_p(logits), logits.stride(0), tokens, experts, top, groups, keep, _p(correction),
+                                      1 if scores == "sigmoid" else 0, 1 if group_score == "top2" else 0,
+                                      1 if renormalize else 0, scale, _p(ids), _p(weights), _stream()), "moe_route")
 
 
 def moe_group(ids: torch.Tensor, pairs: int, experts: int, place_of: torch.Tensor, pair_at: torch.Tensor,
@@ -2040,27 +2068,39 @@ def moe_linear(a: torch.Tensor, pair_at: Optional[torch.Tensor], top_div: int, w
                tile_rows: int = MOE_TILE_ROWS) -> None:
     """c[place] = act(a[row of place] w[expert of place]^T) for every place of every tile: w [experts, N, K], a rows of K
     numbers (the row of a place is pair_at[place] // top_div, or the place itself when pair_at is None), c [places, N]
-    of a's dtype or float32. act: "none" or "relu2"."""
+    of a's dtype or float32. act: "none", "relu2", or "pairs": rows 2j and 2j + 1 of a matrix are the gate and up rows of
+    feature j and c [places, N / 2] = silu(gate) * up."""
     _cuda(a, pair_at, w, c, tiles, n_tiles)
     _rows_contiguous(a, "a")
     _rows_contiguous(c, "c")
-    if w.dim() != 3 or not w.is_contiguous() or w.dtype != a.dtype or a.shape[1] != w.shape[2] or c.shape[1] != w.shape[1] \
-            or c.dtype not in (a.dtype, torch.float32) or act not in ("none", "relu2"):
+    if w.dim() != 3 or not w.is_contiguous() or w.dtype != a.dtype or a.shape[1] != w.shape[2] or c.shape[1] != w.shape[1] // (2 if act == "pairs" else 1) \
+            or c.dtype not in (a.dtype, torch.float32) or act not in MOE_ACTS or (act == "pairs" and w.shape[1] % 2):
         raise InvalidArgument("moe_linear: w [experts, N, K] of a's dtype, a [rows, K], c [places, N] of a's dtype or float32")
     _check(_fn("moe", "dl_moe_linear")(dtype_code(a.dtype), dtype_code(c.dtype), _p(a), a.stride(0), _p(pair_at), top_div,
                                        _p(w), w.shape[1], w.shape[2], _p(c), c.stride(0), _p(tiles), _p(n_tiles), max_tiles,
-                                       1 if act == "relu2" else 0, 1 if MOE_TENSOR_CORES else 0, tile_rows, _stream()),
+                                       MOE_ACTS[act], 1 if MOE_TENSOR_CORES else 0, tile_rows, _stream()),
            "moe_linear")
 
 
-def moe_combine(c: torch.Tensor, place_of: torch.Tensor, weights: torch.Tensor, top: int, y: torch.Tensor) -> None:
-    """y[t] = sum_k weights[t, k] * c[place_of[t * top + k]] in float32, in the order of k. c: float32 [places, width]."""
-    _cuda(c, place_of, weights, y)
+def moe_combine(c: torch.Tensor, place_of: torch.Tensor, weights: torch.Tensor, top: int, y: torch.Tensor,
+                shared: Optional[torch.Tensor] = None, shared_z: Optional[torch.Tensor] = None) -> None:
+    """y[t] = sum_k weights[t, k] * c[place_of[t * top + k]] in float32, in the order of k; with a shared expert's output
+    (`shared`, [tokens, width] or partial sums [parts, tokens, width]) and its gate's logits (`shared_z`, float32, one column
+    of a 2-D tensor) + sigmoid(shared_z[t]) * shared[t]. c: float32 [places, width]."""
+    _cuda(c, place_of, weights, y, shared, shared_z)
     tokens, width = y.shape
     if c.dtype != torch.float32 or not c.is_contiguous() or c.shape[1] != width or not y.is_contiguous() \
             or place_of.dtype != torch.int32 or weights.dtype != torch.float32:
         raise InvalidArgument("moe_combine: c float32 [places, width], y contiguous [tokens, width]")
-    _check(_fn("moe", "dl_moe_combine")(dtype_code(y.dtype), _p(c), width, _p(place_of), _p(weights), top, _p(y), tokens,
+    parts, part_stride = 1, 0
+    if shared is not None:
+        parts, part_stride = _delta_parts(shared, width, "moe_combine")
+        if shared_z is None or shared_z.dtype != torch.float32 or shared_z.dim() != 2 or shared_z.shape[0] < tokens \
+                or shared.shape[-2] < tokens:
+            raise InvalidArgument("moe_combine: the shared expert's output goes with its gate's logits, float32 [tokens, 1]")
+    _check(_fn("moe", "dl_moe_combine")(dtype_code(y.dtype), _p(c), width, _p(place_of), _p(weights), top,
+                                        dtype_code(shared.dtype) if shared is not None else 0, _p(shared), parts, part_stride,
+                                        _p(shared_z), shared_z.stride(0) if shared_z is not None else 0, _p(y), tokens,
                                         _stream()), "moe_combine")
 
 
@@ -2082,14 +2122,23 @@ def masked_flash_attention(q: torch.Tensor, k_cache: torch.Tensor, k_row: int, v
                            block_table: torch.Tensor, q_tiles: torch.Tensor, n_tiles: int, out: torch.Tensor, n_heads: int,
                            n_kv_heads: int, key_dim: int, value_dim: int, page_size: int, scale: float, window: int = 0,
                            keep_first: int = 0, sink: bool = False, one_token_tiles: bool = False, parts: int = 1,
-                           partial: Optional[torch.Tensor] = None) -> None:
+                           partial: Optional[torch.Tensor] = None, rate: Optional[torch.Tensor] = None,
+                           step: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
     """Flash attention of query tiles over the paged cache, bfloat16, with keys of key_dim and values of value_dim
     numbers (a pair of MASKED_FLASH_SIZES), kept first tokens behind the window and an optional extra term exp(0) in the
     denominator; see csrc/attention_masked_flash.cu. q_tiles: int32 [n_tiles, 4] = (request, first row, rows <= 128,
     first position). k_cache / v_cache point at the first token's keys / values, k_row / v_row elements between tokens.
     one_token_tiles: every tile is a single token, tile i being row i of q (a decode step); the heads that share a KV head
     then share a block, and with parts > 1 a row's key tiles are dealt over that many blocks whose results a second
-    kernel merges (partial: float32 scratch of masked_flash_partial_floats elements)."""
+    kernel merges (partial: float32 scratch of masked_flash_partial_floats elements). rate, step (float32 [n_heads], both or
+    neither): rate_h ln(1 + step_h * distance) comes off every score. gate (bfloat16, head h at column h * value_dim): the
+    output is multiplied by its sigmoid."""
+    _cuda(rate, step, gate)
+    _distance_bias(rate, step, n_heads)
+    if gate is not None:
+        _rows_contiguous(gate, "gate")
+        if gate.dtype != torch.bfloat16 or gate.shape[0] < out.shape[0] or gate.shape[1] < n_heads * value_dim:
+            raise InvalidArgument("masked flash attention: the gate is bfloat16 [rows, heads * value_dim]")
     _cuda(q, k_cache, v_cache, block_table, q_tiles, out)
     _rows_contiguous(q, "q")
     _rows_contiguous(out, "out")
@@ -2111,8 +2160,8 @@ def masked_flash_attention(q: torch.Tensor, k_cache: torch.Tensor, k_row: int, v
     _check(_fn("attention_masked_flash", "dl_masked_flash_attention")(
         _p(q), q.stride(0), _p(k_cache), k_row, _p(v_cache), v_row, _p(block_table), block_table.stride(0), _p(q_tiles),
         n_tiles, _p(out), out.stride(0), n_heads, n_kv_heads, key_dim, value_dim, page_size, scale, window, int(keep_first),
-        1 if sink else 0, 1 if one_token_tiles else 0, int(parts), _p(partial) if parts > 1 else None, _stream()),
-        "masked_flash_attention")
+        1 if sink else 0, 1 if one_token_tiles else 0, int(parts), _p(partial) if parts > 1 else None,
+        _p(rate), _p(step), _p(gate), gate.stride(0) if gate is not None else 0, _stream()), "masked_flash_attention")
 
 
 MASKED_FLASH_MAX_PARTS = 8
@@ -2148,9 +2197,11 @@ def moe_gather(a: torch.Tensor, pair_at: torch.Tensor, top_div: int, out: torch.
     _check(_fn("moe", "dl_moe_gather")(_p(a), a.stride(0), _p(pair_at), top_div, _p(out), pairs, K, _stream()), "moe_gather")
 
 
-def moe_linear_tcgen05_applies(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor) -> bool:
+def moe_linear_tcgen05_applies(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, act: str = "none") -> bool:
     """Whether the grouped tcgen05 product takes these operands (bfloat16, aligned rows, an output it can store)."""
     n = w.shape[1]
+    if act == "pairs" and (n % 16 or c.dtype != torch.bfloat16):
+        return False
     return (MOE_TCGEN05 and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and a.shape[1] % 8 == 0
             and a.stride(0) % 8 == 0 and a.stride(1) == 1 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
             and c.data_ptr() % 16 == 0 and c.stride(1) == 1
@@ -2161,13 +2212,148 @@ def moe_linear_tcgen05(a: torch.Tensor, w: torch.Tensor, c: torch.Tensor, tiles:
                        max_tiles: int, act: str = "none") -> None:
     """c[place] = act(a[place] w[expert of place]^T) on the tcgen05 tensor cores: a [places, K] bfloat16 IN PLACE ORDER
     (moe_gather), w [experts, N, K], c [places, N] bfloat16 or float32 (act "none" only), tiles of at most 128 places as
-    moe_group lists them with tile_rows = 128. See csrc/gemm_tcgen05.cu (dl_gemm_tcgen05_grouped)."""
+    moe_group lists them with tile_rows = 128; with act "pairs" c [places, N / 2] bfloat16 (see moe_linear). See
+    csrc/gemm_tcgen05.cu (dl_gemm_tcgen05_grouped)."""
     _cuda(a, w, c, tiles, n_tiles)
-    if not moe_linear_tcgen05_applies(a, w, c) or w.dim() != 3 or a.shape[1] != w.shape[2] or c.shape != (a.shape[0], w.shape[1]) \
-            or act not in ("none", "relu2") or (act == "relu2" and c.dtype != torch.bfloat16):
+    if not moe_linear_tcgen05_applies(a, w, c, act) or w.dim() != 3 or a.shape[1] != w.shape[2] \
+            or c.shape != (a.shape[0], w.shape[1] // (2 if act == "pairs" else 1)) \
+            or act not in MOE_ACTS or (act != "none" and c.dtype != torch.bfloat16):
         raise Unsupported("moe_linear_tcgen05: bfloat16 operands with 16-byte aligned rows; relu2 with a bfloat16 result")
-    mode = 4 if act == "relu2" else (0 if c.dtype == torch.bfloat16 else 1)
+    mode = {"relu2": 4, "pairs": 6}.get(act, 0 if c.dtype == torch.bfloat16 else 1)
     status = _status_word(a.device)
     _check(_fn("gemm_tcgen05", "dl_gemm_tcgen05_grouped")(
         _p(a), a.stride(0), a.shape[0], _p(w), w.shape[0], w.shape[1], w.shape[2], _p(c), c.stride(0), mode, _p(tiles),
         _p(n_tiles), max_tiles, _p(status), _stream()), "moe_linear_tcgen05")
+
+
+# ---------------------------------------------------------------------------------------------
+# a token table of pairs, a fused residual update and norm, short convolutions into the cache, xIELU, a token's gate
+
+def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor, row_request: torch.Tensor,
+                row_slot: torch.Tensor, q_start: torch.Tensor, state: torch.Tensor, out: torch.Tensor, scale: float,
+                mul_prev: int, mul_cur: int) -> None:
+    """out[i] = table[ids[i]] * scale + pairs[r], r = (mul_prev * previous token + mul_cur * ids[i]) mod (rows of pairs - 1),
+    the last row of pairs for a sequence's first token. state: int32 [slots, 1], every request's last token, read and
+    brought up to date. See csrc/embedding.cu."""
+    _cuda(table, pairs, ids, positions, row_request, row_slot, q_start, state, out)
+    rows, width = out.shape
+    if out.dtype != torch.float32 or not out.is_contiguous() or ids.dtype != torch.int32 or state.dtype != torch.int32 \
+            or not table.is_contiguous() or not pairs.is_contiguous() or pairs.dtype != table.dtype:
+        raise InvalidArgument("embed_pairs: out float32 contiguous, ids and state int32, two contiguous tables of one dtype")
+    if table.shape[1] != width or pairs.shape[1] != width or pairs.shape[0] < 2 or ids.numel() < rows or state.dim() != 2:
+        raise InvalidArgument("embed_pairs: shapes disagree")
+    check_limits("embedding", requests=state.shape[0], rows=rows, vocab=table.shape[0])
+    _check(_fn("embedding", "dl_embed_pairs")(dtype_code(table.dtype), _p(table), _p(pairs), _p(ids), _p(positions),
+                                              _p(row_request), _p(row_slot), _p(q_start), _p(state), state.stride(0), _p(out),
+                                              rows, width, table.shape[0], scale, pairs.shape[0] - 1, int(mul_prev),
+                                              int(mul_cur), _stream()), "embed_pairs")
+
+
+def residual_norm(x: torch.Tensor, out: Optional[torch.Tensor], norm: str = "none", weight: Optional[torch.Tensor] = None,
+                  bias: Optional[torch.Tensor] = None, eps: float = 0.0, delta: Optional[torch.Tensor] = None,
+                  delta_scale: float = 1.0, gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None,
+                  post_weight: Optional[torch.Tensor] = None, post_eps: float = 0.0, copy: Optional[torch.Tensor] = None,
+                  rows: Optional[torch.Tensor] = None) -> None:
+    """x (float32 [n, width]) <- x + y, y = delta_scale * delta (of either dtype, or partial sums [parts, n, width]), times
+    sigmoid(gate + gate_bias) when a gate is given (rows of one dtype, any pitch), made unit-RMS times post_weight when that
+    is given; then copy = x and out = norm(x) ("layer": weight, bias; "rms": weight; "none": out None). With `rows` only
+    those rows are normed and x stays as it is. See csrc/residual_norm.cu."""
+    _cuda(x, out, weight, bias, delta, gate, gate_bias, post_weight, copy, rows)
+    width = x.shape[-1]
+    if x.dtype != torch.float32 or not x.is_contiguous() or norm not in ("none", "layer", "rms"):
+        raise InvalidArgument("residual_norm: x float32 contiguous; norm none, layer or rms")
+    for t in (weight, bias, gate_bias, post_weight):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous()):
+            raise InvalidArgument("residual_norm: weights and biases are float32 [width]")
+    if norm != "none" and (out is None or weight is None):
+        raise InvalidArgument("residual_norm: a norm needs its weight and a result")
+    made = [t for t in (out, copy) if t is not None]
+    if any(t.shape[-1] != width or not t.is_contiguous() or t.dtype != made[0].dtype for t in made):
+        raise InvalidArgument("residual_norm: out and copy contiguous [rows, width] of one dtype")
+    n_out = made[0].shape[0] if made else x.shape[0]
+    if any(t.shape[0] != n_out for t in made) or (rows is None and n_out > x.shape[0]) \
+            or (rows is not None and (rows.dtype != torch.int32 or rows.numel() < n_out)):
+        raise InvalidArgument("residual_norm: row counts disagree")
+    parts, part_stride = _delta_parts(delta, width, "residual_norm")
+    if delta is not None and rows is None and delta.shape[-2] < n_out:
+        raise InvalidArgument("residual_norm: delta has fewer rows than x")
+    if gate is not None:
+        _rows_contiguous(gate, "gate")
+        if delta is None or gate.shape[1] < width or (rows is None and gate.shape[0] < n_out):
+            raise InvalidArgument("residual_norm: the gate goes with a delta of its size")
+    out_code = dtype_code(made[0].dtype) if made else (1 if (delta is not None and delta.dtype == torch.bfloat16)
+                                                       or (gate is not None and gate.dtype == torch.bfloat16) else 0)
+    dd = dtype_code(delta.dtype) if delta is not None else 0
+    gd = dtype_code(gate.dtype) if gate is not None else 0
+    check_limits("residual_norm", rows=x.shape[0])
+    ahead, ahead_bytes = _take_ahead()
+    _check(_fn("residual_norm", "dl_residual_norm")(
+        out_code, dd, gd, _p(x), width, _p(delta), parts, part_stride, delta_scale, _p(gate),
+        gate.stride(0) if gate is not None else 0, _p(gate_bias), _p(post_weight), post_eps, _p(copy),
+        {"none": 0, "layer": 1, "rms": 2}[norm], _p(weight), _p(bias), eps, _p(out), _p(rows), n_out, x.shape[0], ahead,
+        ahead_bytes, _stream()), "residual_norm")
+
+
+def conv_cache(proj: torch.Tensor, widths, taps_t: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+               kept: Optional[torch.Tensor], ctx, block_table: Optional[torch.Tensor], page_size: int, q_out: torch.Tensor,
+               k_cache: Optional[torch.Tensor] = None, k_row: int = 0, v_cache: Optional[torch.Tensor] = None,
+               v_row: int = 0) -> None:
+    """Short causal convolutions (taps_t: float32 [K, channels], the last tap the current token's; None: none) of the columns
+    q | k | v of `proj` (their widths in `widths`; no k and v: (n, 0, 0)), every input of the sequence plus `bias` (float32
+    [channels] or None): q into q_out, k and v into the token's place in the cache (k_cache / v_cache point at the first
+    token's keys / values, k_row / v_row elements lie between two tokens). kept: float32 [slots, >= (K - 1) * channels], the
+    requests' last inputs, read and brought up to date. See csrc/conv_cache.cu."""
+    _cuda(proj, taps_t, bias, kept, q_out, k_cache, v_cache, block_table)
+    _rows_contiguous(proj, "proj")
+    _rows_contiguous(q_out, "q_out")
+    cq, ck, cv = (int(w) for w in widths)
+    channels, rows = cq + ck + cv, proj.shape[0]
+    K = taps_t.shape[0] if taps_t is not None else 0
+    if taps_t is not None and (taps_t.dtype != torch.float32 or not taps_t.is_contiguous() or taps_t.dim() != 2 or taps_t.shape[1] != channels):
+        raise InvalidArgument("conv_cache: taps float32 [K, channels]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != channels or not bias.is_contiguous()):
+        raise InvalidArgument("conv_cache: bias float32 [channels]")
+    if K > 1:
+        if kept is None:
+            raise InvalidArgument("conv_cache: more than one tap needs kept inputs")
+        _state_rows(kept, (K - 1) * channels, "conv_cache")
+    if proj.shape[1] < channels or q_out.dtype != proj.dtype or q_out.shape[0] < rows or q_out.shape[1] < cq:
+        raise InvalidArgument("conv_cache: the columns lie inside proj; q_out of its dtype and rows")
+    if ck and (k_cache is None or v_cache is None or block_table is None or k_cache.dtype != proj.dtype or v_cache.dtype != proj.dtype):
+        raise InvalidArgument("conv_cache: keys and values need a cache of proj's dtype")
+    check_limits("conv_cache", pages=k_cache.shape[0] if ck else 0,
+                 requests=block_table.shape[0] if block_table is not None else (kept.shape[0] if kept is not None else 0), rows=rows)
+    kept_stride = kept.stride(0) if kept is not None else 0
+    _check(_fn("conv_cache", "dl_conv_cache")(
+        dtype_code(proj.dtype), _p(proj), proj.stride(0), cq, ck, cv, K, _p(taps_t), _p(bias), _p(kept), kept_stride,
+        _p(ctx.positions), _p(ctx.row_request), _p(ctx.row_slot), _p(ctx.q_start), _p(block_table),
+        block_table.stride(0) if block_table is not None else 0, page_size, _p(q_out), q_out.stride(0), _p(k_cache), k_row,
+        _p(v_cache), v_row, rows, _stream()), "conv_cache")
+    if K > 1 and not ctx.decode_only:                 # (a request's single token has moved its kept inputs already)
+        _check(_fn("conv_cache", "dl_conv_keep_many")(
+            dtype_code(proj.dtype), _p(proj), proj.stride(0), channels, K, _p(kept), kept_stride, _p(ctx.q_start),
+            _p(ctx.state_slots), ctx.num_requests, _stream()), "conv_keep_many")
+
+
+def xielu(x: torch.Tensor, out: torch.Tensor, coeffs: torch.Tensor) -> None:
+    """out = c0 x^2 + x / 2 above zero, c1 (e^x - 1 - x) + x / 2 at and below it; coeffs: float32 [2] = (c0, c1) on the
+    device. x and out contiguous, of one dtype (out may be x)."""
+    _cuda(x, out, coeffs)
+    if x.dtype != out.dtype or x.shape != out.shape or not x.is_contiguous() or not out.is_contiguous() \
+            or coeffs.dtype != torch.float32 or coeffs.numel() != 2:
+        raise InvalidArgument("xielu: x and out contiguous of one shape and dtype, coeffs float32 [2]")
+    _check(_fn("activation", "dl_xielu")(dtype_code(x.dtype), _p(x), _p(out), _p(coeffs), x.numel(), _stream()), "xielu")
+
+
+def token_gate(z: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t, j] = gelu_tanh(z[t, j]) * table[ids[t], j]; z and out contiguous [rows, n] (out may be z), table: [vocab, n],
+    any row pitch, of z's dtype."""
+    _cuda(z, table, ids, out)
+    _rows_contiguous(table, "table")
+    rows, n = z.shape
+    if z.dtype != out.dtype or table.dtype != z.dtype or out.shape != z.shape or not z.is_contiguous() or not out.is_contiguous() \
+            or table.shape[1] != n or ids.dtype != torch.int32 or ids.numel() < rows:
+        raise InvalidArgument("token_gate: z and out contiguous [rows, n], table [vocab, n], one dtype; ids int32")
+    check_limits("gates", rows=rows, vocab=table.shape[0])
+    _check(_fn("gates", "dl_token_gate")(dtype_code(z.dtype), _p(z), _p(table), table.stride(0), _p(ids), _p(out), rows, n,
+                                         table.shape[0], _stream()), "token_gate")

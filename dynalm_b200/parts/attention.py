@@ -169,10 +169,18 @@ class GatedNormedAttention(PagedAttention):
     keep_first  with a window: keys at positions below it stay visible behind the window, at their true positions.
     position    "rotary" (pairs i, i + rotary_dim / 2) or, with qk_norm "head" or "none", "rotary_interleaved" (pairs 2i,
                 2i + 1).
+    conv        K > 0: short causal convolutions of K taps over the channels of q, k and v, directly behind the projections
+                (tensors q_conv, k_conv, v_conv [channels, K]); a request keeps the last K - 1 projected values as a float32
+                state row beside its pages.
+    distance_bias  "log": rate_h ln(1 + step_h * distance) comes off every score (tensors distance_rate, distance_step);
+                "none".
+    own_kv      False: the layer makes queries only and reads the keys and values another run of the order has cached.
+    cache_window  the widest window of all runs that read this layer's cache (0: all earlier keys); default `window`.
     Biases of the four projections are taken when the model has them (q_bias, k_bias, v_bias, o_bias).
 
-    Parameters: num_heads, num_kv_heads, head_dim, value_dim, scale, window, keep_first, eps, qk_norm, gated, sink,
-    position. Tensors: q, k, v, o, and by the parameters q_norm, k_norm, gate.
+    Parameters: num_heads, num_kv_heads, head_dim, value_dim, scale, window, cache_window, keep_first, eps, qk_norm, gated,
+    sink, conv, distance_bias, own_kv, position. Tensors: q, k, v, o, and by the parameters q_norm, k_norm, gate, q_conv,
+    k_conv, v_conv, distance_rate, distance_step.
 
     Where keys and values have one size the cache is the plain attention's (two arrays) and so are the kernels that
     read it, as far as they know the mask and the softmax asked for; otherwise a token's keys and values form one record
@@ -186,8 +194,17 @@ class GatedNormedAttention(PagedAttention):
         qw, kw, vw = spec.num_heads * spec.head_dim, spec.num_kv_heads * spec.head_dim, spec.num_kv_heads * spec.value_dim
         ow = spec.num_heads * spec.value_dim
         normed, gated = spec.get("qk_norm", "none") == "projection", bool(spec.get("gated", False))
+        more = {}
+        if spec.get("own_kv", True):
+            more.update({"k": TensorDecl((kw, spec.width)), "v": TensorDecl((vw, spec.width))})
+        if spec.get("conv", 0) > 0:
+            for name, n in (("q", qw), ("k", kw), ("v", vw)):
+                if name == "q" or spec.get("own_kv", True):
+                    more[name + "_conv"] = TensorDecl((n, spec.conv), role="vector", init="bias")
+        if spec.get("distance_bias", "none") == "log":
+            more.update({n: TensorDecl((spec.num_heads,), role="vector", init="around_one") for n in ("distance_rate", "distance_step")})
         return {
-            "q": TensorDecl((qw, spec.width)), "k": TensorDecl((kw, spec.width)), "v": TensorDecl((vw, spec.width)),
+            "q": TensorDecl((qw, spec.width)), **more,
             "o": TensorDecl((spec.width, ow)),
             "q_norm": TensorDecl((qw,), role="vector", required=normed, init="around_one"),
             "k_norm": TensorDecl((kw,), role="vector", required=normed, init="around_one"),
@@ -220,14 +237,33 @@ class GatedNormedAttention(PagedAttention):
         self.keep_first = int(spec.get("keep_first", 0)) if self.window > 0 else 0
         self.gated = bool(spec.get("gated", False))
         self.same = spec.head_dim == spec.value_dim          # keys and values of one size: the plain attention's cache
-        mats = [tensors["q"], tensors["k"], tensors["v"]] + ([tensors["gate"]] if self.gated else [])
+        self.own_kv = bool(spec.get("own_kv", True))
+        self.taps = int(spec.get("conv", 0))
+        # one product, [q | k | v | gate]; a layer that reads another's keys has [q | gate]
+        self.widths = (self.q_width, self.kv_width, self.v_width) if self.own_kv else (self.q_width, 0, 0)
+        self.channels = sum(self.widths)
+        names = ("q", "k", "v") if self.own_kv else ("q",)
+        mats = [tensors[n] for n in names] + ([tensors["gate"]] if self.gated else [])
         self.w_qkv = torch.cat(mats, dim=0).contiguous()
-        biases = [tensors.get("q_bias"), tensors.get("k_bias"), tensors.get("v_bias")]
+        self.joined_col = self.w_qkv.shape[0]
+        biases = [tensors.get(n + "_bias") for n in names]
         self.b_qkv = None
+        # by itself the kernel of the short convolutions also adds the biases and writes the cache; a layer without a
+        # rotation or norm that has an output gate or reads another's cache goes through it too
+        plain_q = not self.normed and not self.head_normed and spec.get("position") is None
+        self.conv_path = plain_q and (self.taps > 0 or self.gated or not self.own_kv)
+        if not self.conv_path and (self.taps > 0 or not self.own_kv):
+            raise Unsupported("gated_attention: convolutions and the cache of another run go without rotation and norm")
         if any(b is not None for b in biases):
-            widths = [self.q_width, self.kv_width, self.v_width] + ([self.o_width] if self.gated else [])
+            widths = [self.q_width, self.kv_width, self.v_width][:len(names)] + ([self.o_width] if self.gated and not self.conv_path else [])
             self.b_qkv = torch.cat([b if b is not None else torch.zeros(w, dtype=torch.float32, device=runtime.device)
                                     for b, w in zip(biases + [None], widths)]).contiguous()
+        self.taps_t = None
+        if self.taps > 0:
+            self.taps_t = torch.cat([tensors[n + "_conv"] for n in names], dim=0).t().contiguous()      # [K, channels]
+        if spec.get("distance_bias", "none") not in ("log", "none"):
+            raise Unsupported(f"gated_attention: no distance bias '{spec.distance_bias}' (log, none)")
+        self.rate, self.dstep = tensors.get("distance_rate"), tensors.get("distance_step")
         self.q_norm, self.k_norm = (tensors["q_norm"], tensors["k_norm"]) if self.normed else (None, None)
         self.w_o = tensors["o"]
         self.b_o = tensors.get("o_bias")
@@ -239,8 +275,18 @@ class GatedNormedAttention(PagedAttention):
             raise Unsupported("gated_attention: the rotation runs inside its kernel and takes a position encoding with a table")
         if self.interleaved and self.normed:
             raise Unsupported("gated_attention: the interleaved rotation goes with the norm per head or with none")
-        # the kernels of the plain attention's cache know a window and an ordinary softmax
-        self.plain_mask = not self.sink and self.keep_first == 0
+        # the kernels of the plain attention's cache know a window and an ordinary softmax over scaled scores
+        self.plain_mask = not self.sink and self.keep_first == 0 and self.rate is None
+
+    def join_input(self, w: torch.Tensor) -> bool:
+        """Takes the rows of another product over the same input into this part's first one; `joined` gives its result."""
+        if not self.conv_path:
+            return False                                     # (the other paths read the projection by its width)
+        self.w_qkv = torch.cat([self.w_qkv, w], dim=0).contiguous()
+        return True
+
+    def joined(self, rows: int) -> torch.Tensor:
+        return self.rt.buffer("gattn_proj", (rows, self.w_qkv.shape[0]))[:, self.joined_col:]
 
     def step_plans(self) -> list:
         if self.same and self.plain_mask:
@@ -267,10 +313,20 @@ class GatedNormedAttention(PagedAttention):
 
     def cache_spec(self) -> Optional[CacheSpec]:
         s = self.spec
-        window = self.window if self.keep_first == 0 else 0      # kept first tokens: no page is given back
+        window = int(s.get("cache_window", self.window)) if self.keep_first == 0 else 0      # kept first tokens: no page is given back
+        state = self._kept_shape()
         if self.same:
-            return CacheSpec(kind="pages", entry_shape=(s.num_kv_heads, s.head_dim), tensors=2, window=window)
-        return CacheSpec(kind="pages", entry_shape=(self.kv_width + self.v_width,), tensors=1, window=window)
+            return CacheSpec(kind="pages", entry_shape=(s.num_kv_heads, s.head_dim), tensors=2, window=window, state_shape=state)
+        return CacheSpec(kind="pages", entry_shape=(self.kv_width + self.v_width,), tensors=1, window=window, state_shape=state)
+
+    def _kept_shape(self):
+        """The state row beside the pages: the last inputs of the convolutions."""
+        return ((self.taps - 1) * self.channels,) if self.taps > 1 else ()
+
+    def reader_state_spec(self) -> Optional[CacheSpec]:
+        """What a run that reads another's pages keeps by itself."""
+        shape = self._kept_shape()
+        return CacheSpec(kind="state", state_shape=shape, dtype="float32") if shape else None
 
     def _kv(self, cache):
         """(keys of the first token, elements between tokens, values of the first token, elements between tokens)."""
@@ -283,9 +339,11 @@ class GatedNormedAttention(PagedAttention):
 
     def forward(self, x: torch.Tensor, ctx, cache, owns_cache: bool = True) -> torch.Tensor:
         s, rt = self.spec, self.rt
-        if not owns_cache:
-            raise Unsupported("gated_attention: every run of the layer keeps a cache of its own")
+        if owns_cache != self.own_kv:
+            raise Unsupported("gated_attention: a run keeps a cache of its own exactly when its layer makes keys and values")
         rows = x.shape[0]
+        if self.conv_path:
+            return self._forward_conv(x, ctx, cache)
         proj = rt.buffer("gattn_proj", (rows, self.w_qkv.shape[0]))
         by_projection = self.normed or (not self.head_normed and not self.interleaved)
         # a bias joins in the kernel that turns and norms, where that kernel takes one; else in the product (the plain one)
@@ -314,6 +372,10 @@ class GatedNormedAttention(PagedAttention):
         self.attend(proj, cache, ctx, attn)
         if self.gated:
             ops.sigmoid_gate(attn, proj[:, self.q_width + self.kv_width + self.v_width:])
+        return self._project(attn)
+
+    def _project(self, attn: torch.Tensor) -> torch.Tensor:
+        s, rt, rows = self.spec, self.rt, attn.shape[0]
         if self.b_o is None:
             return linear_partial(attn, self.w_o, rt, self.out_name)
         if attn.dtype == torch.float32:
@@ -331,6 +393,26 @@ class GatedNormedAttention(PagedAttention):
         ops.add_bias(out, self.b_o)
         return out
 
+    def _forward_conv(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
+        """One product, one kernel that convolves, adds biases and writes the cache, attention with the output gate."""
+        s, rt = self.spec, self.rt
+        rows = x.shape[0]
+        proj = rt.buffer("gattn_proj", (rows, self.w_qkv.shape[0]))
+        linear(x, self.w_qkv, proj)
+        q = rt.buffer("gattn_q", (rows, self.q_width))
+        kept = cache.state.arrays[0] if cache.state is not None else None
+        k_cache = v_cache = None
+        k_row = v_row = 0
+        if self.own_kv:
+            k_cache, k_row, v_cache, v_row = self._kv(cache)
+        ops.conv_cache(proj, self.widths, self.taps_t, self.b_qkv, kept, ctx, cache.block_table, cache.page_size, q,
+                       k_cache, k_row, v_cache, v_row)
+        attn = rt.buffer("gattn_out", (rows, self.o_width))
+        gate = proj[:, self.channels:self.channels + self.o_width] if self.gated else None
+        if self.attend(q, cache, ctx, attn, gate) is not True and gate is not None:
+            ops.sigmoid_gate(attn, gate)
+        return self._project(attn)
+
     def _flash_applies(self, qkv: torch.Tensor, cache, ctx) -> bool:
         """bfloat16, sizes the masked flash kernel has, a step built with the query tiles, aligned rows."""
         from ..kernels import attention as fast
@@ -339,7 +421,8 @@ class GatedNormedAttention(PagedAttention):
                 and fast.query_tiles(ctx) is not None and cache.page_size & (cache.page_size - 1) == 0
                 and qkv.stride(0) % 8 == 0 and self.kv_width % 8 == 0 and self.v_width % 8 == 0)
 
-    def attend(self, qkv: torch.Tensor, cache, ctx, out: torch.Tensor) -> None:
+    def attend(self, qkv: torch.Tensor, cache, ctx, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> bool:
+        """True when the output gate has been applied on the way out."""
         s = self.spec
         if not (self.same and self.plain_mask) and self._flash_applies(qkv, cache, ctx):
             from ..kernels import attention as fast
@@ -354,13 +437,15 @@ class GatedNormedAttention(PagedAttention):
             ops.masked_flash_attention(qkv, k_cache, k_row, v_cache, v_row, cache.block_table, q_tiles, n_tiles, out,
                                        s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, cache.page_size,
                                        float(s.scale), self.window, self.keep_first, self.sink,
-                                       one_token_tiles=ctx.decode_only, parts=parts, partial=partial)
-            return
+                                       one_token_tiles=ctx.decode_only, parts=parts, partial=partial, rate=self.rate, step=self.dstep,
+                                       gate=gate)
+            return gate is not None
         if self.same and self.plain_mask:
             from ..kernels import attention as fast
             if fast.paged_attention(qkv, cache, ctx, out, s, self.rt):
-                return
+                return False
         k_cache, k_row, v_cache, v_row = self._kv(cache)
         ops.paged_attention_generic_kv(qkv, k_cache, k_row, v_cache, v_row, cache.block_table, ctx.positions, ctx.row_slot,
                                        out, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, cache.page_size,
-                                       float(s.scale), self.window, self.keep_first, self.sink)
+                                       float(s.scale), self.window, self.keep_first, self.sink, rate=self.rate, step=self.dstep)
+        return False

@@ -62,7 +62,7 @@ class CacheSpec:
     tensors: int = 2
     window: int = 0
     state_shape: Tuple[int, ...] = ()
-    dtype: Optional[str] = None      # None = the compute dtype; else "float32" / "bfloat16"
+    dtype: Optional[str] = None      # None = the compute dtype; else "float32" / "bfloat16" (kind "state" also "int32")
     state_dtype: Optional[str] = None      # of the state row beside pages; None = float32
 
     def group_key(self) -> tuple:

@@ -6,6 +6,8 @@ parts fed from the same x. The residual stream is float32; the sum of a part's o
 fused into the norm that follows, so a block leaves its last output (the parallel one: both) pending.
 "post_norm": x <- norm1(a x + mixer(x)); x <- norm2(a x + ffn(x)): the sublayers read the stream itself and each
 norm closes its own sum, so nothing is left pending and the stream is always a normed row.
+"gated_pre_norm": x <- x + sigmoid(W h + b) * sublayer(h), h = norm(x), for mixer and feed-forward, and optionally a small
+input from the token at the layer's end.
 "hyper_connections": the stream has several parts; a sublayer reads a weighted sum of them and every part becomes a
 mix of all parts plus its own share of the sublayer's result.
 """
@@ -17,7 +19,7 @@ from typing import Optional
 
 import torch
 
-from ..kernels import ops
+from ..kernels import linear, ops
 from .base import TensorDecl, build_part, register_block, register_connection
 
 
@@ -36,8 +38,27 @@ class ResidualStream:
     streams: Optional[torch.Tensor] = None
     parts: int = 1
     link: Optional[object] = None
+    # How `pending` joins a stream of one part when not as it is: times sigmoid(gate + via.gate_bias) when `gate` (rows of
+    # any pitch) is set, made unit-RMS times via.post_weight when the part `via` has one.
+    gate: Optional[torch.Tensor] = None
+    via: Optional[object] = None
+
+    def update(self) -> dict:
+        """What is pending, as keyword arguments of ops.residual_norm."""
+        via = self.via
+        return dict(delta=self.pending, delta_scale=self.pending_scale, gate=self.gate,
+                    gate_bias=via.gate_bias if via is not None and self.gate is not None else None,
+                    post_weight=via.post_weight if via is not None else None,
+                    post_eps=via.post_eps if via is not None else 0.0)
+
+    def leave(self, pending: Optional[torch.Tensor], gate: Optional[torch.Tensor] = None, via=None) -> None:
+        """A sublayer's result is pending, to join as `gate` and `via` say."""
+        self.pending, self.pending_scale, self.gate, self.via = pending, 1.0, gate, via
 
     def flush(self) -> torch.Tensor:
+        if self.via is not None:
+            ops.residual_norm(self.x, None, **self.update())
+            self.leave(None)
         if self.streams is not None:
             link = self.link if self.pending is not None else None
             ops.stream_sum(self.streams, self.parts, self.x, delta=self.pending, delta_scale=self.pending_scale,
@@ -52,7 +73,10 @@ class ResidualStream:
         return self.x
 
     def flush_second(self) -> None:
-        """Adds the second pending output now; for a consumer that takes one delta only."""
+        """Adds the second pending output now, and a pending output that does not join as it is; for a consumer that takes
+        one plain delta only."""
+        if self.via is not None:
+            self.flush()
         if self.pending2 is not None:
             ops.residual_add(self.x, self.pending2, 1.0)
             self.pending2 = None
@@ -83,6 +107,11 @@ class Block:
     def cache_spec(self):
         part = getattr(self, self.cache_part, None)
         return part.cache_spec() if part is not None and hasattr(part, "cache_spec") else None
+
+    def reader_state_spec(self):
+        """The state row of a run that reads another entry's pages (None: it keeps none)."""
+        part = getattr(self, self.cache_part, None)
+        return part.reader_state_spec() if part is not None and hasattr(part, "reader_state_spec") else None
 
     def step_plans(self) -> list:
         return [plan for p in self.parts() for plan in (p.step_plans() if hasattr(p, "step_plans") else [])]
@@ -145,7 +174,7 @@ class ParallelBlock(Block):
 
     def forward(self, stream: ResidualStream, ctx, cache, owns_cache: bool) -> ResidualStream:
         rows, width = stream.x.shape
-        if stream.pending is not None and stream.pending_scale != 1.0:
+        if stream.via is not None or (stream.pending is not None and stream.pending_scale != 1.0):
             stream.flush()
         h1 = self.rt.buffer("normed", (rows, width))
         h2 = self.rt.buffer("normed_ffn", (rows, width)) if self.has_ffn else None
@@ -220,6 +249,92 @@ class SandwichNormBlock(Block):
         else:
             ops.norm_add_norm(stream.x, a, post.weight, post.eps)
         stream.pending_scale = 1.0
+        stream.as_input = None
+        return stream
+
+
+@register_connection("sigmoid_gate")
+class SigmoidGate:
+    """The gate with which one sublayer's result joins the stream: sigmoid(weight h + bias), h the sublayer's input. A part
+    that has a product over h anyway takes the gate's rows into it (`join_input`), else the gate makes its own. Tensors:
+    weight [width, width], bias [width]."""
+
+    replay_safe = True     # all device work goes through the recorded launches of kernels/ops.py (engine/launch_memo.py)
+    graph_safe = True
+    post_weight, post_eps = None, 0.0
+
+    @staticmethod
+    def declare(spec):
+        return {"weight": TensorDecl((spec.width, spec.width)), "bias": TensorDecl((spec.width,), role="vector", init="bias")}
+
+    def __init__(self, spec, tensors, runtime):
+        self.spec = spec
+        self.rt = runtime
+        self.weight = tensors["weight"]
+        self.gate_bias = tensors["bias"].contiguous()
+
+    def ride(self, part) -> None:
+        """Called once, when the block is built: lets `part` make this gate's product with its own."""
+        join = getattr(part, "join_input", None)
+        if join is not None and join(self.weight):
+            self.weight = None
+
+    def values(self, part, h: torch.Tensor) -> torch.Tensor:
+        """weight h, without the bias; after `part` has run over h."""
+        if self.weight is None:
+            return part.joined(h.shape[0])
+        g = self.rt.buffer("stream_gate", (h.shape[0], self.spec.width))
+        return linear(h, self.weight, g)
+
+
+@register_block("gated_pre_norm")
+class GatedPreNormBlock(Block):
+    """parts: mixer_norm, mixer, mixer_gate, and optionally ffn_norm, ffn, ffn_gate, and side. x <- x + gate1(h) * mixer(h), h
+    = mixer_norm(x); x <- x + gate2(h) * ffn(h), h = ffn_norm(x); and with `side` (a part that reads the stream itself and
+    whose result joins normed) x <- x + norm(side(x)). The gate or norm of a result is applied, and the result added, by the
+    norm kernel that follows, in this layer or the next (ops.residual_norm); the norms are of a kind that does so
+    (`forward_update`)."""
+
+    def __init__(self, spec, store, runtime):
+        super().__init__(spec, store, runtime)
+        self.has_ffn, self.has_side = "ffn" in spec.parts, "side" in spec.parts
+        self.mixer_gate.ride(self.mixer)
+        if self.has_ffn:
+            self.ffn_gate.ride(self.ffn)
+
+    def last_via(self):
+        """The part through which the result this layer leaves pending joins the stream."""
+        return self.side if self.has_side else (self.ffn_gate if self.has_ffn else self.mixer_gate)
+
+    def entry_tensors(self, stream: ResidualStream) -> list:
+        """The tensors of the layer in front that this layer's first norm reads (engine/launch_memo.py)."""
+        via = stream.via
+        return [t for t in (via.gate_bias, via.post_weight) if t is not None] if via is not None else []
+
+    def forward(self, stream: ResidualStream, ctx, cache, owns_cache: bool) -> ResidualStream:
+        rows, width = stream.x.shape
+        if stream.streams is not None or stream.pending2 is not None:      # (another arrangement may stand in front)
+            stream.flush()
+        few = rows <= ops.SKINNY_FAST_ROWS         # a step bound by the stream of weights: say early what comes next
+        h = self.rt.buffer("normed", (rows, width))
+        if few:
+            ops.stream_ahead(getattr(self.mixer, "first_weights", lambda: None)())
+        self.mixer_norm.forward_update(stream, h)
+        a = self.mixer.forward(h, ctx, cache, owns_cache)
+        stream.leave(a, self.mixer_gate.values(self.mixer, h), self.mixer_gate)
+        if self.has_ffn:
+            if few:
+                ops.stream_ahead(getattr(self.ffn, "first_weights", lambda: None)())
+            self.ffn_norm.forward_update(stream, h)
+            f = self.ffn.forward(h, ctx)
+            stream.leave(f, self.ffn_gate.values(self.ffn, h), self.ffn_gate)
+        if self.has_side:
+            narrow = self.rt.dtype != torch.float32
+            x = self.rt.buffer("stream_copy", (rows, width)) if narrow else stream.x
+            if few:
+                ops.stream_ahead(self.side.w_gate)
+            ops.residual_norm(stream.x, None, copy=x if narrow else None, **stream.update())
+            stream.leave(self.side.forward(x, ctx), None, self.side)
         stream.as_input = None
         return stream
 

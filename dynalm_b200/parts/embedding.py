@@ -2,16 +2,19 @@
 
 from __future__ import annotations
 
-from typing import Dict
+from typing import Dict, Optional
 
 import torch
 
 from ..kernels import linear, ops
-from .base import TensorDecl
+from .base import CacheSpec, TensorDecl
 
 
 def declare_embedding(spec) -> Dict[str, TensorDecl]:
-    return {spec.tensors["weight"]: TensorDecl((spec.vocab, spec.width))}
+    out = {spec.tensors["weight"]: TensorDecl((spec.vocab, spec.width))}
+    if getattr(spec, "pair_rows", 0) > 0:
+        out[spec.tensors["pairs"]] = TensorDecl((spec.pair_rows + 1, spec.width))
+    return out
 
 
 def declare_head(spec) -> Dict[str, TensorDecl]:
@@ -20,17 +23,29 @@ def declare_head(spec) -> Dict[str, TensorDecl]:
 
 class TokenEmbedding:
     """x[i, :] = table[token_i, :] * scale into the float32 residual stream
-    (dynalm/src/model/transformer.cpp:576-577)."""
+    (dynalm/src/model/transformer.cpp:576-577), plus, when the spec has a table of token pairs, the row of it that this
+    token and the one in front of it choose (the last row for a sequence's first token). The last token of every request
+    is then part of its state: one int32 word per request slot, read and written by the embedding's own kernel, so that
+    it is right also where a step's tokens are chosen on the device."""
 
     def __init__(self, spec, store, runtime):
         self.spec = spec
         self.rt = runtime
         self.table = store[spec.tensors["weight"]]
+        self.pairs = store[spec.tensors["pairs"]] if getattr(spec, "pair_rows", 0) > 0 else None
         self.scale = float(spec.scale)
 
-    def forward(self, token_ids: torch.Tensor, rows: int) -> torch.Tensor:
+    def cache_spec(self) -> Optional[CacheSpec]:
+        return CacheSpec(kind="state", state_shape=(1,), dtype="int32") if self.pairs is not None else None
+
+    def forward(self, ctx, cache=None) -> torch.Tensor:
+        rows = ctx.num_tokens
         x = self.rt.buffer("residual", (rows, self.spec.width), torch.float32)
-        ops.embed(self.table, token_ids, x, self.scale)
+        if self.pairs is None:
+            ops.embed(self.table, ctx.token_ids, x, self.scale)
+        else:
+            ops.embed_pairs(self.table, self.pairs, ctx.token_ids, ctx.positions, ctx.row_request, ctx.row_slot, ctx.q_start,
+                            cache.arrays[0], x, self.scale, self.spec.pair_previous, self.spec.pair_current)
         return x
 
 

@@ -9,6 +9,8 @@ Per token the layer's input h gives a query latent and a key/value latent:
     p   = exp(s) / (sum over the window of exp(s) + exp(sink_h))   the sink has no key and no value
     out = o( concat_h(sum p v_h) * sigmoid(g h) )
 
+With q_rank 0 there is no query latent: q = q h (tensor "q" instead of dq, dq_norm and uq), one product with the rest.
+
 Only c and rot(k_rot) are cached, as one record per token, and the attention runs on the records themselves: since
 q_h . uk_h c = (uk_h^T q_h) . c, every head gets a "wide" query [uk_h^T q_h | rot(q_h[d:])] of R + r numbers that is
 scored against the records, the softmax weights sum the records' latents, and uv_h is applied to that sum. The two
@@ -40,10 +42,12 @@ class LatentAttention:
     @staticmethod
     def declare(spec) -> Dict[str, TensorDecl]:
         H, d, r, e = spec.num_heads, spec.head_dim, spec.rot_dim, spec.value_dim
-        return {
+        query = {"q": TensorDecl((H * (d + r), spec.width))} if spec.q_rank == 0 else {
             "dq": TensorDecl((spec.q_rank, spec.width)),
             "dq_norm": TensorDecl((spec.q_rank,), role="vector", init="around_one"),
-            "uq": TensorDecl((H * (d + r), spec.q_rank)),
+            "uq": TensorDecl((H * (d + r), spec.q_rank))}
+        return {
+            **query,
             "dkv": TensorDecl((spec.kv_rank + r, spec.width)),
             "dkv_norm": TensorDecl((spec.kv_rank,), role="vector", init="around_one"),
             "uk": TensorDecl((H * d, spec.kv_rank)),
@@ -60,11 +64,13 @@ class LatentAttention:
         self.spec = spec
         self.rt = runtime
         self.has_gate = "gate" in tensors
-        # one product for everything that reads the layer's input: [query latent | latent | key part | gate]
-        down = [tensors["dq"], tensors["dkv"]] + ([tensors["gate"]] if self.has_gate else [])
+        # one product for everything that reads the layer's input: [query latent or queries | latent | key part | gate]
+        self.q_cols = spec.q_rank or H * (d + r)
+        down = [tensors["dq"] if spec.q_rank else tensors["q"], tensors["dkv"]] + ([tensors["gate"]] if self.has_gate else [])
         self.w_down = torch.cat(down, dim=0).contiguous()
-        self.dq_norm, self.dkv_norm = tensors["dq_norm"], tensors["dkv_norm"]
-        self.w_uq = tensors["uq"]
+        self.dq_norm, self.dkv_norm = tensors.get("dq_norm"), tensors["dkv_norm"]
+        self.w_uq = tensors.get("uq")
+        self.joined_col = self.w_down.shape[0]
         self.w_uk = tensors["uk"].reshape(H, d, R).contiguous()                          # [H, in = d, out = R] as stored
         self.w_uv = tensors["uv"].reshape(H, e, R).transpose(1, 2).contiguous()          # [H, in = R, out = e]
         self.sink = tensors.get("sink")
@@ -76,6 +82,15 @@ class LatentAttention:
             raise Unsupported(f"latent_attention: position encoding '{pos.kind}' has no kernel here (rotary_interleaved has)")
         self.rot = self.position.rotary_dim if self.position is not None else 0
         self.freq = self.position.frequencies if self.position is not None else None
+        self.mag = self.position.magnitude if self.position is not None else 1.0
+
+    def join_input(self, w: torch.Tensor) -> bool:
+        """Takes the rows of another product over the same input into this part's first one; `joined` gives its result."""
+        self.w_down = torch.cat([self.w_down, w], dim=0).contiguous()
+        return True
+
+    def joined(self, rows: int) -> torch.Tensor:
+        return self.rt.buffer("latent_down", (rows, self.w_down.shape[0]))[:, self.joined_col:]
 
     def first_weights(self) -> torch.Tensor:
         return self.w_down
@@ -103,19 +118,24 @@ class LatentAttention:
         (records,) = cache.arrays
         down = rt.buffer("latent_down", (rows, self.w_down.shape[0]))
         linear(x, self.w_down, down)
-        cq = rt.buffer("latent_cq", (rows, s.q_rank))
-        ops.latent_prep(down, s.q_rank, R, r, self.rot, self.dq_norm, self.dkv_norm, self.eps, self.freq, ctx.positions,
-                        ctx.row_slot, cache.block_table, records, cache.page_size, cq)
-        q = rt.buffer("latent_q", (rows, H * (d + r)))
-        linear(cq, self.w_uq, q)
+        if s.q_rank:
+            cq = rt.buffer("latent_cq", (rows, s.q_rank))
+            ops.latent_prep(down, s.q_rank, R, r, self.rot, self.dq_norm, self.dkv_norm, self.eps, self.freq, ctx.positions,
+                            ctx.row_slot, cache.block_table, records, cache.page_size, cq, self.mag)
+            q = rt.buffer("latent_q", (rows, H * (d + r)))
+            linear(cq, self.w_uq, q)
+        else:
+            q = down[:, :self.q_cols]
+            ops.latent_prep(down[:, self.q_cols:], 0, R, r, self.rot, None, self.dkv_norm, self.eps, self.freq, ctx.positions,
+                            ctx.row_slot, cache.block_table, records, cache.page_size, None, self.mag)
         wide = rt.buffer("latent_wide_q", (rows, H * (R + r)))
         ops.head_linear(q, d + r, d, self.w_uk, wide, R + r)
         if r:
-            ops.rotate_pairs(q, d + r, d, wide, R + r, R, r, self.rot, self.freq, ctx.positions, H)
+            ops.rotate_pairs(q, d + r, d, wide, R + r, R, r, self.rot, self.freq, ctx.positions, H, self.mag)
         mixed = rt.buffer("latent_mixed", (rows, H * R))
         self.attend(wide, cache, ctx, mixed)
         heads = rt.buffer("latent_heads", (rows, H * e))
-        gate = down[:, s.q_rank + R + r:] if self.has_gate else None
+        gate = down[:, self.q_cols + R + r:] if self.has_gate else None
         ops.head_linear(mixed, R, R, self.w_uv, heads, e, gate, e)
         return linear_partial(heads, self.w_o, rt, "mixer_out")
 

@@ -33,6 +33,12 @@ class RMSNorm:
         ops.rmsnorm(residual, self.weight, self.eps, out, delta=delta, delta_scale=delta_scale, rows=rows)
         return out
 
+    def forward_update(self, stream, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """out = norm of the stream after what the sublayer in front left pending has joined it (parts/block.py,
+        ResidualStream: gated, normed or as it is); written back unless `rows` picks a subset."""
+        ops.residual_norm(stream.x, out, "rms", self.weight, None, self.eps, rows=rows, **stream.update())
+        return out
+
     def forward_pair(self, residual: torch.Tensor, out: torch.Tensor, other: Optional["RMSNorm"],
                      other_out: Optional[torch.Tensor], delta_a: Optional[torch.Tensor] = None,
                      delta_b: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> None:
@@ -97,6 +103,11 @@ class LayerNorm:
         subset."""
         ops.stream_layer_norm(residual, 1, self.weight, self.bias, self.eps, out, delta=delta, delta_scale=delta_scale,
                               rows=rows)
+        return out
+
+    def forward_update(self, stream, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """As RMSNorm.forward_update."""
+        ops.residual_norm(stream.x, out, "layer", self.weight, self.bias, self.eps, rows=rows, **stream.update())
         return out
 
     def forward_stream(self, streams: torch.Tensor, parts: int, out: torch.Tensor, init: Optional[torch.Tensor] = None,

@@ -8,7 +8,7 @@ frequencies are made here in 32-bit floats exactly as the reference makes them,
 "rotary_interleaved": rotary embedding in the interleaved layout: numbers 2i and 2i + 1 of the first `rotary_dim`
 of a vector form a pair that turns by position * theta^(-2i / rotary_dim). The frequencies are kept in double
 precision and the kernels form the angle in double precision (csrc/latent_attention.cu), so the rotation is exact to
-float32 at any position; the mixer that uses it asks for `frequencies`.
+float32 at any position; the mixer that uses it asks for `frequencies` (and `magnitude`, a factor on the turned numbers).
 "none": no position encoding.
 
 A further kind implements `table()` returning None and `apply(q, k, positions)` rotating its views in
@@ -81,6 +81,7 @@ class InterleavedRotaryEncoding:
             if len(spec.factors) != spec.rotary_dim // 2:
                 raise Unsupported(f"rotary encoding has {len(spec.factors)} factors for {spec.rotary_dim // 2} pairs")
             freq = freq / np.asarray(spec.factors, dtype=np.float64)
+        self.magnitude = float(spec.get("magnitude", 1.0))     # what cos and sin are multiplied by
         self.frequencies = torch.from_numpy(freq).to(runtime.device)
         # the same in float32, for a kernel that forms the angle in float32 (csrc/qk_proj_norm.cu)
         self.inv_freq = torch.from_numpy(freq.astype(np.float32)).to(runtime.device)
