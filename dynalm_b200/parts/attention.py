@@ -200,7 +200,7 @@ class GatedNormedAttention(PagedAttention):
         if spec.get("conv", 0) > 0:
             for name, n in (("q", qw), ("k", kw), ("v", vw)):
                 if name == "q" or spec.get("own_kv", True):
-                    more[name + "_conv"] = TensorDecl((n, spec.conv), role="vector", init="bias")
+                    more[name + "_conv"] = TensorDecl((n, spec.conv), role="vector", init="around_one")
         if spec.get("distance_bias", "none") == "log":
             more.update({n: TensorDecl((spec.num_heads,), role="vector", init="around_one") for n in ("distance_rate", "distance_step")})
         return {

@@ -217,7 +217,7 @@ class PlainSipelorn:
         m, t, p = self.cfg["layers"][i]["mixer"], self.t, f"l{i}.mix."
         T = h.shape[0]
         H, d, r, e, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
-        freq, mag = yarn(m["rot"]["base"], m["rot"]["dims"], m["rot"].get("scaling"))
+        freq, mag = yarn(m["rot"]["base"], m["rot"]["dims"], m["rot"].get("scaling")) if m.get("rot") else (np.zeros(0), 1.0)
         q = (h @ t[p + "q"].T).reshape(T, H, d + r)
         q = np.concatenate([q[..., :d], rotate_pairs(q[..., d:], positions, freq, mag)], axis=-1)
         low = h @ t[p + "dkv"].T
@@ -252,8 +252,9 @@ class PlainSipelorn:
         returns the stream [T, W]."""
         t, cfg = self.t, self.cfg
         tokens = [int(x) for x in tokens]
-        x = t["embed"][tokens] * cfg["embedding"]["scale"]
-        pairs = cfg["embedding"].get("bigram")
+        emb = cfg.get("embedding") or {}
+        x = t["embed"][tokens] * emb.get("scale", 1.0)
+        pairs = emb.get("bigram")
         if pairs:
             x = x + t["bigram"][bigram_rows(tokens, last.get("token"), pairs)]
         last["token"] = tokens[-1]
