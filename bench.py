@@ -450,6 +450,43 @@ def bugapel_pair(name):
     return bugapel, rodelorn
 
 
+# --workload sipelorn: the Sipelorn design (latent attention, and windowed attention with short convolutions, a distance
+# bias and caches read across layers; gated residuals; a token's own input per layer; gated experts with a shared one)
+# beside Bugapel, the closest design here (attention through the same kernels, a mixture of experts), at equal width and
+# depth: the weights a token's feed-forward uses are Bugapel's (its two ungated experts of ff against two gated ones of
+# ff / 2 and a shared one of ff / 3; in the layer with latent attention a dense feed-forward of 2 ff).
+SIPELORN_SIZES = {
+    # name: (width, layer kinds (l: latent attention, w: windowed attention, r: the same reading the layer in front's
+    #        cache), attention (heads, kv_heads, dim, vdim, window, taps), latent (heads, dim, rot_dim, vdim, kv_rank),
+    #        token side, buckets of token pairs, bugapel size)
+    "w2048_d128": (2048, "lwrw", (16, 4, 128, 128, 1024, 4), (16, 128, 64, 128, 512), 256, 65536, "w2048_d128"),
+    "w4096_d128": (4096, "lw", (32, 8, 128, 128, 2048, 4), (32, 128, 64, 128, 512), 256, 65536, "w4096_d128"),
+    "w2048_d64": (2048, "lwrw", (32, 8, 64, 64, 512, 4), (32, 64, 32, 64, 256), 128, 65536, "w2048_d64"),
+}
+
+
+def sipelorn_pair(name):
+    width, kinds, a, l, side, buckets, bug = SIPELORN_SIZES[name]
+    x = BUGAPEL_SIZES[bug][4]
+    windowed = {"heads": a[0], "kv_heads": a[1], "dim": a[2], "vdim": a[3], "scale": a[2] ** -0.5, "mask": {"size": a[4]},
+                "conv": a[5]}
+    lat = {"heads": l[0], "dim": l[1], "rot_dim": l[2], "vdim": l[3], "kv_rank": l[4], "scale": (l[1] + l[2]) ** -0.5,
+           "rot": {"base": 10000.0, "dims": l[2], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    mlp = {"kind": "moe", "expert": {"ff": x[4] // 2}, "shared": {"ff": x[4] // 3},
+           "router": {"experts": x[0], "top": x[1], "groups": {"count": x[2], "keep": x[3]}}}
+    layers = []
+    for i, k in enumerate(kinds):
+        if k == "l":
+            layers.append({"type": "latent_attention", "mixer": dict(lat), "mlp": {"kind": "dense", "ff": 2 * x[4]}})
+        else:
+            layers.append({"type": "attention", "mixer": dict(windowed, **({"kv_from": i - 1} if k == "r" else {})), "mlp": dict(mlp)})
+    sipelorn = {"architecture": "Sipelorn", "vocab": ARCH_VOCAB, "width": width, "norm": {"eps": 1e-5},
+                "embedding": {"scale": 8.0, "bigram": {"buckets": buckets, "mul_prev": 31337, "mul_cur": 7}},
+                "token_side": {"dim": side}, "layers": layers}
+    bugapel, _ = bugapel_pair(bug)
+    return sipelorn, bugapel
+
+
 def arch_compare(args, kernels: bool, design: str = "todupel"):
     """Prefill (one prompt of 2,048 tokens) and decode (batches of 8 and 64 holding 2,048 tokens each) of a design
     and of the model it is set beside (the Llama shape, or Rematar for Rodelorn) at equal size, timed with CUDA events; with `kernels`, instead, the device time of every kernel
@@ -464,9 +501,10 @@ def arch_compare(args, kernels: bool, design: str = "todupel"):
 
     peaks = load_peaks()
     T, HELD_HERE, K = 2048, 2048, max(8, min(args.steps, 64))
-    sizes = {"todupel": ARCH_SIZES, "rematar": REMATAR_SIZES, "rodelorn": RODELORN_SIZES, "bugapel": BUGAPEL_SIZES}[design]
-    other = {"rodelorn": "rematar", "bugapel": "rodelorn"}.get(design, "llama")
-    beside = {"rematar": "Rematar", "rodelorn": "Rodelorn", "llama": "the Llama shape"}[other]
+    sizes = {"todupel": ARCH_SIZES, "rematar": REMATAR_SIZES, "rodelorn": RODELORN_SIZES, "bugapel": BUGAPEL_SIZES,
+             "sipelorn": SIPELORN_SIZES}[design]
+    other = {"rodelorn": "rematar", "bugapel": "rodelorn", "sipelorn": "bugapel"}.get(design, "llama")
+    beside = {"rematar": "Rematar", "rodelorn": "Rodelorn", "bugapel": "Bugapel", "llama": "the Llama shape"}[other]
     out = {"metric": f"{design.capitalize()} beside {beside} of equal size: prefill and decode tokens/s", "unit": "tokens/s",
            "n_gpus": 1, "dtype": "bf16", "data": "synthetic: random weights, random token ids", "peaks": peaks,
            "config": {"prefill_tokens": T, "decode_context": HELD_HERE, "decode_steps": K, "vocab": ARCH_VOCAB,
@@ -489,6 +527,11 @@ def arch_compare(args, kernels: bool, design: str = "todupel"):
             rec = {"shape": {"width": width, "layers": kinds, "attention": list(a), "linear_attention": list(g),
                              "experts": list(x), "streams": 4, "rodelorn": rod}}
             pair = bugapel_pair(size)
+        elif design == "sipelorn":
+            width, kinds, a, l, side, buckets, bug = SIPELORN_SIZES[size]
+            rec = {"shape": {"width": width, "layers": kinds, "attention": list(a), "latent_attention": list(l),
+                             "token_side": side, "token_pairs": buckets, "bugapel": bug}}
+            pair = sipelorn_pair(size)
         else:
             width, kinds, d, a, r, ff, rem = RODELORN_SIZES[size]
             rec = {"shape": {"width": width, "layers": kinds, "delta": list(d), "attention": list(a), "recurrence": list(r),
@@ -568,10 +611,10 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=FULL_LAYERS, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--workload", choices=["decode", "todupel", "todupel-kernels", "rematar", "rematar-kernels", "rodelorn", "rodelorn-kernels", "bugapel", "bugapel-kernels"] + sorted(SERVING), default="decode",
+    ap.add_argument("--workload", choices=["decode", "todupel", "todupel-kernels", "rematar", "rematar-kernels", "rodelorn", "rodelorn-kernels", "bugapel", "bugapel-kernels", "sipelorn", "sipelorn-kernels"] + sorted(SERVING), default="decode",
                     help="decode: the default benchmark; serve3b / serve8b: continuous batching of the 3B / 8B workloads; "
                          "todupel / rematar: that design beside the Llama shape of equal size; rodelorn: that design beside Rematar of "
-                         "equal size; bugapel: that design beside Rodelorn of equal size (<design>-kernels: per kernel)")
+                         "equal size; bugapel: that design beside Rodelorn of equal size; sipelorn: that design beside Bugapel of equal size (<design>-kernels: per kernel)")
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
     ap.add_argument("--no-long", action="store_true", help="skip the points at 8,192 tokens (prefill and decode)")
     ap.add_argument("--no-serve", action="store_true", help="skip the points of the 3B and 8B serving workloads")
@@ -586,7 +629,7 @@ def main():
     if args.gpus != 1:
         print(f"bench.py: this engine runs on one GPU; --gpus {args.gpus} is not supported")
         return 2
-    if args.workload.split("-")[0] in ("todupel", "rematar", "rodelorn", "bugapel"):
+    if args.workload.split("-")[0] in ("todupel", "rematar", "rodelorn", "bugapel", "sipelorn"):
         return arch_compare(args, kernels=args.workload.endswith("-kernels"), design=args.workload.split("-")[0])
     if args.workload != "decode":
         return serving(args.workload, args.layers if args.layers != FULL_LAYERS else None)
