@@ -132,6 +132,15 @@ __device__ __forceinline__ float xielu_f(float z, float c0, float c1) {
   return 0.5f * z + (z > 0.0f ? c0 * z * z : c1 * (expm1f(z) - z));
 }
 
+// The same for results that are rounded to bf16 right away, in few instructions: c1 e^z + ((1/2 - c1) z - c1) with the
+// hardware's 2^x below zero. Near zero its absolute error is a few 2^-23 of c1, far below what the product behind it sees.
+__device__ __forceinline__ float xielu_bf16(float z, float c0, float c1) {
+  float t;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(t) : "f"(z * 1.4426950408889634f));
+  const float neg = fmaf(c1, t, fmaf(0.5f - c1, z, -c1)), pos = z * fmaf(c0, z, 0.5f);
+  return z > 0.0f ? pos : neg;
+}
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // Programmatic dependent launch. A kernel launched with the attribute may begin while the kernel before it on

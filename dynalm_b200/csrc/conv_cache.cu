@@ -118,6 +118,105 @@ conv_cache_kernel(const ConvCacheParams p) {
   }
 }
 
+// The same for steps of many rows: a thread walks R consecutive rows of V channels with its taps and the last K - 1 inputs
+// (bias included, zeros in front of a start) in registers, so that a row is read once; where a request begins among the
+// rows the inputs come from what it kept. Rows of requests of one token shift their kept inputs as above.
+template <typename T, int V, int R, int K>
+__global__ void __launch_bounds__(256)
+conv_cache_rows_kernel(const ConvCacheParams p) {
+  const int C = p.Cq + p.Ck + p.Cv, per_row = C / V;
+  const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  const int row0 = static_cast<int>(idx / per_row) * R, ch = static_cast<int>(idx % per_row) * V;
+  if (row0 >= p.rows) return;
+  const T* col = static_cast<const T*>(p.proj) + ch;
+  float ib[V], tk[K][V], win[K][V];            // win[j]: the input j - (K - 1) tokens from the current one
+#pragma unroll
+  for (int i = 0; i < V; i += 4) {
+    const float4 b4 = p.bias != nullptr ? *reinterpret_cast<const float4*>(p.bias + ch + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ib[i] = b4.x; ib[i + 1] = b4.y; ib[i + 2] = b4.z; ib[i + 3] = b4.w;
+#pragma unroll
+    for (int j = 0; j < K; ++j) {
+      const float4 t4 = *reinterpret_cast<const float4*>(p.taps + static_cast<size_t>(j) * C + ch + i);
+      tk[j][i] = t4.x; tk[j][i + 1] = t4.y; tk[j][i + 2] = t4.z; tk[j][i + 3] = t4.w;
+    }
+  }
+  int req = -1, first_row = 0, next_first = 0, slot = 0;
+  const int* table = nullptr;
+  float* kept = nullptr;
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int row = row0 + r;
+    if (row >= p.rows) return;
+    const int pos = p.positions[row];
+    bool fill = r == 0;
+    if (r == 0 || row >= next_first) {           // another request begins
+      req = p.row_request[row];
+      first_row = p.q_start[req];
+      next_first = p.q_start[req + 1];
+      slot = ck_request(p.row_slot[row]);
+      table = p.block_table + static_cast<size_t>(slot) * p.max_blocks;
+      kept = p.kept + static_cast<size_t>(slot) * p.kept_stride + ch;
+      fill = true;
+    }
+    if (fill) {
+      const bool single = next_first - first_row == 1;
+#pragma unroll
+      for (int j = 0; j < K - 1; ++j) {
+        const int k = K - 1 - j;                 // tokens back
+        float u[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) u[i] = 0.0f;
+        if (pos - k >= 0) {
+          const int back = row - k;
+          if (back >= first_row) {
+            cc_load<T, V>(col + static_cast<size_t>(back) * p.proj_stride, u);
+          } else {
+            const float* kr = kept + static_cast<size_t>(K - 1 - (first_row - back)) * C;
+#pragma unroll
+            for (int i = 0; i < V; ++i) u[i] = kr[i];
+          }
+          if (single && j > 0) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) kept[static_cast<size_t>(j - 1) * C + i] = u[i];
+          }
+#pragma unroll
+          for (int i = 0; i < V; ++i) u[i] += ib[i];
+        } else if (single && j > 0) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) kept[static_cast<size_t>(j - 1) * C + i] = 0.0f;
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) win[j][i] = u[i];
+      }
+    }
+    float u[V], acc[V];
+    cc_load<T, V>(col + static_cast<size_t>(row) * p.proj_stride, u);
+    if (next_first - first_row == 1) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) kept[static_cast<size_t>(K - 2) * C + i] = u[i];
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      win[K - 1][i] = u[i] + ib[i];
+      acc[i] = 0.0f;
+#pragma unroll
+      for (int j = 0; j < K; ++j) acc[i] = fmaf(tk[j][i], win[j][i], acc[i]);      // oldest input first
+#pragma unroll
+      for (int j = 0; j < K - 1; ++j) win[j][i] = win[j + 1][i];
+    }
+    if (ch < p.Cq) {
+      cc_store<T, V>(static_cast<T*>(p.q_out) + static_cast<size_t>(row) * p.q_stride + ch, acc);
+    } else {
+      const int page = ck_page_store(table, pos / p.page_size, p.max_blocks);
+      if (page >= 0) {
+        const size_t place = static_cast<size_t>(page) * p.page_size + pos % p.page_size;
+        if (ch < p.Cq + p.Ck) cc_store<T, V>(static_cast<T*>(p.k_cache) + place * p.k_row + (ch - p.Cq), acc);
+        else cc_store<T, V>(static_cast<T*>(p.v_cache) + place * p.v_row + (ch - p.Cq - p.Ck), acc);
+      }
+    }
+  }
+}
+
 // The last K - 1 inputs of every request that brought more than one token, oldest first. One thread per (request,
 // channel); entries are written in ascending order, and entry j only ever needs an older entry at a higher index.
 template <typename T>
@@ -162,6 +261,18 @@ DL_EXPORT int dl_conv_cache(int dtype, const void* proj, long long proj_stride, 
     const size_t n = static_cast<size_t>((rows + R - 1) / R) * ((Cq + Ck + Cv) / V);                            \
     dl::conv_cache_kernel<T, V, R><<<static_cast<unsigned>((n + 255) / 256), 256, 0, stream>>>(p);              \
   } while (0)
+  // many rows: a thread walks eight of them (bfloat16, 2 to 4 taps)
+  const bool walk = dtype == 1 && wide && rows >= 256 && taps != nullptr && K >= 2 && K <= 4 &&
+                    ((reinterpret_cast<uintptr_t>(taps) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0;
+  if (walk) {
+    constexpr int R = 8;
+    const size_t n = static_cast<size_t>((rows + R - 1) / R) * ((Cq + Ck + Cv) / 8);
+    const unsigned blocks = static_cast<unsigned>((n + 255) / 256);
+    if (K == 2) dl::conv_cache_rows_kernel<dl::bf16, 8, R, 2><<<blocks, 256, 0, stream>>>(p);
+    else if (K == 3) dl::conv_cache_rows_kernel<dl::bf16, 8, R, 3><<<blocks, 256, 0, stream>>>(p);
+    else dl::conv_cache_rows_kernel<dl::bf16, 8, R, 4><<<blocks, 256, 0, stream>>>(p);
+    return dl::launch_status();
+  }
   if (dtype == 0) { if (wide) DL_CC(float, 4, 1); else DL_CC(float, 1, 1); }
   else if (dtype == 1) { if (wide) DL_CC(dl::bf16, 8, 1); else DL_CC(dl::bf16, 1, 1); }
   else return DL_ERR_UNSUPPORTED;

@@ -38,7 +38,7 @@ __device__ __forceinline__ void mma16816(float (&d)[4], uint32_t a0, uint32_t a1
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-enum { SK_OUT_BF16 = 0, SK_OUT_F32 = 1, SK_OUT_SWIGLU = 2, SK_OUT_ARGMAX = 3, SK_OUT_RELU2 = 4, SK_OUT_GELU = 5 };
+enum { SK_OUT_BF16 = 0, SK_OUT_F32 = 1, SK_OUT_SWIGLU = 2, SK_OUT_ARGMAX = 3, SK_OUT_RELU2 = 4, SK_OUT_GELU = 5, SK_OUT_XIELU = 6 };
 
 // The weight stream of one block: y^T tile = W rows (wrow, 16 * MT of them in MMA row order) times x^T, k-blocks
 // [blk_begin, blk_end) dealt to the warps round-robin. Leaves every warp's partial tile in `red`
@@ -149,7 +149,7 @@ template <int MT, int NT>
 __global__ void __launch_bounds__(SK_THREADS, (MT == 1 && NT <= 2) ? (NT == 1 ? SK_BLOCKS_8 : SK_BLOCKS_16) : 1)
 gemm_skinny_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__ w, void* __restrict__ y, int ldy,
                    int M, int N, int K, int mode, float out_scale, long long split_stride,
-                   const void* __restrict__ ahead, long long ahead_bytes) {
+                   const void* __restrict__ ahead, long long ahead_bytes, const float* __restrict__ coeffs) {
   extern __shared__ float red[];     // [SK_WARPS][MT * 16][NT * 8]
   const int lane = threadIdx.x & 31;
   const int g = lane >> 2;
@@ -239,6 +239,8 @@ gemm_skinny_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__
         v *= v;
       } else if (mode == SK_OUT_GELU) {  // or its GELU in the tanh form
         v = gelu_tanh_bf16(v);
+      } else if (mode == SK_OUT_XIELU) {
+        v = xielu_bf16(v, coeffs[0], coeffs[1]);
       }
       static_cast<bf16*>(y)[static_cast<size_t>(b) * ldy + f] = __float2bfloat16_rn(v);
     }
@@ -316,7 +318,7 @@ gemm_skinny_qkv_rope_kernel(const bf16* __restrict__ x, int ldx, const bf16* __r
 template <int MT, int NT>
 int launch_skinny(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode,
                   float out_scale, int n_split, long long split_stride, const void* ahead, long long ahead_bytes,
-                  cudaStream_t stream) {
+                  const float* coeffs, cudaStream_t stream) {
   const int feats = mode == SK_OUT_SWIGLU ? N / 2 : N;
   const int per_block = mode == SK_OUT_SWIGLU ? MT * 8 : MT * 16;
   dim3 grid((feats + per_block - 1) / per_block, n_split);
@@ -330,7 +332,7 @@ int launch_skinny(const void* x, int ldx, const void* w, void* y, int ldy, int M
   }
   return launch_streaming(gemm_skinny_kernel<MT, NT>, grid, dim3(SK_THREADS), smem, stream, static_cast<const bf16*>(x), ldx,
                 static_cast<const bf16*>(w), y, ldy, M, N, K, mode, out_scale, split_stride,
-                pdl_mode() >= 1 ? ahead : nullptr, pdl_mode() >= 1 ? ahead_bytes : 0ll);
+                pdl_mode() >= 1 ? ahead : nullptr, pdl_mode() >= 1 ? ahead_bytes : 0ll, coeffs);
 }
 
 }  // namespace dl
@@ -338,22 +340,22 @@ int launch_skinny(const void* x, int ldx, const void* w, void* y, int ldy, int M
 // x: bf16 [M, K] rows of ldx elements (16-byte aligned rows), w: bf16 [N, K] contiguous, K a multiple of 8,
 // M <= 64. mode 0: y bf16 [M, N]; mode 1: y fp32, n_split partial results of [M, ldy] floats each,
 // split_stride floats apart; mode 2: w = [gate; up] (N even), y bf16 [M, N / 2] = silu(x Wg^T) * (x Wu^T).
-// mode 4: y bf16 [M, N] = max(x W^T, 0)^2. mode 3: nothing but the place of each row's largest output leaves the kernel: y = float [M][blocks] then
+// mode 4: y bf16 [M, N] = max(x W^T, 0)^2; mode 6: = xIELU(x W^T) with coeffs = two float32 on the device. mode 3: nothing but the place of each row's largest output leaves the kernel: y = float [M][blocks] then
 // int [M][blocks] (blocks = ceil(N / features per block), see dl_gemm_skinny_argmax_blocks), the largest value of every
 // block's features and its feature index (the lowest among equals); out_scale must be positive.
 // n_split > 1 needs mode 1. ahead, ahead_bytes: memory that the kernel after this one will stream (weights),
 // requested into L2 before this kernel waits for the one in front of it; null / 0: nothing.
 DL_EXPORT int dl_gemm_skinny(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode,
                              float out_scale, int n_split, long long split_stride, const void* ahead,
-                             long long ahead_bytes, cudaStream_t stream) {
+                             long long ahead_bytes, const float* coeffs, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || (K & 7) || (ldx & 7) || n_split < 1 || n_split > 64 || (n_split > 1 && mode != dl::SK_OUT_F32) ||
-      (mode == dl::SK_OUT_SWIGLU && (N & 1)) || mode < 0 || mode > 5 || (mode == dl::SK_OUT_ARGMAX && !(out_scale > 0.0f)))
+      (mode == dl::SK_OUT_SWIGLU && (N & 1)) || mode < 0 || mode > 6 || (mode == dl::SK_OUT_XIELU && coeffs == nullptr) || (mode == dl::SK_OUT_ARGMAX && !(out_scale > 0.0f)))
     return DL_ERR_UNSUPPORTED;
-  if (M <= 8) return dl::launch_skinny<1, 1>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, stream);
-  if (M <= 16) return dl::launch_skinny<1, 2>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, stream);
-  if (M <= 32) return dl::launch_skinny<2, 4>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, stream);
-  return dl::launch_skinny<2, 8>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, stream);
+  if (M <= 8) return dl::launch_skinny<1, 1>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, coeffs, stream);
+  if (M <= 16) return dl::launch_skinny<1, 2>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, coeffs, stream);
+  if (M <= 32) return dl::launch_skinny<2, 4>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, coeffs, stream);
+  return dl::launch_skinny<2, 8>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, ahead, ahead_bytes, coeffs, stream);
 }
 
 // Blocks (= partial results per row) of dl_gemm_skinny in mode 3 for M rows and N features.

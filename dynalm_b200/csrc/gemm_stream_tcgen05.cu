@@ -30,7 +30,7 @@ constexpr int GS_BM = 128;                 // features per tile
 constexpr int GS_BK = 64;                  // 64 bf16 = 128 bytes: one swizzle row
 constexpr int GS_THREADS = 192;
 constexpr uint32_t GS_A_BYTES = GS_BM * GS_BK * 2;
-enum { GS_OUT_BF16 = 0, GS_OUT_F32 = 1, GS_OUT_SWIGLU = 2, GS_OUT_RELU2 = 3, GS_OUT_GELU = 4 };
+enum { GS_OUT_BF16 = 0, GS_OUT_F32 = 1, GS_OUT_SWIGLU = 2, GS_OUT_RELU2 = 3, GS_OUT_GELU = 4, GS_OUT_XIELU = 5 };
 enum { GS_ERR_PRODUCER = 21, GS_ERR_MMA = 22, GS_ERR_EPILOGUE = 23 };
 
 template <int NB> struct GS {
@@ -59,7 +59,7 @@ template <int NB>
 __global__ void __launch_bounds__(GS_THREADS, 1)
 gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, void* __restrict__ y,
                    int ldy, int M, int N, int K, int mode, float out_scale, int gate_rows, long long split_stride,
-                   int* __restrict__ status) {
+                   int* __restrict__ status, const float* __restrict__ coeffs) {
   constexpr int STAGES = GS<NB>::STAGES;
   constexpr uint32_t STAGE_BYTES = GS<NB>::STAGE_BYTES, B_BYTES = GS<NB>::B_BYTES, TMEM_COLS = GS<NB>::TMEM_COLS;
   extern __shared__ unsigned char gs_raw[];
@@ -182,7 +182,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
 #pragma unroll
         for (int j = 0; j < 16; ++j) acc[c0 + j] = __uint_as_float(v[j]);
       }
-      if (mode == GS_OUT_BF16 || mode == GS_OUT_F32 || mode == GS_OUT_RELU2 || mode == GS_OUT_GELU) {
+      if (mode == GS_OUT_BF16 || mode == GS_OUT_F32 || mode == GS_OUT_RELU2 || mode == GS_OUT_GELU || mode == GS_OUT_XIELU) {
         const int f = f0 + fl;
         if (f < N) {
           if (mode == GS_OUT_F32) {
@@ -201,6 +201,8 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                   v *= v;
                 } else if (mode == GS_OUT_GELU) {  // or its GELU in the tanh form
                   v = gelu_tanh_bf16(v);
+                } else if (mode == GS_OUT_XIELU) {
+                  v = xielu_bf16(v, coeffs[0], coeffs[1]);
                 }
                 out[static_cast<size_t>(b) * ldy] = __float2bfloat16_rn(v);
               }
@@ -260,7 +262,7 @@ static int gs_make_map(CUtensorMap* map, const void* base, int rows, int cols, i
 template <int NB>
 static int gs_launch(const CUtensorMap& map_w, const CUtensorMap& map_x, void* y, int ldy, int M, int N, int K, int mode,
                      float out_scale, int gate_rows, int n_tiles, int n_split, long long split_stride, int* status,
-                     cudaStream_t stream) {
+                     const float* coeffs, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -269,11 +271,11 @@ static int gs_launch(const CUtensorMap& map_w, const CUtensorMap& map_x, void* y
     configured = true;
   }
   return launch_streaming(gemm_stream_kernel<NB>, dim3(n_tiles, n_split), dim3(GS_THREADS), GS<NB>::SMEM, stream, map_w, map_x,
-                          y, ldy, M, N, K, mode, out_scale, gate_rows, split_stride, status);
+                          y, ldy, M, N, K, mode, out_scale, gate_rows, split_stride, status, coeffs);
 }
 
 static int gs_run(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode, float out_scale,
-                  int n_split, long long split_stride, int* status, cudaStream_t stream) {
+                  int n_split, long long split_stride, int* status, const float* coeffs, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || (K & 7) || (ldx & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) ||
       status == nullptr || n_split < 1 || n_split > 64 || (n_split > 1 && mode != GS_OUT_F32) ||
@@ -290,10 +292,10 @@ static int gs_run(const void* x, int ldx, const void* w, void* y, int ldy, int M
   rc = gs_make_map(&map_x, x, M, K, ldx, nb);
   if (rc != 0) return rc;
   if (nb == 16)
-    return gs_launch<16>(map_w, map_x, y, ldy, M, N, K, mode, out_scale, gate_rows, n_tiles, n_split, split_stride, status, stream);
+    return gs_launch<16>(map_w, map_x, y, ldy, M, N, K, mode, out_scale, gate_rows, n_tiles, n_split, split_stride, status, coeffs, stream);
   if (nb == 32)
-    return gs_launch<32>(map_w, map_x, y, ldy, M, N, K, mode, out_scale, gate_rows, n_tiles, n_split, split_stride, status, stream);
-  return gs_launch<64>(map_w, map_x, y, ldy, M, N, K, mode, out_scale, gate_rows, n_tiles, n_split, split_stride, status, stream);
+    return gs_launch<32>(map_w, map_x, y, ldy, M, N, K, mode, out_scale, gate_rows, n_tiles, n_split, split_stride, status, coeffs, stream);
+  return gs_launch<64>(map_w, map_x, y, ldy, M, N, K, mode, out_scale, gate_rows, n_tiles, n_split, split_stride, status, coeffs, stream);
 }
 
 }  // namespace dl
@@ -303,7 +305,9 @@ static int gs_run(const void* x, int ldx, const void* w, void* y, int ldy, int M
 // apart (n_split > 1 needs this mode); mode 2: w = [gate; up] with N = 2F rows, y bf16 [M, F] = silu(x Wg^T) * (x Wu^T).
 // status: one device int, set to a nonzero code if a wait inside the kernel timed out (left untouched otherwise).
 DL_EXPORT int dl_gemm_stream(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode,
-                             float out_scale, int n_split, long long split_stride, int* status, cudaStream_t stream) {
-  if (mode < 0 || mode > 4) return DL_ERR_UNSUPPORTED;     // 3: y bf16 [M, N] = max(x W^T, 0)^2; 4: = gelu_tanh(x W^T)
-  return dl::gs_run(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, status, stream);
+                             float out_scale, int n_split, long long split_stride, const float* coeffs, int* status,
+                             cudaStream_t stream) {
+  // 3: y bf16 [M, N] = max(x W^T, 0)^2; 4: = gelu_tanh(x W^T); 5: = xIELU(x W^T) with coeffs = two float32 on the device
+  if (mode < 0 || mode > 5 || (mode == dl::GS_OUT_XIELU && coeffs == nullptr)) return DL_ERR_UNSUPPORTED;
+  return dl::gs_run(x, ldx, w, y, ldy, M, N, K, mode, out_scale, n_split, split_stride, status, coeffs, stream);
 }

@@ -47,10 +47,10 @@ DL_EXPORT int dl_gemm_tcgen05_tile_coords(int tile, int tiles_n, int num_tiles, 
 }
 
 DL_EXPORT int dl_gemm_tcgen05(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode,
-                              float out_scale, int* status, cudaStream_t stream) {
-  if (mode < 0 || (mode > 2 && mode != dl::T5_OUT_RELU2 && mode != dl::T5_OUT_GELU)) return DL_ERR_UNSUPPORTED;
+                              float out_scale, const float* coeffs, int* status, cudaStream_t stream) {
+  if (mode < 0 || (mode > 2 && mode != dl::T5_OUT_RELU2 && mode != dl::T5_OUT_GELU && mode != dl::T5_OUT_XIELU)) return DL_ERR_UNSUPPORTED;
   const dl::QkvRope none = {};
-  return t5_launch<dl::T5Alone>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, status, none, stream);
+  return t5_launch<dl::T5Alone>(x, ldx, w, y, ldy, M, N, K, mode, out_scale, status, none, stream, coeffs);
 }
 
 // A grouped product on the same kernel: runs of a's rows, listed on the device as row tiles (matrix, first row, rows <=

@@ -23,7 +23,7 @@ template <int BN> struct T5 {
   static constexpr size_t SMEM = static_cast<size_t>(STAGES) * STAGE_BYTES + T5_STORE_BYTES + 1024 /* alignment */ + 256 /* barriers */;
 };
 
-enum { T5_OUT_BF16 = 0, T5_OUT_F32 = 1, T5_OUT_SWIGLU = 2, T5_OUT_QKV_ROPE = 3, T5_OUT_RELU2 = 4, T5_OUT_GELU = 5, T5_OUT_PAIRS = 6 };
+enum { T5_OUT_BF16 = 0, T5_OUT_F32 = 1, T5_OUT_SWIGLU = 2, T5_OUT_QKV_ROPE = 3, T5_OUT_RELU2 = 4, T5_OUT_GELU = 5, T5_OUT_PAIRS = 6, T5_OUT_XIELU = 7 };
 enum { T5_ERR_PRODUCER = 1, T5_ERR_MMA = 2, T5_ERR_EPILOGUE = 3 };
 
 // Which output tile a tile number stands for. Tiles are numbered in groups of `group_m` row blocks: inside a
@@ -74,7 +74,7 @@ __global__ void __launch_bounds__(T5_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                     void* __restrict__ y, int ldy, int M, int N, int K, int mode, float out_scale, int gate_rows,
                     int tiles_n, int num_tiles_plain, int group_m, int* __restrict__ status, const QkvRope rope,
-                    const T5Groups groups) {
+                    const T5Groups groups, const float* __restrict__ coeffs) {
   constexpr int T5_STAGES = T5<T5_BN>::STAGES;
   constexpr uint32_t T5_B_BYTES = T5<T5_BN>::B_BYTES, T5_STAGE_BYTES = T5<T5_BN>::STAGE_BYTES, T5_TMEM_COLS = T5<T5_BN>::TMEM_COLS;
   extern __shared__ unsigned char t5_raw[];
@@ -346,6 +346,27 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
             store_rows_pieces(wlo, whi, my_stage, lane, dst, piece * 32, hd / 2 + piece * 32);
           }
         }
+      } else if (mode == T5_OUT_XIELU) {
+        // xIELU with the two coefficients in memory; a branch of its own, so that the plain epilogue stays as small as it was
+        const float c0_x = coeffs[0], c1_x = coeffs[1];
+        for (int c0 = 0; c0 < T5_BN; c0 += 64) {
+          uint4 w[8];
+#pragma unroll 1
+          for (int hh = 0; hh < 2; ++hh) {
+            uint32_t v[32];
+            tmem_ld32(lane_addr + c0 + hh * 32, v);
+            tmem_ld_wait();
+            auto fin = [&](int j) { return xielu_bf16(__uint_as_float(v[j]), c0_x, c1_x); };
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+              const uint4 q = make_uint4(pack2_bf16(fin(j), fin(j + 1)), pack2_bf16(fin(j + 2), fin(j + 3)),
+                                         pack2_bf16(fin(j + 4), fin(j + 5)), pack2_bf16(fin(j + 6), fin(j + 7)));
+              if (hh == 0) w[j / 8] = q;
+              else w[4 + j / 8] = q;
+            }
+          }
+          store_rows_bf16(w, my_stage, lane, static_cast<bf16*>(y), ldy, row0, M, n0 + c0, N);   // N is a multiple of 8
+        }
       } else if (mode == T5_OUT_PAIRS) {
         // rows 2j and 2j + 1 of W are the gate and up rows of feature j: 128 columns of the tile give 64 of the output
         for (int c0 = 0; c0 < T5_BN; c0 += 128) {
@@ -451,14 +472,15 @@ static inline int make_map(CUtensorMap* map, const void* base, int rows, int col
 
 // x: bf16 [M, K] rows of ldx elements; w: bf16 [N, K] contiguous; both 16-byte aligned with K and ldx multiples of 8.
 // mode 0: y bf16 [M, N] (N % 8 == 0); mode 1: y fp32 [M, N] (N % 4 == 0); mode 2: w = [gate; up] with N = 2F rows,
-// y bf16 [M, F] = silu(x Wg^T) * (x Wu^T) (F % 8 == 0); mode 4: y bf16 [M, N] = max(x W^T, 0)^2; mode 5: = gelu_tanh(x W^T). status: one device int, set to a nonzero code if a wait
+// y bf16 [M, F] = silu(x Wg^T) * (x Wu^T) (F % 8 == 0); mode 4: y bf16 [M, N] = max(x W^T, 0)^2; mode 5: = gelu_tanh(x W^T);
+// mode 7: = xIELU(x W^T) with coeffs = two float32 on the device. status: one device int, set to a nonzero code if a wait
 // inside the kernel timed out (left untouched otherwise).
 template <class P>
 static int t5_launch(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode, float out_scale,
-                     int* status, const dl::QkvRope& rope, cudaStream_t stream) {
+                     int* status, const dl::QkvRope& rope, cudaStream_t stream, const float* coeffs = nullptr) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || (ldx & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) ||
-      status == nullptr || mode < 0 || mode > 5)
+      status == nullptr || mode < 0 || (mode > 5 && mode != dl::T5_OUT_XIELU) || (mode == dl::T5_OUT_XIELU && coeffs == nullptr))
     return DL_ERR_UNSUPPORTED;
   const int feats = mode == dl::T5_OUT_SWIGLU ? N / 2 : N;
   if ((mode == dl::T5_OUT_SWIGLU && (N & 1)) || (mode == dl::T5_OUT_F32 ? (feats & 3) || (ldy & 3) : (feats & 7) || (ldy & 7)) ||
@@ -541,7 +563,7 @@ static int t5_launch(const void* x, int ldx, const void* w, void* y, int ldy, in
     }
     cfg.dynamicSmemBytes = dl::T5<256>::SMEM;
     return static_cast<int>(cudaLaunchKernelEx(&cfg, dl::gemm_tcgen05_kernel<256, P>, map_x, map_w, y, ldy, M, N, K, mode,
-                                               out_scale, gate_rows, tiles_n, static_cast<int>(tiles), group_m, status, rope, dl::T5Groups{nullptr, nullptr, 0}));
+                                               out_scale, gate_rows, tiles_n, static_cast<int>(tiles), group_m, status, rope, dl::T5Groups{nullptr, nullptr, 0}, coeffs));
   } else if (bn == 192) {
     static bool configured = false;
     if (!configured) {
@@ -552,7 +574,7 @@ static int t5_launch(const void* x, int ldx, const void* w, void* y, int ldy, in
     }
     cfg.dynamicSmemBytes = dl::T5<192>::SMEM;
     return static_cast<int>(cudaLaunchKernelEx(&cfg, dl::gemm_tcgen05_kernel<192, P>, map_x, map_w, y, ldy, M, N, K, mode,
-                                               out_scale, gate_rows, tiles_n, static_cast<int>(tiles), group_m, status, rope, dl::T5Groups{nullptr, nullptr, 0}));
+                                               out_scale, gate_rows, tiles_n, static_cast<int>(tiles), group_m, status, rope, dl::T5Groups{nullptr, nullptr, 0}, coeffs));
   } else {
     static bool configured = false;
     if (!configured) {
@@ -563,7 +585,7 @@ static int t5_launch(const void* x, int ldx, const void* w, void* y, int ldy, in
     }
     cfg.dynamicSmemBytes = dl::T5<128>::SMEM;
     return static_cast<int>(cudaLaunchKernelEx(&cfg, dl::gemm_tcgen05_kernel<128, P>, map_x, map_w, y, ldy, M, N, K, mode,
-                                               out_scale, gate_rows, tiles_n, static_cast<int>(tiles), group_m, status, rope, dl::T5Groups{nullptr, nullptr, 0}));
+                                               out_scale, gate_rows, tiles_n, static_cast<int>(tiles), group_m, status, rope, dl::T5Groups{nullptr, nullptr, 0}, coeffs));
   }
 }
 
@@ -615,7 +637,7 @@ static int t5_launch_grouped(const void* a, int lda, int rows, const void* w, in
     }
     cfg.dynamicSmemBytes = dl::T5<256>::SMEM;
     return static_cast<int>(cudaLaunchKernelEx(&cfg, dl::gemm_tcgen05_kernel<256, P>, map_x, map_w, y, ldy, rows, N, K, mode,
-                                               1.0f, 0, tiles_n, 0, 1, status, none, groups));
+                                               1.0f, 0, tiles_n, 0, 1, status, none, groups, nullptr));
   }
   static bool configured = false;
   if (!configured) {
@@ -626,7 +648,7 @@ static int t5_launch_grouped(const void* a, int lda, int rows, const void* w, in
   }
   cfg.dynamicSmemBytes = dl::T5<128>::SMEM;
   return static_cast<int>(cudaLaunchKernelEx(&cfg, dl::gemm_tcgen05_kernel<128, P>, map_x, map_w, y, ldy, rows, N, K, mode,
-                                             1.0f, 0, tiles_n, 0, 1, status, none, groups));
+                                             1.0f, 0, tiles_n, 0, 1, status, none, groups, nullptr));
 }
 
 // Fills the epilogue's parameters for the q | k | v product and launches it (see dl_gemm_tcgen05_qkv_rope).

@@ -413,15 +413,36 @@ __global__ void moe_combine_kernel(const float* __restrict__ c, int width, const
   }
   if (shared != nullptr) {
     const float g = 1.0f / (1.0f + expf(-shared_z[t * z_stride]));
+    float v[V];
 #pragma unroll
-    for (int j = 0; j < V; ++j) {
-      float v = 0.0f;
-      for (int p = 0; p < parts; ++p) v += to_float(shared[p * part_stride + t * width + col + j]);
-      sum[j] = fmaf(g, v, sum[j]);
+    for (int j = 0; j < V; ++j) v[j] = 0.0f;
+    for (int p = 0; p < parts; ++p) {
+      const TS* src = shared + p * part_stride + t * width + col;
+      float s[V];
+      if constexpr (V == 4 && sizeof(TS) == 2) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(src);
+        s[0] = __uint_as_float(raw.x << 16); s[1] = __uint_as_float(raw.x & 0xffff0000u);
+        s[2] = __uint_as_float(raw.y << 16); s[3] = __uint_as_float(raw.y & 0xffff0000u);
+      } else if constexpr (V == 4) {
+        const float4 raw = *reinterpret_cast<const float4*>(src);
+        s[0] = raw.x; s[1] = raw.y; s[2] = raw.z; s[3] = raw.w;
+      } else {
+        s[0] = to_float(src[0]);
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] += s[j];
     }
-  }
 #pragma unroll
-  for (int j = 0; j < V; ++j) y[t * width + col + j] = from_float<TO>(sum[j]);
+    for (int j = 0; j < V; ++j) sum[j] = fmaf(g, v[j], sum[j]);
+  }
+  TO* dst = y + t * width + col;
+  if constexpr (V == 4 && sizeof(TO) == 2) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(sum[0], sum[1]), b = __floats2bfloat162_rn(sum[2], sum[3]);
+    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  } else {
+#pragma unroll
+    for (int j = 0; j < V; ++j) dst[j] = from_float<TO>(sum[j]);
+  }
 }
 
 }  // namespace dl
@@ -524,7 +545,8 @@ DL_EXPORT int dl_moe_combine(int out_dtype, const float* c, int width, const int
                              int z_stride, void* y, int tokens, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (shared != nullptr && (parts <= 0 || shared_z == nullptr)) return DL_ERR_UNSUPPORTED;
-  const bool wide = width % 4 == 0 && (reinterpret_cast<uintptr_t>(c) & 15) == 0;
+  const bool wide = width % 4 == 0 && part_stride % 4 == 0 &&
+                    ((reinterpret_cast<uintptr_t>(c) | reinterpret_cast<uintptr_t>(shared) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
   const size_t total = static_cast<size_t>(tokens) * (wide ? width / 4 : width);
   const unsigned blocks = static_cast<unsigned>((total + 255) / 256);
 #define DL_MC(TO, TS, V)                                                                                              \

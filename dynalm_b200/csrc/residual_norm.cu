@@ -191,6 +191,7 @@ int launch_residual_norm(const ResidualNormParams& p, int n_out, bool wide, cuda
     const int pieces = (p.W + 3) / 4;
     if (pieces <= 128) DL_RN(4, 1, 128);
     if (pieces <= 256) DL_RN(4, 2, 128);
+    if (pieces <= 512 && n_out >= 512) DL_RN(4, 4, 128);      // many rows: more of a row in flight per thread
     if (pieces <= 512) DL_RN(4, 2, 256);
     if (pieces <= 1024) DL_RN(4, 4, 256);
     if (pieces <= 4096) DL_RN(4, 4, 1024);

@@ -184,34 +184,35 @@ def linear_geglu(x: torch.Tensor, w_gate_up: torch.Tensor, runtime, inner: int) 
     return act
 
 
-def linear_act(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int, activation: str) -> torch.Tensor:
-    """act(x W^T), the first half of an ungated feed-forward, act = "relu2" (max(z, 0)^2) or "gelu_tanh": the
+def linear_act(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int, activation: str,
+               coeffs: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(x W^T), the first half of an ungated feed-forward, act = "relu2" (max(z, 0)^2), "gelu_tanh" or "xielu": the
     activation sits in the product's epilogue wherever one of this package's bfloat16 kernels runs the product, else
     the product is followed by the activation kernel (float32, and the few shapes that go to the library)."""
-    if activation not in ("relu2", "gelu_tanh"):
+    if activation not in ("relu2", "gelu_tanh", "xielu"):
         raise ValueError(f"no kernel for activation '{activation}'")
     rows = x.shape[0]
     act = runtime.buffer("ffn_act", (rows, inner))
     if x.dtype == torch.bfloat16 and use_stream(x, w_up):
-        ops.gemm_stream(x, w_up, act, activation)
+        ops.gemm_stream(x, w_up, act, activation, coeffs=coeffs)
         return act
     if x.dtype == torch.bfloat16 and skinny_ok(x, w_up):
-        ops.gemm_skinny(x, w_up, act, activation)
+        ops.gemm_skinny(x, w_up, act, activation, coeffs=coeffs)
         return act
     if x.dtype == torch.bfloat16 and tcgen05_ok(x, w_up, act, inner):
-        ops.gemm_tcgen05(x, w_up, act, activation)
+        ops.gemm_tcgen05(x, w_up, act, activation, coeffs=coeffs)
         return act
     linear(x, w_up, act)
+    if activation == "xielu":
+        ops.xielu(act, act, coeffs)
+        return act
     (ops.relu2 if activation == "relu2" else ops.gelu_tanh)(act, act)
     return act
 
 
 def linear_xielu(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int, coeffs: torch.Tensor) -> torch.Tensor:
-    """xIELU(x W^T) with the coefficients `coeffs` (ops.xielu): the product followed by the activation kernel."""
-    act = runtime.buffer("ffn_act", (x.shape[0], inner))
-    linear(x, w_up, act)
-    ops.xielu(act, act, coeffs)
-    return act
+    """xIELU(x W^T) with the coefficients `coeffs` (ops.xielu), where linear_act puts its activations."""
+    return linear_act(x, w_up, runtime, inner, "xielu", coeffs)
 
 
 def linear_relu2(x: torch.Tensor, w_up: torch.Tensor, runtime, inner: int) -> torch.Tensor:

@@ -123,18 +123,18 @@ _SIGNATURES = {
         "dl_paged_attention_prefill_tcgen05": [_P, _I, _I, _P, _P, _L, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P,
                                                _P, _P, _I, _P]},
     "gemm_skinny": {
-        "dl_gemm_skinny": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _L, _P, _L, _P],
+        "dl_gemm_skinny": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _L, _P, _L, _P, _P],
         "dl_gemm_skinny_qkv_rope": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P, _F, _I, _I, _I, _I, _P]},
     "gemm_tcgen05": {
-        "dl_gemm_tcgen05": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P],
+        "dl_gemm_tcgen05": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P, _P],
         "dl_gemm_tcgen05_tile_coords": [_I, _I, _I, _I, _P, _P],
         "dl_gemm_tcgen05_grouped": [_P, _I, _I, _P, _I, _I, _I, _P, _I, _I, _P, _P, _I, _P, _P],
         "dl_gemm_tcgen05_qkv_rope": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P, _P, _F, _I, _I, _I, _I, _P, _P]},
     "gemm_tcgen05_cluster": {
-        "dl_gemm_tcgen05_cluster": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P],
+        "dl_gemm_tcgen05_cluster": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P, _P],
         "dl_gemm_tcgen05_cluster_qkv_rope": [_P, _I, _P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _P, _P, _F, _I, _I, _I, _I, _P, _P]},
     "gemm_stream_tcgen05": {
-        "dl_gemm_stream": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _L, _P, _P]},
+        "dl_gemm_stream": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _L, _P, _P, _P]},
     "gemm_simt": {"dl_gemm_simt": [_I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P]},
     "sampling": {
         "dl_argmax": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
@@ -1358,19 +1358,27 @@ SKINNY_MAX_ROWS = 64      # what the kernel takes
 SKINNY_FAST_ROWS = int(os.environ.get("DYNALM_SKINNY_ROWS", "16"))     # up to here the dispatchers use it (measured on B200)
 
 
-def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "store", out_scale: float = 1.0) -> None:
+def _xielu_coeffs(mode: str, coeffs: Optional[torch.Tensor]) -> None:
+    if (mode == "xielu") != (coeffs is not None) or (coeffs is not None and (coeffs.dtype != torch.float32 or coeffs.numel() != 2)):
+        raise InvalidArgument("xielu goes with its two float32 coefficients on the device")
+    _cuda(coeffs)
+
+
+def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "store", out_scale: float = 1.0,
+                coeffs: Optional[torch.Tensor] = None) -> None:
     """Weight-streaming product for at most 64 rows, bfloat16 operands; see csrc/gemm_skinny.cu.
 
     mode "store": out [M, N] bfloat16 or float32, or float32 [parts, M, N] to split K over `parts`
     blocks (the consumer adds the parts); mode "swiglu": w = [gate; up], out [M, N/2] bfloat16; mode "relu2":
-    out [M, N] bfloat16 = max(x W^T, 0)^2."""
+    out [M, N] bfloat16 = max(x W^T, 0)^2; "gelu_tanh" and "xielu" (with `coeffs`, see ops.xielu) likewise."""
+    _xielu_coeffs(mode, coeffs)
     _cuda(x, w, out)
     _rows_contiguous(x, "x")
     M, K = x.shape
     N = w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not w.is_contiguous() or w.shape[1] != K:
         raise InvalidArgument("gemm_skinny: x and w bfloat16, w [N, K] contiguous")
-    if mode in ("relu2", "gelu_tanh") and (out.dim() != 2 or out.dtype != torch.bfloat16):
+    if mode in ("relu2", "gelu_tanh", "xielu") and (out.dim() != 2 or out.dtype != torch.bfloat16):
         raise InvalidArgument("gemm_skinny: an activation needs out [M, N] bfloat16")
     if M > SKINNY_MAX_ROWS or K % 8 or x.stride(0) % 8 or x.data_ptr() % 16 or w.data_ptr() % 16:
         raise Unsupported(f"gemm_skinny: at most {SKINNY_MAX_ROWS} rows, K a multiple of 8, 16-byte aligned rows")
@@ -1387,18 +1395,22 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str =
         if out.shape != (M, N) or out.stride(1) != 1 or out.dtype not in (torch.bfloat16, torch.float32):
             raise InvalidArgument("gemm_skinny: out [M, N] bfloat16 or float32")
         code, ldy = (0 if out.dtype == torch.bfloat16 else 1), out.stride(0)
-        if mode in ("relu2", "gelu_tanh"):
-            code = 4 if mode == "relu2" else 5
+        if mode in ("relu2", "gelu_tanh", "xielu"):
+            code = {"relu2": 4, "gelu_tanh": 5, "xielu": 6}[mode]
     ahead, ahead_bytes = _take_ahead()
     _check(_fn("gemm_skinny", "dl_gemm_skinny")(_p(x), x.stride(0), _p(w), _p(out), ldy, M, N, K, code, out_scale,
-                                                 n_split, split_stride, ahead, ahead_bytes, _stream()), "gemm_skinny")
+                                                 n_split, split_stride, ahead, ahead_bytes, _p(coeffs), _stream()),
+           "gemm_skinny")
 
 
-def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "store", out_scale: float = 1.0) -> None:
+def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "store", out_scale: float = 1.0,
+                 coeffs: Optional[torch.Tensor] = None) -> None:
     """x W^T on tcgen05 tensor cores with TMA-fed operands; see csrc/gemm_tcgen05.cu.
 
     x [M, K] and w [N, K] bfloat16; out [M, N] bfloat16 or float32, or with mode "swiglu"
-    (w = [gate; up]) out [M, N/2] bfloat16, or with mode "relu2" out [M, N] bfloat16 = max(x W^T, 0)^2."""
+    (w = [gate; up]) out [M, N/2] bfloat16, or with mode "relu2" out [M, N] bfloat16 = max(x W^T, 0)^2; "gelu_tanh" and
+    "xielu" (with `coeffs`, see ops.xielu) likewise."""
+    _xielu_coeffs(mode, coeffs)
     _cuda(x, w, out)
     _rows_contiguous(x, "x")
     M, K = x.shape
@@ -1417,8 +1429,8 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str 
         if out.dtype == torch.bfloat16:
             if N % 8 or out.stride(0) % 8:
                 raise Unsupported("gemm_tcgen05: bfloat16 output needs N and its row pitch to be multiples of 8")
-            code = 4 if mode == "relu2" else (5 if mode == "gelu_tanh" else 0)
-        elif out.dtype == torch.float32 and mode not in ("relu2", "gelu_tanh"):
+            code = {"relu2": 4, "gelu_tanh": 5, "xielu": 7}.get(mode, 0)
+        elif out.dtype == torch.float32 and mode not in ("relu2", "gelu_tanh", "xielu"):
             if N % 4 or out.stride(0) % 4:
                 raise Unsupported("gemm_tcgen05: float32 output needs N and its row pitch to be multiples of 4")
             code = 1
@@ -1427,7 +1439,7 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str 
     status = _status_word(x.device)
     library, name = (("gemm_tcgen05_cluster", "dl_gemm_tcgen05_cluster") if tcgen05_pairs(M, N)
                      else ("gemm_tcgen05", "dl_gemm_tcgen05"))
-    _check(_fn(library, name)(_p(x), x.stride(0), _p(w), _p(out), out.stride(0), M, N, K, code, out_scale, _p(status),
+    _check(_fn(library, name)(_p(x), x.stride(0), _p(w), _p(out), out.stride(0), M, N, K, code, out_scale, _p(coeffs), _p(status),
                               _stream()), "gemm_tcgen05")
 
 
@@ -1445,12 +1457,14 @@ def gemm_tcgen05_tile_coords(tile: int, tiles_n: int, num_tiles: int, group_m: i
 STREAM_MAX_ROWS = 64       # what the tcgen05 weight-streaming product takes
 
 
-def gemm_stream(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "store", out_scale: float = 1.0) -> None:
+def gemm_stream(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "store", out_scale: float = 1.0,
+                coeffs: Optional[torch.Tensor] = None) -> None:
     """x W^T for up to 64 bfloat16 rows on tcgen05, built around the stream of W (csrc/gemm_stream_tcgen05.cu).
 
     out [M, N] bfloat16 or float32; float32 [parts, M, N] (contiguous): K is split over `parts` blocks and each
     leaves its partial sums; mode "swiglu" (w = [gate; up]): out [M, N/2] bfloat16; mode "relu2": out [M, N] bfloat16 =
-    max(x W^T, 0)^2."""
+    max(x W^T, 0)^2; "gelu_tanh" and "xielu" (with `coeffs`, see ops.xielu) likewise."""
+    _xielu_coeffs(mode, coeffs)
     _cuda(x, w, out)
     _rows_contiguous(x, "x")
     M, K = x.shape
@@ -1472,12 +1486,12 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str =
         if out.shape != (M, N) or out.stride(1) != 1 or out.dtype not in (torch.bfloat16, torch.float32):
             raise InvalidArgument("gemm_stream: out [M, N] bfloat16 or float32")
         code, ldy = (0 if out.dtype == torch.bfloat16 else 1), out.stride(0)
-        if mode in ("relu2", "gelu_tanh"):
+        if mode in ("relu2", "gelu_tanh", "xielu"):
             if out.dtype != torch.bfloat16:
                 raise InvalidArgument("gemm_stream: an activation needs out [M, N] bfloat16")
-            code = 3 if mode == "relu2" else 4
+            code = {"relu2": 3, "gelu_tanh": 4, "xielu": 5}[mode]
     _check(_fn("gemm_stream_tcgen05", "dl_gemm_stream")(
-        _p(x), x.stride(0), _p(w), _p(out), ldy, M, N, K, code, out_scale, n_split, split_stride,
+        _p(x), x.stride(0), _p(w), _p(out), ldy, M, N, K, code, out_scale, n_split, split_stride, _p(coeffs),
         _p(_status_word(x.device)), _stream()), "gemm_stream")
 
 
@@ -1564,7 +1578,7 @@ def gemm_argmax(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, scratch: to
         raise InvalidArgument("gemm_argmax: float32 scratch of 2 * rows * ceil(N / 16) elements, int32 out of one per row")
     ahead, ahead_bytes = _take_ahead()
     _check(_fn("gemm_skinny", "dl_gemm_skinny")(_p(x), x.stride(0), _p(w), _p(scratch), blocks, M, N, K, 3, out_scale,
-                                                 1, 0, ahead, ahead_bytes, _stream()), "gemm_skinny (argmax)")
+                                                 1, 0, ahead, ahead_bytes, None, _stream()), "gemm_skinny (argmax)")
     status = _status_word(x.device) if status_to is not None else None
     _check(_fn("sampling", "dl_argmax_of_parts")(_p(scratch), scratch.data_ptr() + 4 * M * blocks, M, blocks, _p(out),
                                                   _p(status), _p(status_to), _stream()), "argmax_of_parts")

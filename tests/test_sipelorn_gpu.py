@@ -195,6 +195,40 @@ def test_convolutions_into_shuffled_pages_keep_their_inputs(dtype, H, G, d, e, K
         assert kept is None or float(kept[0].abs().max()) == 0.0 and float(kept[:, (K - 1) * C:].abs().max()) == 0.0
 
 
+@pytest.mark.parametrize("K", [2, 3, 4])
+def test_convolutions_over_many_rows(K):
+    """A step of several hundred rows (a thread walks eight of them): three requests, one of a single token in the middle of
+    a thread's rows, all with kept inputs from before; then the inputs that are kept."""
+    from dynalm_b200.kernels import ops
+    rng = np.random.RandomState(K)
+    H, G, d, e, page = 2, 1, 32, 16, 16
+    widths = (H * d, G * d, G * e)
+    C = sum(widths)
+    taps, bias = rng.randn(C, K), rng.randn(C)
+    runs = [(2, 5, 203), (0, 9, 1), (1, 0, 131)]
+    seqs = {s: _np(_t(rng.randn(p + n, C) * 2, torch.bfloat16)) for s, p, n in runs}
+    kept = torch.zeros(3, (K - 1) * C, device=DEV)
+    for s, p, _ in runs:
+        if p:
+            kept[s] = _t(seqs[s][p - K + 1:p].ravel())
+    table = _ints(rng.permutation(60)).view(3, 20)
+    rec = G * (d + e)
+    cache = torch.zeros(60, page, rec, dtype=torch.bfloat16, device=DEV)
+    batch = Batch(runs)
+    q = torch.zeros(batch.num_tokens, H * d, dtype=torch.bfloat16, device=DEV)
+    proj = torch.cat([_t(seqs[s][p:p + n], torch.bfloat16) for s, p, n in runs])
+    ops.conv_cache(proj, widths, _t(taps.T), _t(bias), kept, batch, table, page, q, cache, rec, cache.view(-1)[G * d:], rec)
+    row = 0
+    for s, p, n in runs:
+        want = plain.convolve(seqs[s] + bias, taps, np.zeros((K - 1, C)))[0][p:]
+        _close(_np(q[row:row + n]), want[:, :H * d], 2e-2, f"queries of slot {s}")
+        pos = torch.arange(p, p + n, device=DEV)
+        got = cache[table[s].long()[pos // page], pos % page]
+        _close(_np(got), want[:, H * d:], 2e-2, f"keys and values of slot {s}")
+        _close(_np(kept[s]).reshape(K - 1, C), seqs[s][-(K - 1):], 1e-6, f"kept inputs of slot {s}")
+        row += n
+
+
 def _attention_case(rng, n, H, G, d, e, dtype, page):
     """Keys and values of one request in slot 1 as records on shuffled pages, and queries that point at one key each: the
     newest, the first of the window, the one just outside it, one far away."""
@@ -403,7 +437,7 @@ def test_xielu_behind_the_product(dtype, rows, width, inner):
     want = plain.xielu(x @ w.T, p, q)
     err = np.abs(got - want) / (1.0 + np.abs(want))
     assert err.max() <= (6e-5 if dtype == torch.float32 else 1.5e-2), err.max()
-    assert np.abs(got[:, 1] - want[:, 1]).max() <= 1e-2 * np.abs(want[:, 1]).max(), "near zero"
+    assert np.abs(got[:, 1] - want[:, 1]).max() <= 1e-2 * np.abs(want[:, 1]).max() + 5e-7, "near zero"
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
