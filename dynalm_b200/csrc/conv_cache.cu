@@ -38,13 +38,22 @@ struct ConvCacheParams {
 
 template <typename T, int V>
 __device__ __forceinline__ void cc_load(const T* p, float* v) {
-  if constexpr (V == 1) v[0] = to_float(p[0]);
-  else unpack<T>(*reinterpret_cast<const Vec16*>(p), v);
+  if constexpr (V == 1) {
+    v[0] = to_float(p[0]);
+  } else if constexpr (V * sizeof(T) == 8) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(w.x << 16); v[1] = __uint_as_float(w.x & 0xffff0000u);
+    v[2] = __uint_as_float(w.y << 16); v[3] = __uint_as_float(w.y & 0xffff0000u);
+  } else unpack<T>(*reinterpret_cast<const Vec16*>(p), v);
 }
 template <typename T, int V>
 __device__ __forceinline__ void cc_store(T* p, const float* v) {
-  if constexpr (V == 1) p[0] = from_float<T>(v[0]);
-  else *reinterpret_cast<Vec16*>(p) = pack<T>(v);
+  if constexpr (V == 1) {
+    p[0] = from_float<T>(v[0]);
+  } else if constexpr (V * sizeof(T) == 8) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  } else *reinterpret_cast<Vec16*>(p) = pack<T>(v);
 }
 
 // A thread takes V neighbouring channels of R consecutive rows.
@@ -118,12 +127,13 @@ conv_cache_kernel(const ConvCacheParams p) {
   }
 }
 
-// The same for steps of many rows: a thread walks R consecutive rows of V channels with its taps and the last K - 1 inputs
+// The same for steps of many rows, bfloat16: a thread walks R consecutive rows of V = 4 channels with its taps and the last K - 1 inputs
 // (bias included, zeros in front of a start) in registers, so that a row is read once; where a request begins among the
 // rows the inputs come from what it kept. Rows of requests of one token shift their kept inputs as above.
 template <typename T, int V, int R, int K>
 __global__ void __launch_bounds__(256)
 conv_cache_rows_kernel(const ConvCacheParams p) {
+  static_assert(V == 4 && sizeof(T) == 2, "8 bytes a row and thread");
   const int C = p.Cq + p.Ck + p.Cv, per_row = C / V;
   const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   const int row0 = static_cast<int>(idx / per_row) * R, ch = static_cast<int>(idx % per_row) * V;
@@ -140,7 +150,11 @@ conv_cache_rows_kernel(const ConvCacheParams p) {
       tk[j][i] = t4.x; tk[j][i + 1] = t4.y; tk[j][i + 2] = t4.z; tk[j][i + 3] = t4.w;
     }
   }
-  int req = -1, first_row = 0, next_first = 0, slot = 0;
+  uint2 raw[R];                                // all rows' numbers are asked for before any is used
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+    raw[r] = row0 + r < p.rows ? *reinterpret_cast<const uint2*>(col + static_cast<size_t>(row0 + r) * p.proj_stride) : make_uint2(0u, 0u);
+  int first_row = 0, next_first = 0, slot = 0;
   const int* table = nullptr;
   float* kept = nullptr;
 #pragma unroll
@@ -150,7 +164,7 @@ conv_cache_rows_kernel(const ConvCacheParams p) {
     const int pos = p.positions[row];
     bool fill = r == 0;
     if (r == 0 || row >= next_first) {           // another request begins
-      req = p.row_request[row];
+      const int req = p.row_request[row];
       first_row = p.q_start[req];
       next_first = p.q_start[req + 1];
       slot = ck_request(p.row_slot[row]);
@@ -190,7 +204,8 @@ conv_cache_rows_kernel(const ConvCacheParams p) {
       }
     }
     float u[V], acc[V];
-    cc_load<T, V>(col + static_cast<size_t>(row) * p.proj_stride, u);
+    u[0] = __uint_as_float(raw[r].x << 16); u[1] = __uint_as_float(raw[r].x & 0xffff0000u);
+    u[2] = __uint_as_float(raw[r].y << 16); u[3] = __uint_as_float(raw[r].y & 0xffff0000u);
     if (next_first - first_row == 1) {
 #pragma unroll
       for (int i = 0; i < V; ++i) kept[static_cast<size_t>(K - 2) * C + i] = u[i];
@@ -266,11 +281,11 @@ DL_EXPORT int dl_conv_cache(int dtype, const void* proj, long long proj_stride, 
                     ((reinterpret_cast<uintptr_t>(taps) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0;
   if (walk) {
     constexpr int R = 8;
-    const size_t n = static_cast<size_t>((rows + R - 1) / R) * ((Cq + Ck + Cv) / 8);
+    const size_t n = static_cast<size_t>((rows + R - 1) / R) * ((Cq + Ck + Cv) / 4);
     const unsigned blocks = static_cast<unsigned>((n + 255) / 256);
-    if (K == 2) dl::conv_cache_rows_kernel<dl::bf16, 8, R, 2><<<blocks, 256, 0, stream>>>(p);
-    else if (K == 3) dl::conv_cache_rows_kernel<dl::bf16, 8, R, 3><<<blocks, 256, 0, stream>>>(p);
-    else dl::conv_cache_rows_kernel<dl::bf16, 8, R, 4><<<blocks, 256, 0, stream>>>(p);
+    if (K == 2) dl::conv_cache_rows_kernel<dl::bf16, 4, R, 2><<<blocks, 256, 0, stream>>>(p);
+    else if (K == 3) dl::conv_cache_rows_kernel<dl::bf16, 4, R, 3><<<blocks, 256, 0, stream>>>(p);
+    else dl::conv_cache_rows_kernel<dl::bf16, 4, R, 4><<<blocks, 256, 0, stream>>>(p);
     return dl::launch_status();
   }
   if (dtype == 0) { if (wide) DL_CC(float, 4, 1); else DL_CC(float, 1, 1); }

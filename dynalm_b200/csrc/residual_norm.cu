@@ -111,7 +111,8 @@ residual_norm_kernel(const ResidualNormParams p) {
             for (int i = 0; i < V; ++i) g[i] += gb[i];
           }
 #pragma unroll
-          for (int i = 0; i < V; ++i) y[n][i] *= p.delta_scale / (1.0f + expf(-g[i]));
+          for (int i = 0; i < V; ++i)            // (16-bit results: the fast exponential and division, relative error below 1e-5)
+            y[n][i] *= sizeof(TO) == 2 ? __fdividef(p.delta_scale, 1.0f + __expf(-g[i])) : p.delta_scale / (1.0f + expf(-g[i]));
         } else {
 #pragma unroll
           for (int i = 0; i < V; ++i) y[n][i] *= p.delta_scale;
