@@ -12,6 +12,10 @@ registering it under its `kind` string; the model builder finds it through the r
     Connection     declare(spec); the weights with which a sublayer reads and writes a stream of several parts
     Block          arrangement of the four above around the residual stream
 
+A mixer or feed-forward may take the rows of another product over its input into its own first one (join_input(w) -> bool,
+joined(rows) -> the result's columns), and a mixer may ask for a state row in a run that reads another run's pages
+(reader_state_spec()).
+
 The reference has one fixed arrangement inside `Transformer::forward_batch`
 (dynalm/src/model/transformer.cpp:582-697) switched by flags of `ModelConfig`; the registries
 here replace those flags.

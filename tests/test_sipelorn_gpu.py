@@ -599,7 +599,7 @@ def test_long_decoding_keeps_its_place(name, dtype, folders):
     plan = plan_tail(reqs, 300)
     built = _built(folders[dtype][name], dtype, 320, 64, max_requests=2)
     got = run_plan_in_process(built.step_fn, plan)
-    assert built.step_fn.graph_captures > 0
+    assert built.step_fn.graph_captures > 0 or not built.step_fn.use_graphs
     compare(plan, got, logits, *TOL[dtype], "long decoding", spread=SPREAD[dtype])
     assert built.cache.free_pages == built.cache.num_pages
 
