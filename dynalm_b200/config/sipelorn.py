@@ -23,41 +23,14 @@ of experts without `groups`, no shared expert without `shared`); no default stan
 
 from __future__ import annotations
 
-import math
 from dataclasses import dataclass
 from typing import Any, Mapping, Optional, Tuple, Union
 
 from ..errors import InvalidArgument, NotFound, Unsupported
 from .reader import KeyReader
+from .yarn import YarnStretch
 
 DEFAULT_CONTEXT = 131072      # the design has no positional limit; block tables are sized for this unless told otherwise
-
-
-@dataclass(frozen=True)
-class SipelornStretch:
-    """YaRN: frequencies that turn more than `fast` times over `original` positions are kept, those that turn fewer than
-    `slow` times are divided by `factor`, a linear ramp over the pairs lies in between; the rotated vectors grow by
-    0.1 ln(factor) + 1."""
-    factor: float
-    original: float
-    fast: float
-    slow: float
-
-    def divisors(self, base: float, dims: int) -> Tuple[float, ...]:
-        """What the frequency of every pair is divided by."""
-        def pair_of(turns: float) -> float:
-            return dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
-        lo = max(math.floor(pair_of(self.fast)), 0)
-        hi = min(math.ceil(pair_of(self.slow)), dims - 1)
-        out = []
-        for i in range(dims // 2):
-            ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
-            out.append(1.0 / (ramp / self.factor + (1.0 - ramp)))
-        return tuple(out)
-
-    @property
-    def magnitude(self) -> float:
-        return 0.1 * math.log(self.factor) + 1.0
 
 
 @dataclass(frozen=True)
@@ -82,7 +55,7 @@ class SipelornLatent:
     scale: float
     rot_dims: int                # 0: no rotation
     rot_base: float
-    stretch: Optional[SipelornStretch]
+    stretch: Optional[YarnStretch]
 
 
 @dataclass(frozen=True)
@@ -144,11 +117,7 @@ def _read_latent(mr: KeyReader) -> SipelornLatent:
         dims, base = rot.int_or("dims", rot_dim), rot.float_or("base", 10000.0)
         sc = rot.object_or_none("scaling")
         if sc is not None:
-            stretch = SipelornStretch(sc.float_or("factor", 1.0), sc.float_or("original", 0.0), sc.float_or("fast", 32.0),
-                                      sc.float_or("slow", 1.0))
-            _positive(sc.where, factor=stretch.factor, original=stretch.original, fast=stretch.fast, slow=stretch.slow)
-        if stretch is not None and base == 1.0:
-            raise InvalidArgument(f"{rot.where}: 'base' 1 cannot be stretched")
+            stretch = YarnStretch.read(sc, base)
     m = SipelornLatent(mr.int("heads"), dim, rot_dim, mr.int_or("vdim", dim), mr.int("kv_rank"),
                        mr.float_or("scale", (dim + rot_dim) ** -0.5), dims, base, stretch)
     _positive(mr.where, heads=m.heads, dim=m.dim, vdim=m.vdim, kv_rank=m.kv_rank, rot_base=m.rot_base)

@@ -1,6 +1,7 @@
 // Gated activation: out[t, j] = silu(gu[t, j]) * gu[t, inner + j], gu = [gate | up] side by side.
 // silu(x) = x * sigmoid(x) (dynacore/cpu/cpu_device.cpp:117-123; CpuDevice::act_mul :1912-1929).
-// The math is fp32 whatever the storage type. Also here: the squared ReLU and the tanh form of GELU of an ungated feed-forward.
+// The math is fp32 whatever the storage type. Also here: the squared ReLU, the tanh form of GELU and xIELU of an
+// ungated feed-forward, and a gated activation with clamped halves.
 #include "common.cuh"
 
 namespace dl {
@@ -105,6 +106,37 @@ __global__ void xielu_vec_kernel(const T* __restrict__ x, T* __restrict__ out, c
   reinterpret_cast<Vec16*>(out)[i] = pack<T>(f);
 }
 
+// A gated activation whose halves are clamped: with g = min(gate + bias, limit), u = clamp(up + bias, -limit, limit),
+// g sigmoid(gate_scale g) (u + 1). bias: float32 [2 * inner] over [gate | up], or null.
+template <typename T, int V>
+__global__ void clamped_swiglu_kernel(const T* __restrict__ gu, const float* __restrict__ bias, float limit, float gate_scale,
+                                      T* __restrict__ out, int rows, int inner) {
+  const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  const int per = inner / V;
+  if (idx >= static_cast<size_t>(rows) * per) return;
+  const size_t t = idx / per;
+  const int j = static_cast<int>(idx % per) * V;
+  const T* row = gu + t * 2 * inner + j;
+  float g[V], u[V];
+  if constexpr (V > 1) {
+    unpack<T>(*reinterpret_cast<const Vec16*>(row), g);
+    unpack<T>(*reinterpret_cast<const Vec16*>(row + inner), u);
+  } else {
+    g[0] = to_float(row[0]);
+    u[0] = to_float(row[inner]);
+  }
+#pragma unroll
+  for (int k = 0; k < V; ++k) {
+    if (bias != nullptr) {
+      g[k] += bias[j + k];
+      u[k] += bias[inner + j + k];
+    }
+    g[k] = clamped_swiglu_f(g[k], u[k], limit, gate_scale);
+  }
+  if constexpr (V > 1) *reinterpret_cast<Vec16*>(out + t * inner + j) = pack<T>(g);
+  else out[t * inner + j] = from_float<T>(g[0]);
+}
+
 }  // namespace dl
 
 // out[i] = xIELU(x[i]) over n contiguous elements (out may be x); coeffs: two float32 on the device.
@@ -177,5 +209,23 @@ DL_EXPORT int dl_silu_mul(int dtype, const void* gu, void* out, int rows, int in
   if (dtype == 0) dl::silu_mul_kernel<float><<<blocks, threads, 0, stream>>>(static_cast<const float*>(gu), static_cast<float*>(out), rows, inner);
   else if (dtype == 1) dl::silu_mul_kernel<dl::bf16><<<blocks, threads, 0, stream>>>(static_cast<const dl::bf16*>(gu), static_cast<dl::bf16*>(out), rows, inner);
   else return DL_ERR_UNSUPPORTED;
+  return dl::launch_status();
+}
+
+// gu: contiguous [rows, 2 * inner] = [gate | up]; bias: float32 [2 * inner] or null; out: contiguous [rows, inner].
+DL_EXPORT int dl_clamped_swiglu(int dtype, const void* gu, const float* bias, float limit, float gate_scale, void* out, int rows,
+                                int inner, cudaStream_t stream) {
+  if (rows <= 0 || inner <= 0) return 0;
+  if ((dtype != 0 && dtype != 1) || !(limit > 0.0f)) return DL_ERR_UNSUPPORTED;
+  const int vec = dtype == 0 ? 4 : 8;
+  const bool wide = inner % vec == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const size_t n = static_cast<size_t>(rows) * (wide ? inner / vec : inner);
+  const unsigned blocks = static_cast<unsigned>((n + 255) / 256);
+#define DL_CS(T, V)                                                                                                     \
+  dl::clamped_swiglu_kernel<T, V><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gu), bias, limit, gate_scale,       \
+                                                              static_cast<T*>(out), rows, inner)
+  if (dtype == 0) { if (wide) DL_CS(float, 4); else DL_CS(float, 1); }
+  else { if (wide) DL_CS(dl::bf16, 8); else DL_CS(dl::bf16, 1); }
+#undef DL_CS
   return dl::launch_status();
 }

@@ -2,7 +2,7 @@
 //
 // It serves the true 32-bit path and every shape the faster kernels refuse. A row at position
 // `pos` of request r reads keys t in [lo, pos], lo = window > 0 ? max(0, pos - window + 1) : 0, and the keys
-// t < keep_first behind them, through block_table[r]; with `sink` the softmax's denominator holds one more term exp(0); query head h reads KV head h / (heads / kv_heads).
+// t < keep_first behind them (or, in chunks, the keys from pos / chunk * chunk on), through block_table[r]; with `sink` the softmax's denominator holds one more term exp(0); query head h reads KV head h / (heads / kv_heads).
 // With (rate, step) per head a distance bias comes off the scores: s_t = scale * q.k_t - rate_h ln(1 + step_h (pos - t)).
 //   s_t = scale * q.k_t;  out = sum_t exp(s_t - max) v_t / sum_t exp(s_t - max)
 // (dynacore/cpu/cpu_device.cpp:1309-1412,1717-1776). Keys are visited in chunks whose boundaries
@@ -25,7 +25,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* _
                                const int* __restrict__ row_request, T* __restrict__ out, int out_stride,
                                int n_heads, int n_kv_heads, int head_dim, int page_size, float scale,
                                int window, int vdim, size_t k_row, size_t v_row, int wide, int keep_first,
-                               int sink, const float* __restrict__ rate, const float* __restrict__ dstep) {
+                               int sink, const float* __restrict__ rate, const float* __restrict__ dstep, int chunk) {
   __shared__ float red[33];
   __shared__ float sq[256];                 // the query, fp32
   __shared__ float sp[ATT_CHUNK];           // scores, then probabilities, of one chunk
@@ -33,7 +33,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* _
   const int row = blockIdx.x, head = blockIdx.y;
   const int kvh = head / (n_heads / n_kv_heads);
   const int pos = positions[row];
-  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int lo = chunk > 0 ? pos / chunk * chunk : (window > 0 ? max(0, pos - window + 1) : 0);
   const int* table = block_table + static_cast<size_t>(ck_request(row_request[row])) * max_blocks;
   const int tid = threadIdx.x;
 
@@ -123,16 +123,17 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_stride, const T* _
 // column h * vdim. Keys of a token lie k_row elements apart from the next token's in k_cache (KV head j at j * head_dim),
 // values v_row elements apart in v_cache (KV head j at j * vdim): two arrays [pages, page_size, n_kv_heads, size], or
 // one array of records [k | v] given twice with two offsets. head_dim and vdim: 1 to 256; keys that all start on a
-// 16-byte boundary are read 16 bytes at a time. rate, dstep: float32 [n_heads] of the distance bias, or both null.
+// 16-byte boundary are read 16 bytes at a time. chunk > 0 (without a window): a position sees its own chunk alone. rate, dstep: float32 [n_heads] of the distance bias, or both null.
 DL_EXPORT int dl_paged_attention_generic_masked(int dtype, const void* q, int q_stride, const void* k_cache, long long k_row,
                                                 const void* v_cache, long long v_row, const int* block_table, int max_blocks,
                                                 const int* positions, const int* row_request, void* out, int out_stride,
                                                 int rows, int n_heads, int n_kv_heads, int head_dim, int vdim, int page_size,
                                                 float scale, int window, int keep_first, int sink, const float* rate,
-                                                const float* dstep, cudaStream_t stream) {
+                                                const float* dstep, int chunk, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (head_dim > 256 || head_dim <= 0 || vdim <= 0 || vdim > 256 || n_kv_heads <= 0 || n_heads % n_kv_heads != 0 ||
-      page_size <= 0 || n_heads > 65535 || (dtype != 0 && dtype != 1) || keep_first < 0 || (rate != nullptr) != (dstep != nullptr))
+      page_size <= 0 || n_heads > 65535 || (dtype != 0 && dtype != 1) || keep_first < 0 || (rate != nullptr) != (dstep != nullptr) ||
+      chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0)))
     return DL_ERR_UNSUPPORTED;
   const int per = dtype == 0 ? 4 : 8;           // numbers in 16 bytes
   const int wide = head_dim % per == 0 && k_row % per == 0 && (reinterpret_cast<uintptr_t>(k_cache) & 15) == 0;
@@ -142,7 +143,7 @@ DL_EXPORT int dl_paged_attention_generic_masked(int dtype, const void* q, int q_
       static_cast<const T*>(q), q_stride, static_cast<const T*>(k_cache), static_cast<const T*>(v_cache),     \
       block_table, max_blocks, positions, row_request, static_cast<T*>(out), out_stride, n_heads, n_kv_heads, \
       head_dim, page_size, scale, window, vdim, static_cast<size_t>(k_row), static_cast<size_t>(v_row), wide,    \
-      keep_first, sink, rate, dstep)
+      keep_first, sink, rate, dstep, chunk)
   if (dtype == 0) DL_LAUNCH(float);
   else if (dtype == 1) DL_LAUNCH(dl::bf16);
   else return DL_ERR_UNSUPPORTED;
@@ -158,7 +159,7 @@ DL_EXPORT int dl_paged_attention_generic_kv(int dtype, const void* q, int q_stri
                                             float scale, int window, cudaStream_t stream) {
   return dl_paged_attention_generic_masked(dtype, q, q_stride, k_cache, k_row, v_cache, v_row, block_table, max_blocks,
                                            positions, row_request, out, out_stride, rows, n_heads, n_kv_heads, head_dim, vdim,
-                                           page_size, scale, window, 0, 0, nullptr, nullptr, stream);
+                                           page_size, scale, window, 0, 0, nullptr, nullptr, 0, stream);
 }
 
 // The same for keys and values of one size in two arrays [pages, page_size, n_kv_heads, head_dim].

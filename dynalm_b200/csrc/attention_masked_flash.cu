@@ -9,6 +9,7 @@
 //     the next token's and its values v_row, so the cache may be two arrays or one array of records [k | v];
 //   * a row at position p sees key j <= p if p - j < window (window 0: all) or j < keep_first: the key tiles that hold
 //     kept tokens are walked first, then the tiles of the window;
+//   * with a chunk (and no window) a row sees the keys from p / chunk * chunk on instead;
 //   * with `sink` the denominator of a row's softmax holds one more term exp(0), which carries no value;
 //   * with (rate, step) per head a distance bias rate_h ln(1 + step_h (p - j)) comes off every score; its values for the
 //     127 distances of a 64 x 64 tile of rows and keys are worked out once per tile, in shared memory;
@@ -75,7 +76,7 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                     const bf16* __restrict__ v_cache, size_t v_row, const int* __restrict__ block_table, int max_blocks,
                     const int4* __restrict__ tiles, bf16* __restrict__ out, int out_stride, int n_heads, int n_kv_heads,
                     int page_shift, float scale_log2, int window, int keep_first, int sink, int grp, float* __restrict__ partial,
-                    const float* __restrict__ rate, const float* __restrict__ dstep, const bf16* __restrict__ gate, int gate_stride) {
+                    const float* __restrict__ rate, const float* __restrict__ dstep, const bf16* __restrict__ gate, int gate_stride, int chunk) {
   __shared__ float bias_tab[2][2 * MF_BN];
   constexpr int SUB = MF_TILE / MF_BM;    // blocks per query tile
   constexpr int LDK = KD + 8;             // row strides in elements: 16 bytes of padding keep ldmatrix conflict-free
@@ -104,7 +105,8 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
   const bool warp_live = warp * 16 < nrows;
 
   const int pos_last = grp > 0 ? pos0 : pos0 + nrows - 1;
-  const int lo_tile = window > 0 ? max(0, pos0 - window + 1) : 0;     // the first key of the window any row of the tile reads
+  auto first_key = [&](int p) { return chunk > 0 ? p / chunk * chunk : (window > 0 ? max(0, p - window + 1) : 0); };
+  const int lo_tile = first_key(pos0);     // the first key of the window any row of the tile reads
   const int j_begin = lo_tile / MF_BN, j_end = pos_last / MF_BN;
   // key tiles in front of the window's that hold kept tokens: 0 .. n_kept - 1
   const int kept = lo_tile > 0 ? min(keep_first, lo_tile) : 0;
@@ -150,7 +152,7 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
     m_run[h] = -INFINITY;
     l_run[h] = 0.0f;
     pos_r[h] = grp > 0 ? pos0 : pos0 + warp * 16 + g + h * 8;
-    lo_r[h] = window > 0 ? max(0, pos_r[h] - window + 1) : 0;
+    lo_r[h] = first_key(pos_r[h]);
   }
   uint32_t qf[KS][4];
   // with a distance bias the scores are scaled before it comes off (base-2 units), else on the way into the exponential
@@ -219,7 +221,7 @@ masked_flash_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
         }
       }
       const bool edge = it < n_kept || key0 + MF_BN - 1 > (grp > 0 ? pos0 : pos0 + warp * 16) ||
-                        (window > 0 && key0 < max(lo_r[0], lo_r[1]));
+                        key0 < max(lo_r[0], lo_r[1]);
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int i = 0; i < MF_BN / 8; ++i) {
@@ -366,7 +368,7 @@ int launch_masked_flash(const void* q, int q_stride, const void* kc, long long k
                         const int* block_table, int max_blocks, const int* tiles, int n_tiles, void* out, int out_stride,
                         int n_heads, int n_kv_heads, int page_shift, float scale, int window, int keep_first, int sink,
                         int grp, int parts, float* partial, int rows, const float* rate, const float* dstep, const void* gate,
-                        int gate_stride, cudaStream_t stream) {
+                        int gate_stride, int chunk, cudaStream_t stream) {
   constexpr size_t smem = (static_cast<size_t>(MF_BM + 2 * MF_BN) * (KD + 8) + static_cast<size_t>(2 * MF_BN) * (VD + 8)) * sizeof(bf16);
   static bool configured = false;
   if (!configured) {
@@ -380,7 +382,7 @@ int launch_masked_flash(const void* q, int q_stride, const void* kc, long long k
       static_cast<const bf16*>(q), q_stride, static_cast<const bf16*>(kc), static_cast<size_t>(k_row),
       static_cast<const bf16*>(vc), static_cast<size_t>(v_row), block_table, max_blocks, reinterpret_cast<const int4*>(tiles),
       static_cast<bf16*>(out), out_stride, n_heads, n_kv_heads, page_shift, scale * 1.4426950408889634f, window, keep_first,
-      sink, grp, parts > 1 ? partial : nullptr, rate, dstep, static_cast<const bf16*>(gate), gate_stride);
+      sink, grp, parts > 1 ? partial : nullptr, rate, dstep, static_cast<const bf16*>(gate), gate_stride, chunk);
   if (parts > 1) {
     dim3 mgrid(rows, n_heads);
     masked_flash_merge_kernel<<<mgrid, VD < 64 ? 32 : 64, 0, stream>>>(partial, parts, VD, n_heads, sink, static_cast<bf16*>(out),
@@ -403,7 +405,7 @@ DL_EXPORT int dl_masked_flash_attention(const void* q, int q_stride, const void*
                                         void* out, int out_stride, int n_heads, int n_kv_heads, int key_dim, int value_dim,
                                         int page_size, float scale, int window, int keep_first, int sink, int one_token_tiles,
                                         int parts, float* partial, const float* rate, const float* dstep, const void* gate,
-                                        int gate_stride, cudaStream_t stream) {
+                                        int gate_stride, int chunk, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
   int page_shift = 0;
   while ((1 << page_shift) < page_size) ++page_shift;
@@ -411,7 +413,7 @@ DL_EXPORT int dl_masked_flash_attention(const void* q, int q_stride, const void*
       (out_stride & 1) || !(scale > 0.0f) || (k_row & 7) || (v_row & 7) || window < 0 || keep_first < 0 ||
       (reinterpret_cast<uintptr_t>(k_cache) & 15) || (reinterpret_cast<uintptr_t>(v_cache) & 15))
     return DL_ERR_UNSUPPORTED;
-  if ((rate != nullptr) != (dstep != nullptr)) return DL_ERR_UNSUPPORTED;
+  if ((rate != nullptr) != (dstep != nullptr) || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return DL_ERR_UNSUPPORTED;
   // every tile one token (the caller says so) and heads that share keys: the heads of a KV head are the rows of a tile
   const int group = n_heads / n_kv_heads;
   const int grp = (one_token_tiles && group > 1 && group <= dl::MF_BM) ? group : 0;
@@ -422,7 +424,7 @@ DL_EXPORT int dl_masked_flash_attention(const void* q, int q_stride, const void*
   if (key_dim == K && value_dim == V)                                                                                   \
     return dl::launch_masked_flash<K, V>(q, q_stride, k_cache, k_row, v_cache, v_row, block_table, max_blocks, tiles,   \
                                          n_tiles, out, out_stride, n_heads, n_kv_heads, page_shift, scale, window,      \
-                                         keep_first, sink, grp, parts, partial, n_tiles, rate, dstep, gate, gate_stride, stream)
+                                         keep_first, sink, grp, parts, partial, n_tiles, rate, dstep, gate, gate_stride, chunk, stream)
   DL_CASE(16, 16); DL_CASE(32, 32); DL_CASE(48, 48); DL_CASE(64, 64); DL_CASE(80, 80); DL_CASE(96, 96); DL_CASE(112, 112);
   DL_CASE(128, 128);
   DL_CASE(32, 16); DL_CASE(48, 32); DL_CASE(64, 32); DL_CASE(96, 48); DL_CASE(96, 64); DL_CASE(128, 64); DL_CASE(64, 128);

@@ -141,6 +141,13 @@ __device__ __forceinline__ float xielu_bf16(float z, float c0, float c1) {
   return z > 0.0f ? pos : neg;
 }
 
+// A gated activation with clamped halves: min(g, limit) sigmoid(scale min(g, limit)) (clamp(u, -limit, limit) + 1).
+__device__ __forceinline__ float clamped_swiglu_f(float g, float u, float limit, float scale) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + expf(-scale * g)) * (u + 1.0f);
+}
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // Programmatic dependent launch. A kernel launched with the attribute may begin while the kernel before it on

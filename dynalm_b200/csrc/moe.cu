@@ -1,7 +1,7 @@
 // Mixture of experts: routing, the grouping of (token, expert) pairs by expert, the experts' products over those
 // groups, and the weighted sum of a token's experts.
 //
-//   dl_moe_route     scores = softmax(router logits) over all experts, or sigmoid of each, float32; choice scores = scores
+//   dl_moe_route     scores = softmax(router logits, + a bias per expert where there is one) over all experts, or sigmoid of each, float32; choice scores = scores
 //                    (+ a correction per expert). Experts form `groups` equal groups of neighbours; a group's score is
 //                    its largest choice score, or the sum of its two largest, and only experts of the `keep` best groups
 //                    can be chosen. The `top` allowed experts with the largest choice scores are chosen (equal ones: the
@@ -41,7 +41,7 @@ __device__ __forceinline__ int moe_warp_best(float v, int index) {      // the i
 
 __global__ void __launch_bounds__(MOE_ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ logits, int stride, int tokens, int E, int top, int groups, int keep,
-                 const float* __restrict__ correction, int sigmoid_scores, int group_top2, int renormalize, float scale,
+                 const float* __restrict__ bias, const float* __restrict__ correction, int sigmoid_scores, int group_top2, int renormalize, float scale,
                  int* __restrict__ ids, float* __restrict__ weights) {
   __shared__ float choice_s[MOE_ROUTE_WARPS][MOE_MAX_EXPERTS];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -53,7 +53,7 @@ moe_route_kernel(const float* __restrict__ logits, int stride, int tokens, int E
 #pragma unroll
   for (int k = 0; k < MOE_PER_LANE; ++k) {
     const int i = lane + 32 * k;
-    s[k] = i < E ? z[i] : -INFINITY;
+    s[k] = i < E ? z[i] + (bias != nullptr ? bias[i] : 0.0f) : -INFINITY;
     m = fmaxf(m, s[k]);
   }
   if (sigmoid_scores) {
@@ -447,16 +447,16 @@ __global__ void moe_combine_kernel(const float* __restrict__ c, int width, const
 
 }  // namespace dl
 
-// correction: float32 [E] or null; sigmoid_scores 0: softmax over all experts; group_top2 0: a group's largest choice score.
+// bias (joins the logits), correction (joins the scores for the choice alone): float32 [E] or null; sigmoid_scores 0: softmax over all experts; group_top2 0: a group's largest choice score.
 DL_EXPORT int dl_moe_route(const float* logits, int stride, int tokens, int E, int top, int groups, int keep,
-                           const float* correction, int sigmoid_scores, int group_top2, int renormalize, float scale, int* ids,
+                           const float* bias, const float* correction, int sigmoid_scores, int group_top2, int renormalize, float scale, int* ids,
                            float* weights, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (E <= 0 || E > dl::MOE_MAX_EXPERTS || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
       top > keep * (E / groups))
     return DL_ERR_UNSUPPORTED;
   constexpr int WARPS = dl::MOE_ROUTE_WARPS;
-  dl::moe_route_kernel<<<(tokens + WARPS - 1) / WARPS, WARPS * 32, 0, stream>>>(logits, stride, tokens, E, top, groups, keep, correction,
+  dl::moe_route_kernel<<<(tokens + WARPS - 1) / WARPS, WARPS * 32, 0, stream>>>(logits, stride, tokens, E, top, groups, keep, bias, correction,
                                                                                sigmoid_scores, group_top2, renormalize, scale, ids, weights);
   return dl::launch_status();
 }

@@ -157,6 +157,147 @@ qk_rot_head_norm_kernel(T* __restrict__ proj, int stride, const float* __restric
   }
 }
 
+// The third order: every head of q and k normed by itself with a weight that all heads share, x / sqrt(mean(x^2) + eps) *
+// w[i], then turned: numbers i and i + rot / 2 of its first `rot` numbers by position * freq[i], cos and sin times mag. The
+// angle is formed and brought into half a turn around zero in double precision, so it is exact to float32 at any position.
+// The values are columns of their own behind k, or (values_are_keys) the keys as they were projected.
+__device__ __forceinline__ void qk_angle(int pos, double freq, float mag, float& cs, float& sn) {
+  constexpr double TURN = 6.283185307179586476925286766559, INV_TURN = 0.15915494309189533576888376337251;
+  const double a = static_cast<double>(pos) * freq;
+  float s, c;
+  sincosf(static_cast<float>(fma(-rint(a * INV_TURN), TURN, a)), &s, &c);
+  cs = c * mag;
+  sn = s * mag;
+}
+
+// One block per row; the row's angles are worked out once, in shared memory. A head is TG neighbouring lanes with 16 bytes
+// each (the lanes past its end idle), TG a power of two up to 32, and half of `rot` a multiple of a lane's numbers.
+template <typename T>
+__global__ void __launch_bounds__(512)
+qk_norm_turn_vec_kernel(T* __restrict__ proj, int stride, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                        const double* __restrict__ freq, int rot, float mag, const int* __restrict__ positions,
+                        const int* __restrict__ row_slot, const int* __restrict__ block_table, int max_blocks,
+                        T* __restrict__ k_cache, size_t k_row, T* __restrict__ v_cache, size_t v_row, int H, int G, int d, int e,
+                        int page_size, int values_are_keys, int TG) {
+  constexpr int V = PerVec<T>::n;
+  constexpr int MAX_PAIRS = 128;
+  __shared__ float cos_s[MAX_PAIRS], sin_s[MAX_PAIRS];
+  const int row = blockIdx.x, tid = threadIdx.x;
+  const int pos = positions[row];
+  const int* table = block_table + static_cast<size_t>(ck_request(row_slot[row])) * max_blocks;
+  const int page = ck_page_store(table, pos / page_size, max_blocks);
+  const size_t slot = static_cast<size_t>(page < 0 ? 0 : page) * page_size + pos % page_size;
+  T* base = proj + static_cast<size_t>(row) * stride;
+  const int half = rot / 2;
+  for (int i = tid; i < half; i += blockDim.x) qk_angle(pos, freq[i], mag, cos_s[i], sin_s[i]);
+  __syncthreads();
+  const int per_head = d / V, half_lanes = half / V, own_values = values_are_keys ? 0 : G * e / V;
+  const int turned = (H + G) * TG, total = turned + own_values;
+  // whole warps walk the heads, so that the shuffles below find their lanes
+  for (int i = tid; i < (total + 31) / 32 * 32; i += blockDim.x) {
+    const int head = i / TG, l = i % TG;
+    const bool is_head = i < turned;
+    const bool live = is_head && l < per_head;
+    Vec16 raw;
+    raw.raw = make_uint4(0u, 0u, 0u, 0u);
+    T* src = base + static_cast<size_t>(head) * d + l * V;
+    if (live) raw = *reinterpret_cast<const Vec16*>(src);
+    float x[V];
+    unpack<T>(raw, x);
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss = fmaf(x[j], x[j], ss);
+    for (int o = TG >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float r = 1.0f / sqrtf(ss / static_cast<float>(d) + eps);
+    const float* w = head < H ? wq : wk;
+    if (live) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= r * w[l * V + j];
+    }
+    const bool first = l < half_lanes, pair = l < 2 * half_lanes;
+    const int lane = tid & 31, partner = pair ? (first ? lane + half_lanes : lane - half_lanes) : lane;
+    const int a0 = pair ? (first ? l : l - half_lanes) * V : 0;
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float y = __shfl_sync(0xffffffffu, x[j], partner);
+      if (pair && live) {
+        const float c = cos_s[a0 + j], s = sin_s[a0 + j];
+        x[j] = first ? x[j] * c - y * s : x[j] * c + y * s;
+      }
+    }
+    if (live && head < H) {
+      *reinterpret_cast<Vec16*>(src) = pack<T>(x);
+    } else if (live && page >= 0) {
+      const size_t at = static_cast<size_t>(head - H) * d + l * V;
+      *reinterpret_cast<Vec16*>(k_cache + slot * k_row + at) = pack<T>(x);
+      if (values_are_keys) *reinterpret_cast<Vec16*>(v_cache + slot * v_row + at) = raw;
+    } else if (!is_head && i < total && page >= 0) {
+      const size_t at = static_cast<size_t>(i - turned) * V;
+      *reinterpret_cast<Vec16*>(v_cache + slot * v_row + at) = *reinterpret_cast<const Vec16*>(base + static_cast<size_t>(H + G) * d + at);
+    }
+  }
+}
+
+// Any size up to 256: one warp per unit, a unit being a query head, a key head or the values of a KV head.
+template <typename T>
+__global__ void __launch_bounds__(256)
+qk_norm_turn_kernel(T* __restrict__ proj, int stride, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                    const double* __restrict__ freq, int rot, float mag, const int* __restrict__ positions,
+                    const int* __restrict__ row_slot, const int* __restrict__ block_table, int max_blocks,
+                    T* __restrict__ k_cache, size_t k_row, T* __restrict__ v_cache, size_t v_row, int rows, int H, int G, int d,
+                    int e, int page_size, int values_are_keys) {
+  constexpr int PER = 8;
+  const int units = H + 2 * G;
+  const long long unit = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (unit >= static_cast<long long>(rows) * units) return;
+  const int row = static_cast<int>(unit / units), u = static_cast<int>(unit % units);
+  const int pos = positions[row];
+  const int* table = block_table + static_cast<size_t>(ck_request(row_slot[row])) * max_blocks;
+  T* base = proj + static_cast<size_t>(row) * stride;
+  size_t slot = 0;
+  int page = 0;
+  if (u >= H) {
+    page = ck_page_store(table, pos / page_size, max_blocks);
+    if (page < 0) return;
+    slot = static_cast<size_t>(page) * page_size + pos % page_size;
+  }
+  if (u >= H + G) {                                         // values: a copy into the token's place
+    const int j = u - H - G;
+    const T* v = base + (values_are_keys ? (H + j) * d : (H + G) * d + j * e);
+    T* dst = v_cache + slot * v_row + static_cast<size_t>(j) * e;
+    for (int i = lane; i < e; i += 32) dst[i] = v[i];
+    return;
+  }
+  T* src = base + static_cast<size_t>(u) * d;
+  const float* w = u < H ? wq : wk;
+  const int half = rot / 2;
+  float x[PER], xp[PER], ss = 0.0f;
+#pragma unroll
+  for (int j = 0; j < PER; ++j) {
+    const int i = lane + 32 * j;
+    x[j] = i < d ? to_float(src[i]) : 0.0f;
+    xp[j] = i < rot ? to_float(src[i < half ? i + half : i - half]) : 0.0f;
+    ss = fmaf(x[j], x[j], ss);
+  }
+  const float r = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(d) + eps);      // (the shuffles also order reads before writes)
+  T* dst = u < H ? src : k_cache + slot * k_row + static_cast<size_t>(u - H) * d;
+#pragma unroll
+  for (int j = 0; j < PER; ++j) {
+    const int i = lane + 32 * j;
+    if (i >= d) continue;
+    float v = x[j] * r * w[i];
+    if (i < rot) {
+      const bool first = i < half;
+      const float y = xp[j] * r * w[first ? i + half : i - half];
+      float c, s;
+      qk_angle(pos, freq[first ? i : i - half], mag, c, s);
+      v = first ? v * c - y * s : v * c + y * s;
+    }
+    dst[i] = from_float<T>(v);
+  }
+}
+
 }  // namespace dl
 
 DL_EXPORT int dl_qk_proj_norm_cache(int dtype, void* proj, int stride, const float* wq, const float* wk, float eps, int do_norm,
@@ -203,6 +344,50 @@ DL_EXPORT int dl_qk_rot_head_norm_cache(int dtype, void* proj, int stride, const
   if (dtype == 0) DL_QK(float);
   else if (dtype == 1) DL_QK(dl::bf16);
   else return DL_ERR_UNSUPPORTED;
+#undef DL_QK
+  return dl::launch_status();
+}
+
+// Rows [q: H*d | k: G*d | v: G*e | ...] (without the values when they are the keys): every head of q and k normed by itself
+// (wq, wk: float32 [d]), then turned (rot numbers, pairs i and i + rot / 2, freq: float64 [rot / 2]); q in
+// place, k and v into the pages. d and e at most 256.
+DL_EXPORT int dl_qk_norm_turn_cache(int dtype, void* proj, int stride, const float* wq, const float* wk, float eps,
+                                    const double* freq, int rot, float mag, const int* positions, const int* row_slot,
+                                    const int* block_table, int max_blocks, void* k_cache, long long k_row, void* v_cache,
+                                    long long v_row, int rows, int H, int G, int d, int e, int page_size, int values_are_keys,
+                                    cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (H <= 0 || G <= 0 || d <= 0 || d > 256 || e <= 0 || e > 256 || rot < 0 || rot > d || (rot & 1) || page_size <= 0 ||
+      wq == nullptr || wk == nullptr || (rot > 0 && freq == nullptr) || (values_are_keys && d != e) || (dtype != 0 && dtype != 1))
+    return DL_ERR_UNSUPPORTED;
+  const int V = dtype == 0 ? 4 : 8;
+  int TG = 1;
+  while (TG * V < d) TG *= 2;
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
+  if (d % V == 0 && e % V == 0 && TG <= 32 && (rot / 2) % V == 0 && stride % V == 0 && k_row % V == 0 && v_row % V == 0 && (bases & 15) == 0) {
+    const int lanes = (H + G) * TG + (values_are_keys ? 0 : G * e / V);
+    const int threads = lanes <= 64 ? 64 : lanes <= 128 ? 128 : lanes <= 256 ? 256 : 512;
+#define DL_QK(T)                                                                                                            \
+  dl::qk_norm_turn_vec_kernel<T><<<rows, threads, 0, stream>>>(static_cast<T*>(proj), stride, wq, wk, eps, freq, rot, mag,  \
+                                                               positions, row_slot, block_table, max_blocks,                \
+                                                               static_cast<T*>(k_cache), static_cast<size_t>(k_row),        \
+                                                               static_cast<T*>(v_cache), static_cast<size_t>(v_row), H, G,  \
+                                                               d, e, page_size, values_are_keys, TG)
+    if (dtype == 0) DL_QK(float);
+    else DL_QK(dl::bf16);
+#undef DL_QK
+    return dl::launch_status();
+  }
+  const long long units = static_cast<long long>(rows) * (H + 2 * G);
+  const unsigned blocks = static_cast<unsigned>((units + 7) / 8);
+#define DL_QK(T)                                                                                                            \
+  dl::qk_norm_turn_kernel<T><<<blocks, 256, 0, stream>>>(static_cast<T*>(proj), stride, wq, wk, eps, freq, rot, mag,        \
+                                                         positions, row_slot, block_table, max_blocks,                      \
+                                                         static_cast<T*>(k_cache), static_cast<size_t>(k_row),              \
+                                                         static_cast<T*>(v_cache), static_cast<size_t>(v_row), rows, H, G,  \
+                                                         d, e, page_size, values_are_keys)
+  if (dtype == 0) DL_QK(float);
+  else DL_QK(dl::bf16);
 #undef DL_QK
   return dl::launch_status();
 }

@@ -154,6 +154,38 @@ def linear_partial(x: torch.Tensor, w: torch.Tensor, runtime, name: str) -> torc
     return linear(x, w, out)
 
 
+def linear_short(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out = x W^T for a short K (an inner vector of a few dozen or hundred numbers, x often a slice of wider rows): there is
+    no K to split, so this package's products take every row count and however few tiles, float32 results included."""
+    ok = (x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and x.stride(1) == 1 and x.stride(0) % 8 == 0
+          and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and w.is_contiguous() and w.shape[0] % 8 == 0
+          and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)
+    if not ok:
+        return linear(x, w, out)
+    if x.shape[0] <= ops.SKINNY_MAX_ROWS:
+        ops.gemm_skinny(x, w, out, "store", 1.0)
+    else:
+        ops.gemm_tcgen05(x, w, out, "store", 1.0)
+    return out
+
+
+def linear_partial_biased(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], runtime, name: str) -> torch.Tensor:
+    """linear_partial plus a float32 bias [N]. With 16-bit operands the product leaves float32 sums (whole, or split-K
+    partial sums) and the bias joins those."""
+    if bias is None:
+        return linear_partial(x, w, runtime, name)
+    M, N = x.shape[0], w.shape[0]
+    if x.dtype == torch.float32:
+        return linear(x, w, runtime.buffer(name, (M, N)), bias)
+    if use_stream(x, w) or skinny_ok(x, w):
+        out = linear_partial(x, w, runtime, name)
+        ops.add_bias(out[0] if out.dim() == 3 else out, bias)
+        return out
+    out = linear(x, w, runtime.buffer(name + "_wide", (M, N), torch.float32))
+    ops.add_bias(out, bias)
+    return out
+
+
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, runtime, inner: int) -> torch.Tensor:
     """silu(x Wg^T) * (x Wu^T) with w_gate_up = [Wg; Wu]: fused in the product's epilogue for few
     bfloat16 rows, else the product followed by the activation kernel."""
@@ -171,6 +203,17 @@ def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, runtime, inner: int)
     gate_up = runtime.buffer("ffn_gate_up", (rows, 2 * inner))
     linear(x, w_gate_up, gate_up)
     ops.silu_mul(gate_up, act)
+    return act
+
+
+def linear_clamped_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, bias: Optional[torch.Tensor], limit: float, gate_scale: float,
+                          runtime, inner: int) -> torch.Tensor:
+    """With [g | u] = x [Wg; Wu]^T + bias: min(g, limit) sigmoid(gate_scale min(g, limit)) (clamp(u, -limit, limit) + 1)."""
+    rows = x.shape[0]
+    act = runtime.buffer("ffn_act", (rows, inner))
+    gate_up = runtime.buffer("ffn_gate_up", (rows, 2 * inner))
+    linear(x, w_gate_up, gate_up)
+    ops.clamped_swiglu(gate_up, bias, limit, gate_scale, act)
     return act
 
 

@@ -35,7 +35,8 @@ _SIGNATURES = {
         "dl_rmsnorm_pair": [_I, _P, _P, _I, _I, _L, _P, _I, _I, _L, _P, _P, _F, _P, _P, _P, _I, _I, _I, _P],
     },
     "activation": {"dl_silu_mul": [_I, _P, _P, _I, _I, _P], "dl_relu2": [_I, _P, _P, _L, _P],
-                   "dl_gelu_tanh": [_I, _P, _P, _L, _P], "dl_xielu": [_I, _P, _P, _P, _L, _P]},
+                   "dl_gelu_tanh": [_I, _P, _P, _L, _P], "dl_xielu": [_I, _P, _P, _P, _L, _P],
+                   "dl_clamped_swiglu": [_I, _P, _P, _F, _F, _P, _I, _I, _P]},
     "norm_after_sum": {
         "dl_norm_after_sum": [_I, _I, _P, _P, _I, _L, _P, _F, _P, _F, _P, _I, _I, _P],
         "dl_cast_rows": [_I, _P, _P, _L, _P]},
@@ -75,11 +76,13 @@ _SIGNATURES = {
         "dl_paged_attention_generic_kv": [_I, _P, _I, _P, _L, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I,
                                           _P],
         "dl_paged_attention_generic_masked": [_I, _P, _I, _P, _L, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F,
-                                              _I, _I, _I, _P, _P, _P]},
+                                              _I, _I, _I, _P, _P, _I, _P]},
     "delta_rule": {
-        "dl_delta_rule": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
-        "dl_delta_rule_step": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
-        "dl_head_norm_gate": [_I, _P, _P, _I, _I, _P, _F, _P, _I, _I, _I, _P]},
+        "dl_delta_rule": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+        "dl_delta_rule_step": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I,
+                               _P],
+        "dl_delta_decay": [_P, _I, _P, _P, _I, _I, _I, _P],
+        "dl_head_norm_gate": [_I, _I, _P, _P, _I, _I, _P, _F, _I, _P, _I, _I, _I, _P]},
     "rglru": {
         "dl_rglru_gates": [_I, _P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P],
         "dl_rglru_scan": [_I, _P, _P, _P, _I, _I, _P, _P, _L, _P, _P, _P, _I, _I, _I, _P]},
@@ -87,10 +90,12 @@ _SIGNATURES = {
         "dl_qk_proj_norm_cache": [_I, _P, _I, _P, _P, _F, _I, _P, _I, _F, _P, _P, _P, _I, _P, _L, _P, _L, _I, _I, _I, _I,
                                   _I, _I, _P],
         "dl_qk_rot_head_norm_cache": [_I, _P, _I, _P, _P, _I, _I, _I, _F, _P, _P, _P, _I, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I,
-                                      _P]},
+                                      _P],
+        "dl_qk_norm_turn_cache": [_I, _P, _I, _P, _P, _F, _P, _I, _F, _P, _P, _P, _I, _P, _L, _P, _L, _I, _I, _I, _I, _I, _I, _I,
+                                  _P]},
     "attention_masked_flash": {
         "dl_masked_flash_attention": [_P, _I, _P, _L, _P, _L, _P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _I, _I, _P,
-                                      _P, _P, _P, _I, _P]},
+                                      _P, _P, _P, _I, _I, _P]},
     "layer_norm": {
         "dl_stream_layer_norm": [_I, _I, _P, _I, _I, _P, _P, _I, _L, _F, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _P],
         "dl_stream_sum": [_I, _P, _I, _I, _P, _I, _L, _F, _P, _P, _P, _I, _P]},
@@ -98,7 +103,7 @@ _SIGNATURES = {
         "dl_gla_decay": [_P, _I, _I, _I, _P, _F, _P],
         "dl_gla_scan": [_I, _P, _I, _I, _I, _I, _P, _I, _F, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P]},
     "moe": {
-        "dl_moe_route": [_P, _I, _I, _I, _I, _I, _I, _P, _I, _I, _I, _F, _P, _P, _P],
+        "dl_moe_route": [_P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _I, _I, _F, _P, _P, _P],
         "dl_moe_group": [_P, _I, _I, _P, _P, _P, _P, _I, _P],
         "dl_moe_linear": [_I, _I, _P, _I, _P, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
         "dl_moe_gather": [_P, _I, _P, _I, _P, _I, _I, _P],
@@ -111,7 +116,8 @@ _SIGNATURES = {
         "dl_softcap": [_P, _L, _F, _P],
         "dl_add_bias": [_I, _P, _L, _P, _I, _I, _P]},
     "norm_sandwich": {
-        "dl_norm_add_norm": [_I, _I, _P, _P, _I, _L, _P, _F, _P, _F, _P, _I, _I, _P]},
+        "dl_norm_add_norm": [_I, _I, _P, _P, _I, _L, _P, _F, _P, _F, _P, _I, _I, _P],
+        "dl_normed_sum": [_I, _P, _I, _L, _P, _F, _I, _P, _I, _L, _P, _F, _F, _P, _I, _I, _P]},
     "attention_decode": {
         "dl_paged_attention_decode": [_I, _P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
         "dl_paged_attention_decode_planned": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P,
@@ -1697,46 +1703,60 @@ def short_conv(proj: torch.Tensor, col0: int, channels: int, taps_t: torch.Tenso
 def delta_rule(u: torch.Tensor, q_col: int, k_col: int, v_col: int, proj: torch.Tensor, b_col: int, a_col: int,
                a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor,
                state_slots: torch.Tensor, out: torch.Tensor, requests: int, heads: int, kv_heads: int, dim: int,
-               vdim: int) -> None:
+               vdim: int, channel_decay: Optional[torch.Tensor] = None) -> None:
     """The gated delta rule of every head over every request's rows of the step, from and into state[slot, :H*d*e]
     ([H, d, e]). u: rows with q (G*d) at q_col, k (G*d) at k_col, v (H*e) at v_col, after convolution and silu; proj:
     rows with the raw write strengths (H) at b_col and the raw step sizes (H) at a_col; out: float32 [rows, H*e].
-    See csrc/delta_rule.cu."""
-    _cuda(u, proj, a_log, dt_bias, state, q_start, state_slots, out)
+    channel_decay (float32 [rows, >= H*d], overwritten): the raw numbers of a decay per head and key channel instead of the
+    raw step sizes; dt_bias is then [H*d]. See csrc/delta_rule.cu."""
+    _cuda(u, proj, a_log, dt_bias, state, q_start, state_slots, out, channel_decay)
     _rows_contiguous(u, "u")
     _rows_contiguous(proj, "proj")
+    by_channel = channel_decay is not None
     if u.dtype != proj.dtype or max(q_col, k_col) + kv_heads * dim > u.shape[1] or v_col + heads * vdim > u.shape[1] \
-            or max(b_col, a_col) + heads > proj.shape[1]:
+            or max(b_col, 0 if by_channel else a_col) + heads > proj.shape[1]:
         raise InvalidArgument("delta_rule: the columns lie outside u or proj, or their dtypes differ")
-    if any(t.dtype != torch.float32 or t.numel() != heads for t in (a_log, dt_bias)):
-        raise InvalidArgument("delta_rule: a_log and dt_bias are float32 [heads]")
+    if any(t.dtype != torch.float32 for t in (a_log, dt_bias)) or a_log.numel() != heads \
+            or dt_bias.numel() != heads * (dim if by_channel else 1):
+        raise InvalidArgument("delta_rule: a_log is float32 [heads], dt_bias float32 [heads] or one per channel")
     if heads % kv_heads or dim > 512:
         raise Unsupported(f"delta_rule: {heads} heads over {kv_heads} query/key heads of {dim} (at most 512) has no kernel")
     _state_rows(state, heads * dim * vdim, "delta_rule")
     if out.dtype != torch.float32 or not out.is_contiguous() or out.shape != (u.shape[0], heads * vdim):
         raise InvalidArgument("delta_rule: out float32 contiguous [rows, H*e]")
+    stride = 0
+    if by_channel:
+        _rows_contiguous(channel_decay, "channel_decay")
+        stride = channel_decay.stride(0)
+        if channel_decay.dtype != torch.float32 or channel_decay.shape[0] < u.shape[0] or channel_decay.shape[1] < heads * dim:
+            raise InvalidArgument("delta_rule: channel_decay float32 [rows, >= H*d]")
     check_limits("delta_rule", requests=state.shape[0], rows=u.shape[0])
     # a step of single tokens goes to the light kernel that is bound by the state's trip through memory alone
-    entry = "dl_delta_rule_step" if u.shape[0] <= requests else "dl_delta_rule"
-    _check(_fn("delta_rule", entry)(dtype_code(u.dtype), _p(u), u.stride(0), q_col, k_col, v_col, _p(proj),
-                                               proj.stride(0), b_col, a_col, _p(a_log), _p(dt_bias), _p(state),
-                                               state.stride(0), _p(q_start), _p(state_slots), _p(out), requests, heads,
-                                               kv_heads, dim, vdim, _stream()), "delta_rule")
+    single = u.shape[0] <= requests
+    if by_channel and not single:
+        _check(_fn("delta_rule", "dl_delta_decay")(_p(channel_decay), stride, _p(a_log), _p(dt_bias), u.shape[0], heads, dim,
+                                                    _stream()), "delta_decay")
+    _check(_fn("delta_rule", "dl_delta_rule_step" if single else "dl_delta_rule")(
+        dtype_code(u.dtype), _p(u), u.stride(0), q_col, k_col, v_col, _p(proj), proj.stride(0), b_col, a_col, _p(a_log),
+        _p(dt_bias), _p(channel_decay), stride, _p(state), state.stride(0), _p(q_start), _p(state_slots), _p(out), requests,
+        heads, kv_heads, dim, vdim, _stream()), "delta_rule")
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, gate_col: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
-                   heads: int, vdim: int) -> None:
-    """out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * silu(gate[t, gate_col + h * e ...]).
-    o: float32 contiguous [rows, H*e]; weight: float32 [e]; out: contiguous [rows, H*e] of gate's dtype."""
+                   heads: int, vdim: int, act: str = "silu") -> None:
+    """out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * act(gate[t, gate_col + h * e ...]), act "silu" or
+    "sigmoid". o: float32 contiguous [rows, H*e]; weight: float32 [e]; gate: of out's dtype or float32; out: contiguous
+    [rows, H*e]."""
     _cuda(o, gate, weight, out)
     _rows_contiguous(gate, "gate")
     rows = o.shape[0]
     if o.dtype != torch.float32 or not o.is_contiguous() or o.shape != (rows, heads * vdim) or weight.dtype != torch.float32 \
-            or weight.numel() != vdim or out.shape != o.shape or not out.is_contiguous() or out.dtype != gate.dtype \
-            or gate_col + heads * vdim > gate.shape[1] or gate.shape[0] < rows:
-        raise InvalidArgument("head_norm_gate: o float32 [rows, H*e], weight float32 [e], out [rows, H*e] of the gate's dtype")
-    _check(_fn("delta_rule", "dl_head_norm_gate")(dtype_code(gate.dtype), _p(o), _p(gate), gate.stride(0), gate_col,
-                                                   _p(weight), eps, _p(out), rows, heads, vdim, _stream()), "head_norm_gate")
+            or weight.numel() != vdim or out.shape != o.shape or not out.is_contiguous() or gate.dtype not in (out.dtype, torch.float32) \
+            or gate_col + heads * vdim > gate.shape[1] or gate.shape[0] < rows or act not in ("silu", "sigmoid"):
+        raise InvalidArgument("head_norm_gate: o float32 [rows, H*e], weight float32 [e], out [rows, H*e], a gate of its dtype or float32")
+    _check(_fn("delta_rule", "dl_head_norm_gate")(dtype_code(out.dtype), dtype_code(gate.dtype), _p(o), _p(gate), gate.stride(0),
+                                                   gate_col, _p(weight), eps, 1 if act == "sigmoid" else 0, _p(out), rows, heads,
+                                                   vdim, _stream()), "head_norm_gate")
 
 
 def rglru_gates(u: torch.Tensor, wa_t: torch.Tensor, ba: torch.Tensor, wi_t: torch.Tensor, bi: torch.Tensor,
@@ -1810,12 +1830,14 @@ def paged_attention_generic_kv(q: torch.Tensor, k_cache: torch.Tensor, k_row: in
                                block_table: torch.Tensor, positions: torch.Tensor, row_request: torch.Tensor,
                                out: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, vdim: int, page_size: int,
                                scale: float, window: int = 0, keep_first: int = 0, sink: bool = False,
-                               rate: Optional[torch.Tensor] = None, step: Optional[torch.Tensor] = None) -> None:
+                               rate: Optional[torch.Tensor] = None, step: Optional[torch.Tensor] = None,
+                               chunk: int = 0) -> None:
     """paged_attention_generic with keys of head_dim and values of vdim numbers: k_cache / v_cache point at the first
     token's keys / values (KV head j at j * head_dim / j * vdim), k_row / v_row elements lie between two tokens.
     out: rows with head h at column h * vdim. keep_first: keys at positions below it stay visible behind the window;
     sink: the softmax's denominator holds one more term of score 0, which carries no value; rate, step (float32 [n_heads],
-    both or neither): rate_h ln(1 + step_h * distance) comes off every score."""
+    both or neither): rate_h ln(1 + step_h * distance) comes off every score; chunk > 0 (without a window): a position sees
+    keys of its own chunk of that many positions alone."""
     _cuda(rate, step)
     _distance_bias(rate, step, n_heads)
     _cuda(q, k_cache, v_cache, block_table, positions, row_request, out)
@@ -1831,7 +1853,7 @@ def paged_attention_generic_kv(q: torch.Tensor, k_cache: torch.Tensor, k_row: in
     _check(_fn("attention_generic", "dl_paged_attention_generic_masked")(
         dtype_code(q.dtype), _p(q), q.stride(0), _p(k_cache), k_row, _p(v_cache), v_row, _p(block_table),
         block_table.stride(0), _p(positions), _p(row_request), _p(out), out.stride(0), q.shape[0], n_heads, n_kv_heads,
-        head_dim, vdim, page_size, scale, window, int(keep_first), 1 if sink else 0, _p(rate), _p(step), _stream()),
+        head_dim, vdim, page_size, scale, window, int(keep_first), 1 if sink else 0, _p(rate), _p(step), int(chunk), _stream()),
            "paged_attention_generic_kv")
 
 
@@ -2038,13 +2060,13 @@ def moe_tile_rows(pairs: int, experts: int, a: torch.Tensor, widths) -> int:
 
 def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, scale: float, ids: torch.Tensor,
               weights: torch.Tensor, correction: Optional[torch.Tensor] = None, scores: str = "softmax",
-              group_score: str = "max", renormalize: bool = True) -> None:
-    """Per row of float32 router logits [tokens, experts]: scores = softmax over all experts (or the sigmoid of each), choice
+              group_score: str = "max", renormalize: bool = True, bias: Optional[torch.Tensor] = None) -> None:
+    """Per row of float32 router logits [tokens, experts] (+ `bias`, float32 [experts], when given): scores = softmax over all experts (or the sigmoid of each), choice
     scores = scores + correction (float32 [experts], or None), the `keep` best of `groups` equal groups of neighbouring
     experts (a group's score: its largest choice score, or with group_score "top2" the sum of its two largest), the `top`
     experts of those groups with the largest choice scores (ids int32 [tokens, top]) and their scores, over their sum
     (renormalize) or as they are, times `scale` (weights float32 [tokens, top])."""
-    _cuda(logits, ids, weights, correction)
+    _cuda(logits, ids, weights, correction, bias)
     _rows_contiguous(logits, "logits")
     tokens, experts = logits.shape
     if logits.dtype != torch.float32 or ids.dtype != torch.int32 or weights.dtype != torch.float32 \
@@ -2052,12 +2074,12 @@ def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, scale: flo
         raise InvalidArgument("moe_route: logits float32, ids int32 [tokens, top], weights float32 [tokens, top]")
     if scores not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
         raise InvalidArgument(f"moe_route: no scores '{scores}' (softmax, sigmoid) or group score '{group_score}' (max, top2)")
-    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts):
-        raise InvalidArgument("moe_route: correction float32 [experts]")
+    if any(t is not None and (t.dtype != torch.float32 or t.numel() != experts) for t in (correction, bias)):
+        raise InvalidArgument("moe_route: correction and bias are float32 [experts]")
     if experts > MOE_MAX_EXPERTS or top > experts or groups <= 0 or experts % groups or not 0 < keep <= groups \
             or top > keep * (experts // groups):
         raise Unsupported(f"moe_route: {experts} experts in {groups} groups, {keep} kept, {top} a token")
-    _check(_fn("moe", "dl_moe_route")(_p(logits), logits.stride(0), tokens, experts, top, groups, keep, _p(correction),
+    _check(_fn("moe", "dl_moe_route")(_p(logits), logits.stride(0), tokens, experts, top, groups, keep, _p(bias), _p(correction),
                                       1 if scores == "sigmoid" else 0, 1 if group_score == "top2" else 0,
                                       1 if renormalize else 0, scale, _p(ids), _p(weights), _stream()), "moe_route")
 
@@ -2137,7 +2159,7 @@ def masked_flash_attention(q: torch.Tensor, k_cache: torch.Tensor, k_row: int, v
                            n_kv_heads: int, key_dim: int, value_dim: int, page_size: int, scale: float, window: int = 0,
                            keep_first: int = 0, sink: bool = False, one_token_tiles: bool = False, parts: int = 1,
                            partial: Optional[torch.Tensor] = None, rate: Optional[torch.Tensor] = None,
-                           step: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                           step: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """Flash attention of query tiles over the paged cache, bfloat16, with keys of key_dim and values of value_dim
     numbers (a pair of MASKED_FLASH_SIZES), kept first tokens behind the window and an optional extra term exp(0) in the
     denominator; see csrc/attention_masked_flash.cu. q_tiles: int32 [n_tiles, 4] = (request, first row, rows <= 128,
@@ -2146,7 +2168,7 @@ def masked_flash_attention(q: torch.Tensor, k_cache: torch.Tensor, k_row: int, v
     then share a block, and with parts > 1 a row's key tiles are dealt over that many blocks whose results a second
     kernel merges (partial: float32 scratch of masked_flash_partial_floats elements). rate, step (float32 [n_heads], both or
     neither): rate_h ln(1 + step_h * distance) comes off every score. gate (bfloat16, head h at column h * value_dim): the
-    output is multiplied by its sigmoid."""
+    output is multiplied by its sigmoid. chunk > 0 (without a window): a position sees keys of its own chunk alone."""
     _cuda(rate, step, gate)
     _distance_bias(rate, step, n_heads)
     if gate is not None:
@@ -2175,7 +2197,7 @@ def masked_flash_attention(q: torch.Tensor, k_cache: torch.Tensor, k_row: int, v
         _p(q), q.stride(0), _p(k_cache), k_row, _p(v_cache), v_row, _p(block_table), block_table.stride(0), _p(q_tiles),
         n_tiles, _p(out), out.stride(0), n_heads, n_kv_heads, key_dim, value_dim, page_size, scale, window, int(keep_first),
         1 if sink else 0, 1 if one_token_tiles else 0, int(parts), _p(partial) if parts > 1 else None,
-        _p(rate), _p(step), _p(gate), gate.stride(0) if gate is not None else 0, _stream()), "masked_flash_attention")
+        _p(rate), _p(step), _p(gate), gate.stride(0) if gate is not None else 0, int(chunk), _stream()), "masked_flash_attention")
 
 
 MASKED_FLASH_MAX_PARTS = 8
@@ -2371,3 +2393,56 @@ def token_gate(z: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, out: tor
     check_limits("gates", rows=rows, vocab=table.shape[0])
     _check(_fn("gates", "dl_token_gate")(dtype_code(z.dtype), _p(z), _p(table), table.stride(0), _p(ids), _p(out), rows, n,
                                          table.shape[0], _stream()), "token_gate")
+
+
+def qk_norm_turn_cache(proj: torch.Tensor, wq: torch.Tensor, wk: torch.Tensor, eps: float, freq: Optional[torch.Tensor], rot: int,
+                       mag: float, positions: torch.Tensor, row_slot: torch.Tensor, block_table: torch.Tensor,
+                       k_cache: torch.Tensor, k_row: int, v_cache: torch.Tensor, v_row: int, heads: int, kv_heads: int, dim: int,
+                       vdim: int, page_size: int, values_are_keys: bool = False) -> None:
+    """Rows [q: H*d | k: G*d | v: G*e | ...] of a projection: every head of q and k divided by its own root mean square and
+    multiplied by a weight that all heads share (wq, wk: float32 [d]), then its first `rot` numbers turned by position * freq
+    (float64 [rot / 2], pairs i and i + rot / 2), lengths times `mag`; q written back in place, k and v to the token's place
+    in the cache. values_are_keys: there are no columns v, a key as projected is the value too. See csrc/qk_proj_norm.cu."""
+    _cuda(proj, wq, wk, freq, positions, row_slot, block_table, k_cache, v_cache)
+    _rows_contiguous(proj, "proj")
+    if proj.shape[1] < heads * dim + kv_heads * (dim + (0 if values_are_keys else vdim)) or k_cache.dtype != proj.dtype \
+            or v_cache.dtype != proj.dtype:
+        raise InvalidArgument("qk_norm_turn_cache: proj holds q | k | v; the cache has proj's dtype")
+    if any(w.dtype != torch.float32 or w.numel() != dim for w in (wq, wk)):
+        raise InvalidArgument("qk_norm_turn_cache: a norm weight is float32 [dim]")
+    if rot and (freq is None or freq.dtype != torch.float64 or freq.numel() < rot // 2):
+        raise InvalidArgument("qk_norm_turn_cache: freq float64 [rot / 2]")
+    if dim > 256 or vdim > 256:
+        raise Unsupported(f"qk_norm_turn_cache: heads of {dim} and {vdim} numbers (256 at most)")
+    check_limits("qk_proj_norm", pages=k_cache.shape[0], requests=block_table.shape[0], rows=proj.shape[0])
+    _check(_fn("qk_proj_norm", "dl_qk_norm_turn_cache")(
+        dtype_code(proj.dtype), _p(proj), proj.stride(0), _p(wq), _p(wk), eps, _p(freq), rot, mag, _p(positions), _p(row_slot),
+        _p(block_table), block_table.stride(0), _p(k_cache), k_row, _p(v_cache), v_row, proj.shape[0], heads, kv_heads, dim, vdim,
+        page_size, 1 if values_are_keys else 0, _stream()), "qk_norm_turn_cache")
+
+
+def normed_sum(a: torch.Tensor, wa: torch.Tensor, sa: float, b: torch.Tensor, wb: torch.Tensor, sb: float, eps: float,
+               out: torch.Tensor) -> None:
+    """out = sa * rmsnorm(a) * wa + sb * rmsnorm(b) * wb (float32 [n, width]); a and b are [n, width] or split-K partial sums
+    [parts, n, width] of either dtype, added in order; wa, wb: float32 [width]. See csrc/norm_sandwich.cu."""
+    _cuda(a, wa, b, wb, out)
+    rows, width = out.shape
+    pa, stride_a = _delta_parts(a, width, "normed_sum")
+    pb, stride_b = _delta_parts(b, width, "normed_sum")
+    if out.dtype != torch.float32 or not out.is_contiguous() or a.shape[-2:] != out.shape or b.shape[-2:] != out.shape \
+            or any(w.dtype != torch.float32 or w.numel() != width for w in (wa, wb)):
+        raise InvalidArgument("normed_sum: out float32 contiguous, of the shape of a and b; weights float32 [width]")
+    _check(_fn("norm_sandwich", "dl_normed_sum")(dtype_code(a.dtype), _p(a), pa, stride_a, _p(wa), sa, dtype_code(b.dtype), _p(b),
+                                                  pb, stride_b, _p(wb), sb, eps, _p(out), rows, width, _stream()), "normed_sum")
+
+
+def clamped_swiglu(gate_up: torch.Tensor, bias: Optional[torch.Tensor], limit: float, gate_scale: float, out: torch.Tensor) -> None:
+    """With [g | u] = gate_up + bias (float32 [2 * inner], or None): out = min(g, limit) sigmoid(gate_scale min(g, limit))
+    (clamp(u, -limit, limit) + 1)."""
+    _cuda(gate_up, bias, out)
+    rows, inner = out.shape
+    if gate_up.shape != (rows, 2 * inner) or gate_up.dtype != out.dtype or not gate_up.is_contiguous() or not out.is_contiguous() \
+            or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != 2 * inner)):
+        raise InvalidArgument("clamped_swiglu: gate_up contiguous [rows, 2 * inner], out contiguous [rows, inner], one dtype")
+    _check(_fn("activation", "dl_clamped_swiglu")(dtype_code(out.dtype), _p(gate_up), _p(bias), limit, gate_scale, _p(out), rows,
+                                                   inner, _stream()), "clamped_swiglu")

@@ -1,2 +1,2 @@
 """Architectures; importing this package registers them."""
-from . import bugapel, llama, rematar, rodelorn, sipelorn, todupel  # noqa: F401
+from . import bugapel, llama, nisotar, rematar, rodelorn, sipelorn, todupel  # noqa: F401

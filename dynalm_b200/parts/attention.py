@@ -14,7 +14,7 @@ import torch
 
 from ..errors import Unsupported
 from ..kernels import linear, ops
-from ..kernels.gemm import linear_partial
+from ..kernels.gemm import linear_partial, linear_partial_biased
 from .base import POSITIONS, CacheSpec, TensorDecl, register_mixer
 
 
@@ -162,13 +162,19 @@ class GatedNormedAttention(PagedAttention):
     qk_norm     "projection": queries and keys normed over their WHOLE projection before the heads are cut and before
                 the rotation (one statistic for all H * d numbers of q, one for the G * d of k; weights q_norm, k_norm);
                 "head": after the rotation every head of q and k is divided by its own root mean square (no weight);
+                "head_first": before the rotation every head of q and k is normed by itself, with weights q_norm, k_norm of
+                one head that all heads share;
                 "none".
     gated       the concatenated heads times sigmoid(W_g h) before the output projection (one product gives
                 [q | k | v | gate]).
     sink        "zero": the softmax's denominator holds one more term of score 0, which carries no value; "none".
     keep_first  with a window: keys at positions below it stay visible behind the window, at their true positions.
+    chunk       n > 0: a position sees keys of its own chunk alone, floor(i / n) = floor(j / n), counted from the start of the
+                sequence (instead of a window).
+    values      "own": the projection v; "keys": a key as projected, before norm and rotation, is the value too (no tensor v;
+                with qk_norm "head_first").
     position    "rotary" (pairs i, i + rotary_dim / 2) or, with qk_norm "head" or "none", "rotary_interleaved" (pairs 2i,
-                2i + 1).
+                2i + 1); with qk_norm "head_first" "rotary_halves" (pairs i, i + rotary_dim / 2, and a magnitude).
     conv        K > 0: short causal convolutions of K taps over the channels of q, k and v, directly behind the projections
                 (tensors q_conv, k_conv, v_conv [channels, K]); a request keeps the last K - 1 projected values as a float32
                 state row beside its pages.
@@ -178,8 +184,8 @@ class GatedNormedAttention(PagedAttention):
     cache_window  the widest window of all runs that read this layer's cache (0: all earlier keys); default `window`.
     Biases of the four projections are taken when the model has them (q_bias, k_bias, v_bias, o_bias).
 
-    Parameters: num_heads, num_kv_heads, head_dim, value_dim, scale, window, cache_window, keep_first, eps, qk_norm, gated,
-    sink, conv, distance_bias, own_kv, position. Tensors: q, k, v, o, and by the parameters q_norm, k_norm, gate, q_conv,
+    Parameters: num_heads, num_kv_heads, head_dim, value_dim, scale, window, chunk, cache_window, keep_first, eps, qk_norm,
+    gated, sink, conv, distance_bias, own_kv, values, position. Tensors: q, k, v, o, and by the parameters q_norm, k_norm, gate, q_conv,
     k_conv, v_conv, distance_rate, distance_step.
 
     Where keys and values have one size the cache is the plain attention's (two arrays) and so are the kernels that
@@ -193,10 +199,14 @@ class GatedNormedAttention(PagedAttention):
     def declare(spec) -> Dict[str, TensorDecl]:
         qw, kw, vw = spec.num_heads * spec.head_dim, spec.num_kv_heads * spec.head_dim, spec.num_kv_heads * spec.value_dim
         ow = spec.num_heads * spec.value_dim
-        normed, gated = spec.get("qk_norm", "none") == "projection", bool(spec.get("gated", False))
+        qk_norm, gated = spec.get("qk_norm", "none"), bool(spec.get("gated", False))
+        normed = qk_norm in ("projection", "head_first")
+        one_head = qk_norm == "head_first"
         more = {}
         if spec.get("own_kv", True):
-            more.update({"k": TensorDecl((kw, spec.width)), "v": TensorDecl((vw, spec.width))})
+            more["k"] = TensorDecl((kw, spec.width))
+            if spec.get("values", "own") == "own":
+                more["v"] = TensorDecl((vw, spec.width))
         if spec.get("conv", 0) > 0:
             for name, n in (("q", qw), ("k", kw), ("v", vw)):
                 if name == "q" or spec.get("own_kv", True):
@@ -206,8 +216,8 @@ class GatedNormedAttention(PagedAttention):
         return {
             "q": TensorDecl((qw, spec.width)), **more,
             "o": TensorDecl((spec.width, ow)),
-            "q_norm": TensorDecl((qw,), role="vector", required=normed, init="around_one"),
-            "k_norm": TensorDecl((kw,), role="vector", required=normed, init="around_one"),
+            "q_norm": TensorDecl((spec.head_dim if one_head else qw,), role="vector", required=normed, init="around_one"),
+            "k_norm": TensorDecl((spec.head_dim if one_head else kw,), role="vector", required=normed, init="around_one"),
             "gate": TensorDecl((ow, spec.width), required=gated),
             "q_bias": TensorDecl((qw,), role="vector", required=False, init="bias"),
             "k_bias": TensorDecl((kw,), role="vector", required=False, init="bias"),
@@ -220,8 +230,8 @@ class GatedNormedAttention(PagedAttention):
             raise Unsupported(f"gated_attention: head_dim {spec.head_dim} and value_dim {spec.value_dim} must be at most 256")
         if spec.num_heads % spec.num_kv_heads:
             raise Unsupported(f"gated_attention: {spec.num_heads} heads do not divide into {spec.num_kv_heads} KV heads")
-        if spec.get("qk_norm", "none") not in ("projection", "head", "none"):
-            raise Unsupported(f"gated_attention: no query/key norm '{spec.qk_norm}' (projection, head, none)")
+        if spec.get("qk_norm", "none") not in ("projection", "head", "head_first", "none"):
+            raise Unsupported(f"gated_attention: no query/key norm '{spec.qk_norm}' (projection, head, head_first, none)")
         if spec.get("sink", "none") not in ("zero", "none"):
             raise Unsupported(f"gated_attention: no sink '{spec.sink}' (zero, none)")
         self.spec = spec
@@ -232,9 +242,16 @@ class GatedNormedAttention(PagedAttention):
         self.o_width = spec.num_heads * spec.value_dim
         self.normed = spec.get("qk_norm", "none") == "projection"
         self.head_normed = spec.get("qk_norm", "none") == "head"
+        self.head_first = spec.get("qk_norm", "none") == "head_first"
         self.sink = spec.get("sink", "none") == "zero"
         self.window = int(spec.get("window", 0))
+        self.chunk = int(spec.get("chunk", 0))
         self.keep_first = int(spec.get("keep_first", 0)) if self.window > 0 else 0
+        if self.chunk > 0 and (self.window > 0 or self.keep_first > 0):
+            raise Unsupported("gated_attention: a layer has chunks or a window, not both")
+        self.values_are_keys = spec.get("values", "own") == "keys"
+        if self.values_are_keys and (not self.head_first or spec.head_dim != spec.value_dim):
+            raise Unsupported("gated_attention: values that are the keys have their size and go with qk_norm 'head_first'")
         self.gated = bool(spec.get("gated", False))
         self.same = spec.head_dim == spec.value_dim          # keys and values of one size: the plain attention's cache
         self.own_kv = bool(spec.get("own_kv", True))
@@ -242,7 +259,9 @@ class GatedNormedAttention(PagedAttention):
         # one product, [q | k | v | gate]; a layer that reads another's keys has [q | gate]
         self.widths = (self.q_width, self.kv_width, self.v_width) if self.own_kv else (self.q_width, 0, 0)
         self.channels = sum(self.widths)
-        names = ("q", "k", "v") if self.own_kv else ("q",)
+        names = (("q", "k") if self.values_are_keys else ("q", "k", "v")) if self.own_kv else ("q",)
+        if self.head_first and (self.gated or not self.own_kv or self.taps > 0 or any(tensors.get(n + "_bias") is not None for n in names)):
+            raise Unsupported("gated_attention: qk_norm 'head_first' goes without gate, biases, convolutions and readers")
         mats = [tensors[n] for n in names] + ([tensors["gate"]] if self.gated else [])
         self.w_qkv = torch.cat(mats, dim=0).contiguous()
         self.joined_col = self.w_qkv.shape[0]
@@ -250,7 +269,7 @@ class GatedNormedAttention(PagedAttention):
         self.b_qkv = None
         # by itself the kernel of the short convolutions also adds the biases and writes the cache; a layer without a
         # rotation or norm that has an output gate or reads another's cache goes through it too
-        plain_q = not self.normed and not self.head_normed and spec.get("position") is None
+        plain_q = not self.normed and not self.head_normed and not self.head_first and spec.get("position") is None
         self.conv_path = plain_q and (self.taps > 0 or self.gated or not self.own_kv)
         if not self.conv_path and (self.taps > 0 or not self.own_kv):
             raise Unsupported("gated_attention: convolutions and the cache of another run go without rotation and norm")
@@ -264,19 +283,22 @@ class GatedNormedAttention(PagedAttention):
         if spec.get("distance_bias", "none") not in ("log", "none"):
             raise Unsupported(f"gated_attention: no distance bias '{spec.distance_bias}' (log, none)")
         self.rate, self.dstep = tensors.get("distance_rate"), tensors.get("distance_step")
-        self.q_norm, self.k_norm = (tensors["q_norm"], tensors["k_norm"]) if self.normed else (None, None)
+        self.q_norm, self.k_norm = (tensors["q_norm"], tensors["k_norm"]) if self.normed or self.head_first else (None, None)
         self.w_o = tensors["o"]
         self.b_o = tensors.get("o_bias")
         self.eps = float(spec.get("eps", 1e-6))
         pos = spec.get("position")
         self.position = POSITIONS.get(pos.kind)(pos, runtime) if pos is not None else None
         self.interleaved = bool(getattr(self.position, "interleaved", False))
-        if self.position is not None and self.position.table() is None and not self.interleaved:
+        if self.head_first:
+            if self.position is not None and not getattr(self.position, "halves", False):
+                raise Unsupported("gated_attention: qk_norm 'head_first' goes with the rotation 'rotary_halves' or with none")
+        elif self.position is not None and self.position.table() is None and not self.interleaved:
             raise Unsupported("gated_attention: the rotation runs inside its kernel and takes a position encoding with a table")
         if self.interleaved and self.normed:
             raise Unsupported("gated_attention: the interleaved rotation goes with the norm per head or with none")
         # the kernels of the plain attention's cache know a window and an ordinary softmax over scaled scores
-        self.plain_mask = not self.sink and self.keep_first == 0 and self.rate is None
+        self.plain_mask = not self.sink and self.keep_first == 0 and self.rate is None and self.chunk == 0
 
     def join_input(self, w: torch.Tensor) -> bool:
         """Takes the rows of another product over the same input into this part's first one; `joined` gives its result."""
@@ -304,7 +326,9 @@ class GatedNormedAttention(PagedAttention):
         if not ctx.decode_only:
             return 1
         s = self.spec
-        span = ctx.max_kv_len if self.window <= 0 else min(ctx.max_kv_len, self.window + self.keep_first)
+        span = ctx.max_kv_len
+        if self.window > 0 or self.chunk > 0:
+            span = min(span, self.chunk or self.window + self.keep_first)
         bucket = 256
         while bucket < span:
             bucket *= 2
@@ -313,7 +337,8 @@ class GatedNormedAttention(PagedAttention):
 
     def cache_spec(self) -> Optional[CacheSpec]:
         s = self.spec
-        window = int(s.get("cache_window", self.window)) if self.keep_first == 0 else 0      # kept first tokens: no page is given back
+        # kept first tokens: no page is given back; a key of the same chunk is less than a chunk away
+        window = int(s.get("cache_window", self.chunk or self.window)) if self.keep_first == 0 else 0
         state = self._kept_shape()
         if self.same:
             return CacheSpec(kind="pages", entry_shape=(s.num_kv_heads, s.head_dim), tensors=2, window=window, state_shape=state)
@@ -345,11 +370,18 @@ class GatedNormedAttention(PagedAttention):
         if self.conv_path:
             return self._forward_conv(x, ctx, cache)
         proj = rt.buffer("gattn_proj", (rows, self.w_qkv.shape[0]))
-        by_projection = self.normed or (not self.head_normed and not self.interleaved)
+        by_projection = self.normed or (not self.head_normed and not self.head_first and not self.interleaved)
         # a bias joins in the kernel that turns and norms, where that kernel takes one; else in the product (the plain one)
         linear(x, self.w_qkv, proj, self.b_qkv if (by_projection or self.gated) else None)
         k_cache, k_row, v_cache, v_row = self._kv(cache)
-        if by_projection:
+        if self.head_first:
+            pos = self.position
+            ops.qk_norm_turn_cache(proj, self.q_norm, self.k_norm, self.eps, pos.frequencies if pos is not None else None,
+                                   pos.rotary_dim if pos is not None else 0, pos.magnitude if pos is not None else 1.0,
+                                   ctx.positions, ctx.row_slot, cache.block_table, k_cache, k_row, v_cache, v_row,
+                                   s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, cache.page_size,
+                                   values_are_keys=self.values_are_keys)
+        elif by_projection:
             inv_freq, rot, pos_scale = self.position.table() if self.position is not None else (None, 0, 1.0)
             ops.qk_proj_norm_cache(proj, self.q_norm, self.k_norm, self.eps, self.normed, inv_freq, rot, pos_scale,
                                    ctx.positions, ctx.row_slot, cache.block_table, k_cache, k_row, v_cache, v_row,
@@ -375,23 +407,7 @@ class GatedNormedAttention(PagedAttention):
         return self._project(attn)
 
     def _project(self, attn: torch.Tensor) -> torch.Tensor:
-        s, rt, rows = self.spec, self.rt, attn.shape[0]
-        if self.b_o is None:
-            return linear_partial(attn, self.w_o, rt, self.out_name)
-        if attn.dtype == torch.float32:
-            out = rt.buffer(self.out_name, (rows, s.width))
-            linear(attn, self.w_o, out, self.b_o)
-            return out
-        # 16-bit operands: the product leaves float32 sums (whole, or split-K partial sums) and the bias joins those
-        from ..kernels.gemm import skinny_ok, use_stream
-        if use_stream(attn, self.w_o) or skinny_ok(attn, self.w_o):
-            out = linear_partial(attn, self.w_o, rt, self.out_name)
-            ops.add_bias(out[0] if out.dim() == 3 else out, self.b_o)
-            return out
-        out = rt.buffer(self.out_name + "_wide", (rows, s.width), torch.float32)
-        linear(attn, self.w_o, out)
-        ops.add_bias(out, self.b_o)
-        return out
+        return linear_partial_biased(attn, self.w_o, self.b_o, self.rt, self.out_name)
 
     def _forward_conv(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         """One product, one kernel that convolves, adds biases and writes the cache, attention with the output gate."""
@@ -438,7 +454,7 @@ class GatedNormedAttention(PagedAttention):
                                        s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, cache.page_size,
                                        float(s.scale), self.window, self.keep_first, self.sink,
                                        one_token_tiles=ctx.decode_only, parts=parts, partial=partial, rate=self.rate, step=self.dstep,
-                                       gate=gate)
+                                       gate=gate, chunk=self.chunk)
             return gate is not None
         if self.same and self.plain_mask:
             from ..kernels import attention as fast
@@ -447,5 +463,6 @@ class GatedNormedAttention(PagedAttention):
         k_cache, k_row, v_cache, v_row = self._kv(cache)
         ops.paged_attention_generic_kv(qkv, k_cache, k_row, v_cache, v_row, cache.block_table, ctx.positions, ctx.row_slot,
                                        out, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, cache.page_size,
-                                       float(s.scale), self.window, self.keep_first, self.sink, rate=self.rate, step=self.dstep)
+                                       float(s.scale), self.window, self.keep_first, self.sink, rate=self.rate, step=self.dstep,
+                                       chunk=self.chunk)
         return False

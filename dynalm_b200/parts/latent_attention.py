@@ -18,8 +18,10 @@ per-head products are block-diagonal (ops.head_linear). The window (0: every ear
 manager which pages may be given back.
 
 All sizes and constants come from the spec: num_heads, head_dim (d), rot_dim (r), value_dim (e), q_rank, kv_rank (R),
-scale, window, eps, position (a PositionSpec of kind "rotary_interleaved", or None); the sinks and the output gate are
-there when the model has their tensors.
+scale, window, eps, position (a PositionSpec of kind "rotary_interleaved" or "rotary_halves", or None); the sinks and the
+output gate are there when the model has their tensors. The kernels turn neighbours: for a rotation by halves the rows of
+the projections that make the rotated parts of queries and keys are put in another order at load time, pair by pair, which
+changes no score.
 """
 
 from __future__ import annotations
@@ -66,20 +68,27 @@ class LatentAttention:
         self.has_gate = "gate" in tensors
         # one product for everything that reads the layer's input: [query latent or queries | latent | key part | gate]
         self.q_cols = spec.q_rank or H * (d + r)
-        down = [tensors["dq"] if spec.q_rank else tensors["q"], tensors["dkv"]] + ([tensors["gate"]] if self.has_gate else [])
+        pos = spec.get("position")
+        self.position = POSITIONS.get(pos.kind)(pos, runtime) if pos is not None else None
+        w_q, w_dkv = tensors["uq"] if spec.q_rank else tensors["q"], tensors["dkv"]
+        if getattr(self.position, "halves", False):
+            order = self.position.neighbours(r).to(w_q.device)
+            per_head = w_q.reshape(H, d + r, -1)
+            w_q = torch.cat([per_head[:, :d], per_head[:, d:][:, order]], dim=1).reshape(H * (d + r), -1).contiguous()
+            w_dkv = torch.cat([w_dkv[:R], w_dkv[R:][order]], dim=0)
+        elif self.position is not None and not getattr(self.position, "interleaved", False):
+            raise Unsupported(f"latent_attention: position encoding '{pos.kind}' has no kernel here (rotary_interleaved and "
+                              f"rotary_halves have)")
+        down = [tensors["dq"] if spec.q_rank else w_q, w_dkv] + ([tensors["gate"]] if self.has_gate else [])
         self.w_down = torch.cat(down, dim=0).contiguous()
         self.dq_norm, self.dkv_norm = tensors.get("dq_norm"), tensors["dkv_norm"]
-        self.w_uq = tensors.get("uq")
+        self.w_uq = w_q if spec.q_rank else None
         self.joined_col = self.w_down.shape[0]
         self.w_uk = tensors["uk"].reshape(H, d, R).contiguous()                          # [H, in = d, out = R] as stored
         self.w_uv = tensors["uv"].reshape(H, e, R).transpose(1, 2).contiguous()          # [H, in = R, out = e]
         self.sink = tensors.get("sink")
         self.w_o = tensors["o"]
         self.eps = float(spec.eps)
-        pos = spec.get("position")
-        self.position = POSITIONS.get(pos.kind)(pos, runtime) if pos is not None else None
-        if self.position is not None and not getattr(self.position, "interleaved", False):
-            raise Unsupported(f"latent_attention: position encoding '{pos.kind}' has no kernel here (rotary_interleaved has)")
         self.rot = self.position.rotary_dim if self.position is not None else 0
         self.freq = self.position.frequencies if self.position is not None else None
         self.mag = self.position.magnitude if self.position is not None else 1.0

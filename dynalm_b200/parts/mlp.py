@@ -1,6 +1,8 @@
 """Gated feed-forward: down(act(gate x) * up x), the "gated_mlp" kind
 (dynalm/src/model/transformer.cpp:671-693), act silu or the tanh form of GELU (parameter `activation`). Gate and up
-run as one product against [Wg; Wu].
+run as one product against [Wg; Wu]. Its third activation, "clamped_swiglu", clamps both halves: with g = min(gate x, limit)
+and u = clamp(up x, -limit, limit), g sigmoid(gate_scale g) (u + 1). The projections' biases are taken when the model has
+them, with that activation.
 Ungated feed-forward: down(act(up x)), the "mlp" kind, act the squared ReLU, the tanh form of GELU or xIELU.
 A small input that depends on the token alone: the "token_side" kind."""
 
@@ -13,7 +15,8 @@ import torch
 from ..errors import Unsupported
 from ..kernels import ops
 from ..kernels import linear
-from ..kernels.gemm import linear_act, linear_geglu, linear_partial, linear_swiglu, linear_xielu
+from ..kernels.gemm import (linear_act, linear_clamped_swiglu, linear_geglu, linear_partial, linear_partial_biased, linear_swiglu,
+                            linear_xielu)
 from .base import TensorDecl, register_feed_forward
 
 
@@ -28,12 +31,23 @@ class GatedMLP:
             "gate": TensorDecl((spec.inner, spec.width)),
             "up": TensorDecl((spec.inner, spec.width)),
             "down": TensorDecl((spec.width, spec.inner)),
+            "gate_bias": TensorDecl((spec.inner,), role="vector", required=False, init="bias"),
+            "up_bias": TensorDecl((spec.inner,), role="vector", required=False, init="bias"),
+            "down_bias": TensorDecl((spec.width,), role="vector", required=False, init="bias"),
         }
 
     def __init__(self, spec, tensors: Dict[str, torch.Tensor], runtime):
         self.activation = spec.get("activation", "silu")
-        if self.activation not in ("silu", "gelu_tanh"):
-            raise Unsupported(f"gated_mlp: activation '{self.activation}' has no kernel (silu and gelu_tanh do)")
+        if self.activation not in ("silu", "gelu_tanh", "clamped_swiglu"):
+            raise Unsupported(f"gated_mlp: activation '{self.activation}' has no kernel (silu, gelu_tanh and clamped_swiglu do)")
+        self.b_gate_up = None
+        biases = [tensors.get("gate_bias"), tensors.get("up_bias")]
+        if any(b is not None for b in biases):
+            self.b_gate_up = torch.cat([b if b is not None else torch.zeros(spec.inner, dtype=torch.float32, device=runtime.device)
+                                        for b in biases]).contiguous()
+        self.b_down = tensors.get("down_bias")
+        if self.activation != "clamped_swiglu" and (self.b_gate_up is not None or self.b_down is not None):
+            raise Unsupported(f"gated_mlp: biases go with clamped_swiglu, not with {self.activation}")
         self.spec = spec
         self.rt = runtime
         self.w_gate_up = torch.cat([tensors["gate"], tensors["up"]], dim=0).contiguous()
@@ -47,6 +61,9 @@ class GatedMLP:
         s, rt = self.spec, self.rt
         if x.shape[0] <= ops.SKINNY_FAST_ROWS:
             ops.stream_ahead(self.w_down)              # taken by the gate | up product, read by the product after it
+        if self.activation == "clamped_swiglu":
+            act = linear_clamped_swiglu(x, self.w_gate_up, self.b_gate_up, float(s.limit), float(s.gate_scale), rt, s.inner)
+            return linear_partial_biased(act, self.w_down, self.b_down, rt, "ffn_out")
         if self.activation == "gelu_tanh":
             act = linear_geglu(x, self.w_gate_up, rt, s.inner)
         else:

@@ -2,7 +2,7 @@
 
 Every token uses `top` of `experts` small feed-forward layers without biases, expert j being down_j(act(up_j x))
 (activation "relu2") or down_j(silu(gate_j x) * up_j x) (activation "swiglu"). The router's logits z = W_router x are
-float32; scores are their softmax over ALL experts, or with scores "sigmoid" the sigmoid of each. Choice scores are the
+float32 (with `biased` plus a number per expert); scores are their softmax over ALL experts, or with scores "sigmoid" the sigmoid of each. Choice scores are the
 scores, with `corrected` plus a number per expert. Experts form `groups` equal groups of neighbours, a group's score is its
 largest choice score, or with group_score "top2" the sum of its two largest, and only experts of the `keep_groups` best
 groups can be chosen; of those the `top` with the largest choice scores are. Their weights are their scores (without the
@@ -18,8 +18,8 @@ tile's expert (`moe_linear`: the activation sits in the first one's epilogue, th
 Another product over the same input can ride with the router's (`join_input`), whose results are float32 then too.
 
 Parameters: inner, experts, top, groups, keep_groups, weight_scale, activation ("relu2", "swiglu"), scores, group_score,
-renormalize, corrected, shared_inner. Tensors: router [experts, width], up<j> [inner, width], down<j> [width, inner], and by
-the parameters gate<j> [inner, width], correction [experts], shared_gate, shared_up [shared_inner, width], shared_down
+renormalize, corrected, biased, shared_inner. Tensors: router [experts, width], up<j> [inner, width], down<j> [width, inner], and by
+the parameters gate<j> [inner, width], correction [experts], router_bias [experts], shared_gate, shared_up [shared_inner, width], shared_down
 [width, shared_inner], shared_sg [1, width].
 """
 
@@ -45,6 +45,8 @@ class RoutedMLP:
         out = {"router": TensorDecl((spec.experts, spec.width))}
         if spec.get("corrected", False):
             out["correction"] = TensorDecl((spec.experts,), role="vector", init="bias")
+        if spec.get("biased", False):
+            out["router_bias"] = TensorDecl((spec.experts,), role="vector", init="bias")
         shared = int(spec.get("shared_inner", 0))
         if shared > 0:
             out.update(shared_gate=TensorDecl((shared, spec.width)), shared_up=TensorDecl((shared, spec.width)),
@@ -71,6 +73,7 @@ class RoutedMLP:
         self.route = dict(scores=spec.get("scores", "softmax"), group_score=spec.get("group_score", "max"),
                           renormalize=bool(spec.get("renormalize", True)))
         self.correction = tensors.get("correction")
+        self.router_bias = tensors.get("router_bias")
         self.shared = int(spec.get("shared_inner", 0))
         # everything that wants float32 results of the layer's input in one product: [router | shared expert's gate | rider],
         # padded to a multiple of 8 rows
@@ -117,7 +120,7 @@ class RoutedMLP:
         linear(x, self.w_router, logits)                                  # float32 accumulation and result
         ids = rt.buffer("moe_ids", (rows, top), torch.int32)
         weights = rt.buffer("moe_weights", (rows, top), torch.float32)
-        ops.moe_route(logits[:, :E], top, self.groups, self.keep, self.scale, ids, weights, self.correction, **self.route)
+        ops.moe_route(logits[:, :E], top, self.groups, self.keep, self.scale, ids, weights, self.correction, bias=self.router_bias, **self.route)
         most = rt.max_tokens * top
         place_of = rt.flat(f"moe_place_of_{top}", most, torch.int32)
         pair_at = rt.flat(f"moe_pair_at_{top}", most, torch.int32)

@@ -9,6 +9,8 @@ frequencies are made here in 32-bit floats exactly as the reference makes them,
 of a vector form a pair that turns by position * theta^(-2i / rotary_dim). The frequencies are kept in double
 precision and the kernels form the angle in double precision (csrc/latent_attention.cu), so the rotation is exact to
 float32 at any position; the mixer that uses it asks for `frequencies` (and `magnitude`, a factor on the turned numbers).
+"rotary_halves": the same precision for the half-split layout: numbers i and i + rotary_dim / 2 form a pair. A mixer whose
+kernels turn neighbours only may reorder its rows with `neighbours()` (queries and keys alike: their products stay).
 "none": no position encoding.
 
 A further kind implements `table()` returning None and `apply(q, k, positions)` rotating its views in
@@ -88,6 +90,19 @@ class InterleavedRotaryEncoding:
 
     def table(self):
         return None
+
+
+@register_position("rotary_halves")
+class HalvesRotaryEncoding(InterleavedRotaryEncoding):
+    interleaved = False
+    halves = True
+
+    def neighbours(self, size: int) -> torch.Tensor:
+        """The order of a vector's `size` numbers in which the two of a pair stand side by side: 0, h, 1, h + 1, ... (h =
+        rotary_dim / 2), then the numbers that are not turned."""
+        half = self.rotary_dim // 2
+        turned = torch.arange(self.rotary_dim).view(2, half).t().reshape(-1)
+        return torch.cat([turned, torch.arange(self.rotary_dim, size)])
 
 
 @register_position("none")

@@ -1,6 +1,8 @@
 """Two mixers side by side: the "side_by_side" mixer.
 
-Both read the same input; the result is left_scale * left(h) + right_scale * right(h), summed in float32. The two are
+Both read the same input; the result is left_scale * left(h) + right_scale * right(h), summed in float32; with `normed` each
+of the two is first divided by its root mean square over the width (eps) and multiplied by a weight of its own (tensors
+left_norm, right_norm [width]). The two are
 mixers in their own right, given as MixerSpecs in the parameters `left` and `right`; their tensors are declared under
 "left.<name>" and "right.<name>". One of them may keep pages and the other a state row (attention beside a
 recurrence): the pair then asks for pages that carry a state row (CacheSpec.state_shape on a spec of kind "pages"), and
@@ -29,6 +31,8 @@ class SideBySideMixer:
             sub = getattr(spec, side)
             for local, decl in MIXERS.get(sub.kind).declare(sub).items():
                 out[f"{side}.{local}"] = decl
+            if spec.get("normed", False):
+                out[f"{side}_norm"] = TensorDecl((spec.width,), role="vector", init="around_one")
         return out
 
     def __init__(self, spec, tensors: Dict[str, torch.Tensor], runtime):
@@ -44,6 +48,9 @@ class SideBySideMixer:
             setattr(self, side, part)
         self.left_scale = float(spec.get("left_scale", 1.0))
         self.right_scale = float(spec.get("right_scale", 1.0))
+        self.normed = bool(spec.get("normed", False))
+        self.left_norm, self.right_norm = tensors.get("left_norm"), tensors.get("right_norm")
+        self.eps = float(spec.get("eps", 1e-6))
         self.replay_safe = all(getattr(getattr(self, s), "replay_safe", False) for s in SIDES)
         self.graph_safe = all(getattr(getattr(self, s), "graph_safe", False) for s in SIDES)
         specs = [getattr(self, s).cache_spec() for s in SIDES]
@@ -88,5 +95,8 @@ class SideBySideMixer:
         a = self.left.forward(x, ctx, self._share(cache, self._kinds[0]), owns_cache)
         b = self.right.forward(x, ctx, self._share(cache, self._kinds[1]), owns_cache)
         out = self.rt.buffer("pair_out", (x.shape[0], self.spec.width), torch.float32)
-        ops.scaled_sum(a, self.left_scale, b, self.right_scale, out)
+        if self.normed:
+            ops.normed_sum(a, self.left_norm, self.left_scale, b, self.right_norm, self.right_scale, self.eps, out)
+        else:
+            ops.scaled_sum(a, self.left_scale, b, self.right_scale, out)
         return out
