@@ -487,6 +487,42 @@ def sipelorn_pair(name):
     return sipelorn, bugapel
 
 
+# --workload nisotar: the Nisotar design (latent attention with a window, windowed attention normed head by head, and pairs of
+# chunked attention and a delta rule with a decay per key channel; a mixture of gated experts) beside Sipelorn, the closest
+# design here (the same latent attention, attention and experts' kernels), at equal width and depth: the weights a token's
+# feed-forward uses are Sipelorn's (two gated experts of 2 ff / 3 against two of ff / 2 and a shared one of ff / 3; in the
+# layer with latent attention a gated one of 4 ff / 3 against an ungated one of 2 ff).
+NISOTAR_SIZES = {
+    # name: (width, layer kinds (l: latent attention, p: pair, a: windowed attention), attention (heads, kv_heads, dim, vdim,
+    #        turned, window or chunk), latent (heads, dim, rot_dim, vdim, kv_rank, window), delta (heads, kv_heads, dim, vdim,
+    #        taps, inner size), sipelorn size)
+    "w2048_d128": (2048, "lpap", (16, 4, 128, 128, 128, 1024), (16, 128, 64, 128, 512, 1024), (16, 16, 128, 128, 4, 128),
+                   "w2048_d128"),
+    "w4096_d128": (4096, "lp", (32, 8, 128, 128, 128, 2048), (32, 128, 64, 128, 512, 2048), (32, 16, 128, 128, 4, 128),
+                   "w4096_d128"),
+    "w2048_d64": (2048, "lpap", (32, 8, 64, 64, 32, 512), (32, 64, 32, 64, 256, 512), (32, 8, 64, 64, 4, 64), "w2048_d64"),
+}
+
+
+def nisotar_pair(name):
+    width, kinds, a, l, d, sip = NISOTAR_SIZES[name]
+    x = BUGAPEL_SIZES[SIPELORN_SIZES[sip][6]][4]
+    stretch = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    att = {"heads": a[0], "kv_heads": a[1], "dim": a[2], "vdim": a[3], "scale": a[2] ** -0.5, "mask": {"size": a[5]}}
+    delta = {"heads": d[0], "kv_heads": d[1], "dim": d[2], "vdim": d[3], "conv": d[4], "decay_rank": d[5], "gate_rank": d[5]}
+    lat = {"heads": l[0], "dim": l[1], "rot_dim": l[2], "vdim": l[3], "kv_rank": l[4], "scale": (l[1] + l[2]) ** -0.5,
+           "mask": {"size": l[5]}, "rot": {"base": 10000.0, "dims": l[2]}}
+    mixers = {"l": ("latent_attention", lat),
+              "a": ("attention", dict(att, rot={"base": 50000.0, "dims": a[4], "scaling": stretch})),
+              "p": ("parallel", {"left": dict(att, rot={"base": 500000.0, "dims": a[4]}), "right": delta})}
+    moe = {"kind": "moe", "expert": {"ff": 2 * x[4] // 3}, "router": {"experts": x[0], "top": x[1]}}
+    dense = {"kind": "dense", "ff": 4 * x[4] // 3, "limit": 7.0}
+    nisotar = {"architecture": "Nisotar", "vocab": ARCH_VOCAB, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+               "layers": [{"type": mixers[k][0], "mixer": mixers[k][1], "mlp": dense if k == "l" else moe} for k in kinds]}
+    sipelorn, _ = sipelorn_pair(sip)
+    return nisotar, sipelorn
+
+
 def arch_compare(args, kernels: bool, design: str = "todupel"):
     """Prefill (one prompt of 2,048 tokens) and decode (batches of 8 and 64 holding 2,048 tokens each) of a design
     and of the model it is set beside (the Llama shape, or Rematar for Rodelorn) at equal size, timed with CUDA events; with `kernels`, instead, the device time of every kernel
@@ -502,9 +538,9 @@ def arch_compare(args, kernels: bool, design: str = "todupel"):
     peaks = load_peaks()
     T, HELD_HERE, K = 2048, 2048, max(8, min(args.steps, 64))
     sizes = {"todupel": ARCH_SIZES, "rematar": REMATAR_SIZES, "rodelorn": RODELORN_SIZES, "bugapel": BUGAPEL_SIZES,
-             "sipelorn": SIPELORN_SIZES}[design]
-    other = {"rodelorn": "rematar", "bugapel": "rodelorn", "sipelorn": "bugapel"}.get(design, "llama")
-    beside = {"rematar": "Rematar", "rodelorn": "Rodelorn", "bugapel": "Bugapel", "llama": "the Llama shape"}[other]
+             "sipelorn": SIPELORN_SIZES, "nisotar": NISOTAR_SIZES}[design]
+    other = {"rodelorn": "rematar", "bugapel": "rodelorn", "sipelorn": "bugapel", "nisotar": "sipelorn"}.get(design, "llama")
+    beside = {"rematar": "Rematar", "rodelorn": "Rodelorn", "bugapel": "Bugapel", "sipelorn": "Sipelorn", "llama": "the Llama shape"}[other]
     out = {"metric": f"{design.capitalize()} beside {beside} of equal size: prefill and decode tokens/s", "unit": "tokens/s",
            "n_gpus": 1, "dtype": "bf16", "data": "synthetic: random weights, random token ids", "peaks": peaks,
            "config": {"prefill_tokens": T, "decode_context": HELD_HERE, "decode_steps": K, "vocab": ARCH_VOCAB,
@@ -532,6 +568,11 @@ def arch_compare(args, kernels: bool, design: str = "todupel"):
             rec = {"shape": {"width": width, "layers": kinds, "attention": list(a), "latent_attention": list(l),
                              "token_side": side, "token_pairs": buckets, "bugapel": bug}}
             pair = sipelorn_pair(size)
+        elif design == "nisotar":
+            width, kinds, a, l, d, sip = NISOTAR_SIZES[size]
+            rec = {"shape": {"width": width, "layers": kinds, "attention": list(a), "latent_attention": list(l), "delta": list(d),
+                             "sipelorn": sip}}
+            pair = nisotar_pair(size)
         else:
             width, kinds, d, a, r, ff, rem = RODELORN_SIZES[size]
             rec = {"shape": {"width": width, "layers": kinds, "delta": list(d), "attention": list(a), "recurrence": list(r),
@@ -611,10 +652,10 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=FULL_LAYERS, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--batch", type=int, default=8)
-    ap.add_argument("--workload", choices=["decode", "todupel", "todupel-kernels", "rematar", "rematar-kernels", "rodelorn", "rodelorn-kernels", "bugapel", "bugapel-kernels", "sipelorn", "sipelorn-kernels"] + sorted(SERVING), default="decode",
+    ap.add_argument("--workload", choices=["decode", "todupel", "todupel-kernels", "rematar", "rematar-kernels", "rodelorn", "rodelorn-kernels", "bugapel", "bugapel-kernels", "sipelorn", "sipelorn-kernels", "nisotar", "nisotar-kernels"] + sorted(SERVING), default="decode",
                     help="decode: the default benchmark; serve3b / serve8b: continuous batching of the 3B / 8B workloads; "
                          "todupel / rematar: that design beside the Llama shape of equal size; rodelorn: that design beside Rematar of "
-                         "equal size; bugapel: that design beside Rodelorn of equal size; sipelorn: that design beside Bugapel of equal size (<design>-kernels: per kernel)")
+                         "equal size; bugapel: that design beside Rodelorn of equal size; sipelorn: that design beside Bugapel of equal size; nisotar: that design beside Sipelorn of equal size (<design>-kernels: per kernel)")
     ap.add_argument("--no-points", action="store_true", help="skip decode at batch 1 and 64")
     ap.add_argument("--no-long", action="store_true", help="skip the points at 8,192 tokens (prefill and decode)")
     ap.add_argument("--no-serve", action="store_true", help="skip the points of the 3B and 8B serving workloads")
@@ -629,7 +670,7 @@ def main():
     if args.gpus != 1:
         print(f"bench.py: this engine runs on one GPU; --gpus {args.gpus} is not supported")
         return 2
-    if args.workload.split("-")[0] in ("todupel", "rematar", "rodelorn", "bugapel", "sipelorn"):
+    if args.workload.split("-")[0] in ("todupel", "rematar", "rodelorn", "bugapel", "sipelorn", "nisotar"):
         return arch_compare(args, kernels=args.workload.endswith("-kernels"), design=args.workload.split("-")[0])
     if args.workload != "decode":
         return serving(args.workload, args.layers if args.layers != FULL_LAYERS else None)

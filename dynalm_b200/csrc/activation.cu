@@ -107,16 +107,17 @@ __global__ void xielu_vec_kernel(const T* __restrict__ x, T* __restrict__ out, c
 }
 
 // A gated activation whose halves are clamped: with g = min(gate + bias, limit), u = clamp(up + bias, -limit, limit),
-// g sigmoid(gate_scale g) (u + 1). bias: float32 [2 * inner] over [gate | up], or null.
+// g sigmoid(gate_scale g) (u + 1). coeffs: as common.cuh says at CLAMPED_HEADER.
 template <typename T, int V>
-__global__ void clamped_swiglu_kernel(const T* __restrict__ gu, const float* __restrict__ bias, float limit, float gate_scale,
-                                      T* __restrict__ out, int rows, int inner) {
+__global__ void clamped_swiglu_kernel(const T* __restrict__ gu, const float* __restrict__ coeffs, T* __restrict__ out, int rows,
+                                      int inner) {
   const size_t idx = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   const int per = inner / V;
   if (idx >= static_cast<size_t>(rows) * per) return;
   const size_t t = idx / per;
   const int j = static_cast<int>(idx % per) * V;
   const T* row = gu + t * 2 * inner + j;
+  const float* bias = coeffs + CLAMPED_HEADER;
   float g[V], u[V];
   if constexpr (V > 1) {
     unpack<T>(*reinterpret_cast<const Vec16*>(row), g);
@@ -127,11 +128,7 @@ __global__ void clamped_swiglu_kernel(const T* __restrict__ gu, const float* __r
   }
 #pragma unroll
   for (int k = 0; k < V; ++k) {
-    if (bias != nullptr) {
-      g[k] += bias[j + k];
-      u[k] += bias[inner + j + k];
-    }
-    g[k] = clamped_swiglu_f(g[k], u[k], limit, gate_scale);
+    g[k] = clamped_swiglu_f(g[k] + bias[j + k], u[k] + bias[inner + j + k], coeffs[0], coeffs[1]);
   }
   if constexpr (V > 1) *reinterpret_cast<Vec16*>(out + t * inner + j) = pack<T>(g);
   else out[t * inner + j] = from_float<T>(g[0]);
@@ -212,18 +209,17 @@ DL_EXPORT int dl_silu_mul(int dtype, const void* gu, void* out, int rows, int in
   return dl::launch_status();
 }
 
-// gu: contiguous [rows, 2 * inner] = [gate | up]; bias: float32 [2 * inner] or null; out: contiguous [rows, inner].
-DL_EXPORT int dl_clamped_swiglu(int dtype, const void* gu, const float* bias, float limit, float gate_scale, void* out, int rows,
-                                int inner, cudaStream_t stream) {
+// gu: contiguous [rows, 2 * inner] = [gate | up]; coeffs: float32 [4 + 2 * inner]; out: contiguous [rows, inner].
+DL_EXPORT int dl_clamped_swiglu(int dtype, const void* gu, const float* coeffs, void* out, int rows, int inner,
+                                cudaStream_t stream) {
   if (rows <= 0 || inner <= 0) return 0;
-  if ((dtype != 0 && dtype != 1) || !(limit > 0.0f)) return DL_ERR_UNSUPPORTED;
+  if ((dtype != 0 && dtype != 1) || coeffs == nullptr) return DL_ERR_UNSUPPORTED;
   const int vec = dtype == 0 ? 4 : 8;
   const bool wide = inner % vec == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   const size_t n = static_cast<size_t>(rows) * (wide ? inner / vec : inner);
   const unsigned blocks = static_cast<unsigned>((n + 255) / 256);
 #define DL_CS(T, V)                                                                                                     \
-  dl::clamped_swiglu_kernel<T, V><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gu), bias, limit, gate_scale,       \
-                                                              static_cast<T*>(out), rows, inner)
+  dl::clamped_swiglu_kernel<T, V><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gu), coeffs, static_cast<T*>(out), rows, inner)
   if (dtype == 0) { if (wide) DL_CS(float, 4); else DL_CS(float, 1); }
   else { if (wide) DL_CS(dl::bf16, 8); else DL_CS(dl::bf16, 1); }
 #undef DL_CS

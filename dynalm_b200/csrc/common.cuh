@@ -148,6 +148,17 @@ __device__ __forceinline__ float clamped_swiglu_f(float g, float u, float limit,
   return g / (1.0f + expf(-scale * g)) * (u + 1.0f);
 }
 
+// The same for results that are rounded to bf16 right away, with the fast exponential and division.
+__device__ __forceinline__ float clamped_swiglu_bf16(float g, float u, float limit, float scale) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.0f + __expf(-scale * g)) * (u + 1.0f);
+}
+
+// What the products' SwiGLU epilogue reads beside the sums when its halves are clamped: [limit, gate scale, 0, 0 | a bias for
+// every gate feature | a bias for every up feature], float32 on the device.
+constexpr int CLAMPED_HEADER = 4;
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // Programmatic dependent launch. A kernel launched with the attribute may begin while the kernel before it on

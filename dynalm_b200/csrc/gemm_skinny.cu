@@ -196,8 +196,14 @@ gemm_skinny_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__
         gate += red[(static_cast<size_t>(wv) * FT + mt * 16 + i) * BT + b];
         up += red[(static_cast<size_t>(wv) * FT + mt * 16 + 8 + i) * BT + b];
       }
-      const float s = gate / (1.0f + expf(-gate));
-      static_cast<bf16*>(y)[static_cast<size_t>(b) * ldy + j] = __float2bfloat16_rn(s * up);
+      float v;
+      if (coeffs != nullptr) {           // clamped halves with biases
+        v = clamped_swiglu_bf16(gate + coeffs[CLAMPED_HEADER + j], up + coeffs[CLAMPED_HEADER + half + j], coeffs[0], coeffs[1]);
+      } else {
+        const float s = gate / (1.0f + expf(-gate));
+        v = s * up;
+      }
+      static_cast<bf16*>(y)[static_cast<size_t>(b) * ldy + j] = __float2bfloat16_rn(v);
     }
     return;
   }
@@ -339,7 +345,8 @@ int launch_skinny(const void* x, int ldx, const void* w, void* y, int ldy, int M
 
 // x: bf16 [M, K] rows of ldx elements (16-byte aligned rows), w: bf16 [N, K] contiguous, K a multiple of 8,
 // M <= 64. mode 0: y bf16 [M, N]; mode 1: y fp32, n_split partial results of [M, ldy] floats each,
-// split_stride floats apart; mode 2: w = [gate; up] (N even), y bf16 [M, N / 2] = silu(x Wg^T) * (x Wu^T).
+// split_stride floats apart; mode 2: w = [gate; up] (N even), y bf16 [M, N / 2] = silu(x Wg^T) * (x Wu^T), or with coeffs (N +
+// 4 float32: common.cuh, CLAMPED_HEADER) the gated activation with clamped halves and biases.
 // mode 4: y bf16 [M, N] = max(x W^T, 0)^2; mode 6: = xIELU(x W^T) with coeffs = two float32 on the device. mode 3: nothing but the place of each row's largest output leaves the kernel: y = float [M][blocks] then
 // int [M][blocks] (blocks = ceil(N / features per block), see dl_gemm_skinny_argmax_blocks), the largest value of every
 // block's features and its feature index (the lowest among equals); out_scale must be positive.

@@ -223,13 +223,22 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
         epilogue_sync();
         if (f0 + feat < gate_rows) {
           bf16* out = static_cast<bf16*>(y) + f0 + feat;
+          float limit = 0.0f, gate_scale = 0.0f, bias_g = 0.0f, bias_u = 0.0f;
+          if (coeffs != nullptr) {             // clamped halves with biases
+            limit = coeffs[0];
+            gate_scale = coeffs[1];
+            bias_g = coeffs[CLAMPED_HEADER + f0 + feat];
+            bias_u = coeffs[CLAMPED_HEADER + gate_rows + f0 + feat];
+          }
 #pragma unroll
           for (int b = 0; b < HALF; ++b) {
             const int col = is_gate ? b : HALF + b;
             if (col < M) {
               const float other = exchange[col * 64 + feat];
               const float g = is_gate ? acc[b] : other, u = is_gate ? other : acc[HALF + b];
-              out[static_cast<size_t>(col) * ldy] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * u);
+              const float v = coeffs != nullptr ? clamped_swiglu_bf16(g + bias_g, u + bias_u, limit, gate_scale)
+                                                : __fdividef(g, 1.0f + __expf(-g)) * u;
+              out[static_cast<size_t>(col) * ldy] = __float2bfloat16_rn(v);
             }
           }
         }
@@ -302,7 +311,8 @@ static int gs_run(const void* x, int ldx, const void* w, void* y, int ldy, int M
 
 // x: bf16 [M, K] (M <= 64) rows of ldx elements; w: bf16 [N, K] contiguous; both 16-byte aligned, K and ldx multiples
 // of 8. mode 0: y bf16 [M, N]; mode 1: y fp32, n_split partial results of [M, ldy] floats each, split_stride floats
-// apart (n_split > 1 needs this mode); mode 2: w = [gate; up] with N = 2F rows, y bf16 [M, F] = silu(x Wg^T) * (x Wu^T).
+// apart (n_split > 1 needs this mode); mode 2: w = [gate; up] with N = 2F rows, y bf16 [M, F] = silu(x Wg^T) * (x Wu^T), or
+// with coeffs (N + 4 float32: common.cuh, CLAMPED_HEADER) the gated activation with clamped halves and biases.
 // status: one device int, set to a nonzero code if a wait inside the kernel timed out (left untouched otherwise).
 DL_EXPORT int dl_gemm_stream(const void* x, int ldx, const void* w, void* y, int ldy, int M, int N, int K, int mode,
                              float out_scale, int n_split, long long split_stride, const float* coeffs, int* status,

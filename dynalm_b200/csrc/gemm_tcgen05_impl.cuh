@@ -253,7 +253,39 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
       const uint32_t lane_addr = tmem_base + buf * T5_BN + (static_cast<uint32_t>(quarter * 32) << 16);
       unsigned char* my_stage = store_stage + (warp - 2) * (T5_STORE_BYTES / 4);
       const int row0 = m0 + quarter * 32;
-      if (swiglu) {
+      if (swiglu && coeffs != nullptr) {
+        // clamped halves with biases: a branch of its own, so that the plain epilogue stays as small as it was
+        const float limit = coeffs[0], gate_scale = coeffs[1];
+        const float* bias_g = coeffs + CLAMPED_HEADER;
+        const float* bias_u = bias_g + gate_rows;            // (gate_rows is a multiple of 8)
+        for (int c0 = 0; c0 < T5_BN / 2; c0 += 64) {
+          uint4 w[8];
+#pragma unroll 1
+          for (int hh = 0; hh < 2; ++hh) {
+            uint32_t g[32], u[32];
+            tmem_ld32(lane_addr + c0 + hh * 32, g);
+            tmem_ld32(lane_addr + T5_BN / 2 + c0 + hh * 32, u);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+              const int f = n0 + c0 + hh * 32 + j;
+              uint4 q = make_uint4(0u, 0u, 0u, 0u);
+              if (f < gate_rows) {
+                const float4 ga = *reinterpret_cast<const float4*>(bias_g + f), gb = *reinterpret_cast<const float4*>(bias_g + f + 4);
+                const float4 ua = *reinterpret_cast<const float4*>(bias_u + f), ub = *reinterpret_cast<const float4*>(bias_u + f + 4);
+                auto fin = [&](int e, float bg, float bu) {
+                  return clamped_swiglu_bf16(__uint_as_float(g[j + e]) + bg, __uint_as_float(u[j + e]) + bu, limit, gate_scale);
+                };
+                q = make_uint4(pack2_bf16(fin(0, ga.x, ua.x), fin(1, ga.y, ua.y)), pack2_bf16(fin(2, ga.z, ua.z), fin(3, ga.w, ua.w)),
+                               pack2_bf16(fin(4, gb.x, ub.x), fin(5, gb.y, ub.y)), pack2_bf16(fin(6, gb.z, ub.z), fin(7, gb.w, ub.w)));
+              }
+              if (hh == 0) w[j / 8] = q;
+              else w[4 + j / 8] = q;
+            }
+          }
+          store_rows_bf16(w, my_stage, lane, static_cast<bf16*>(y), ldy, row0, M, n0 + c0, gate_rows);
+        }
+      } else if (swiglu) {
         bf16* out = static_cast<bf16*>(y);
         for (int c0 = 0; c0 < T5_BN / 2; c0 += 64) {
           uint4 w[8];
@@ -472,7 +504,8 @@ static inline int make_map(CUtensorMap* map, const void* base, int rows, int col
 
 // x: bf16 [M, K] rows of ldx elements; w: bf16 [N, K] contiguous; both 16-byte aligned with K and ldx multiples of 8.
 // mode 0: y bf16 [M, N] (N % 8 == 0); mode 1: y fp32 [M, N] (N % 4 == 0); mode 2: w = [gate; up] with N = 2F rows,
-// y bf16 [M, F] = silu(x Wg^T) * (x Wu^T) (F % 8 == 0); mode 4: y bf16 [M, N] = max(x W^T, 0)^2; mode 5: = gelu_tanh(x W^T);
+// y bf16 [M, F] = silu(x Wg^T) * (x Wu^T) (F % 8 == 0), or with coeffs (N + 4 float32, 16-byte aligned: common.cuh,
+// CLAMPED_HEADER) the gated activation with clamped halves and biases; mode 4: y bf16 [M, N] = max(x W^T, 0)^2; mode 5: = gelu_tanh(x W^T);
 // mode 7: = xIELU(x W^T) with coeffs = two float32 on the device. status: one device int, set to a nonzero code if a wait
 // inside the kernel timed out (left untouched otherwise).
 template <class P>
@@ -482,6 +515,7 @@ static int t5_launch(const void* x, int ldx, const void* w, void* y, int ldy, in
   if (K <= 0 || (K & 7) || (ldx & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15) ||
       status == nullptr || mode < 0 || (mode > 5 && mode != dl::T5_OUT_XIELU) || (mode == dl::T5_OUT_XIELU && coeffs == nullptr))
     return DL_ERR_UNSUPPORTED;
+  if (mode == dl::T5_OUT_SWIGLU && (reinterpret_cast<uintptr_t>(coeffs) & 15)) return DL_ERR_UNSUPPORTED;
   const int feats = mode == dl::T5_OUT_SWIGLU ? N / 2 : N;
   if ((mode == dl::T5_OUT_SWIGLU && (N & 1)) || (mode == dl::T5_OUT_F32 ? (feats & 3) || (ldy & 3) : (feats & 7) || (ldy & 7)) ||
       (reinterpret_cast<uintptr_t>(y) & 15))

@@ -186,19 +186,28 @@ def linear_partial_biased(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch
     return out
 
 
+def _gated_epilogue(x: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, inner: int, coeffs: Optional[torch.Tensor] = None) -> bool:
+    """act = the gated activation of x [Wg; Wu]^T in the epilogue of one of this package's bfloat16 products; False when none
+    of them takes the product."""
+    if x.dtype != torch.bfloat16:
+        return False
+    if use_stream(x, w_gate_up):
+        ops.gemm_stream(x, w_gate_up, act, "swiglu", coeffs=coeffs)
+    elif skinny_ok(x, w_gate_up):
+        ops.gemm_skinny(x, w_gate_up, act, "swiglu", coeffs=coeffs)
+    elif inner % 8 == 0 and w_gate_up.shape[0] == 2 * inner and tcgen05_ok(x, w_gate_up, act, 2 * inner):
+        ops.gemm_tcgen05(x, w_gate_up, act, "swiglu", coeffs=coeffs)
+    else:
+        return False
+    return True
+
+
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, runtime, inner: int) -> torch.Tensor:
-    """silu(x Wg^T) * (x Wu^T) with w_gate_up = [Wg; Wu]: fused in the product's epilogue for few
-    bfloat16 rows, else the product followed by the activation kernel."""
+    """silu(x Wg^T) * (x Wu^T) with w_gate_up = [Wg; Wu]: fused in the product's epilogue wherever one of this package's
+    bfloat16 kernels runs the product, else the product followed by the activation kernel."""
     rows = x.shape[0]
     act = runtime.buffer("ffn_act", (rows, inner))
-    if x.dtype == torch.bfloat16 and use_stream(x, w_gate_up):
-        ops.gemm_stream(x, w_gate_up, act, "swiglu")
-        return act
-    if x.dtype == torch.bfloat16 and skinny_ok(x, w_gate_up):
-        ops.gemm_skinny(x, w_gate_up, act, "swiglu")
-        return act
-    if x.dtype == torch.bfloat16 and inner % 8 == 0 and w_gate_up.shape[0] == 2 * inner and tcgen05_ok(x, w_gate_up, act, 2 * inner):
-        ops.gemm_tcgen05(x, w_gate_up, act, "swiglu")
+    if _gated_epilogue(x, w_gate_up, act, inner):
         return act
     gate_up = runtime.buffer("ffn_gate_up", (rows, 2 * inner))
     linear(x, w_gate_up, gate_up)
@@ -206,14 +215,16 @@ def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, runtime, inner: int)
     return act
 
 
-def linear_clamped_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, bias: Optional[torch.Tensor], limit: float, gate_scale: float,
-                          runtime, inner: int) -> torch.Tensor:
-    """With [g | u] = x [Wg; Wu]^T + bias: min(g, limit) sigmoid(gate_scale min(g, limit)) (clamp(u, -limit, limit) + 1)."""
+def linear_clamped_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, coeffs: torch.Tensor, runtime, inner: int) -> torch.Tensor:
+    """With [g | u] = x [Wg; Wu]^T + bias: min(g, limit) sigmoid(gate_scale min(g, limit)) (clamp(u, -limit, limit) + 1), where
+    linear_swiglu puts its activation; `coeffs`: ops.clamped_coeffs(limit, gate_scale, bias, ...)."""
     rows = x.shape[0]
     act = runtime.buffer("ffn_act", (rows, inner))
+    if _gated_epilogue(x, w_gate_up, act, inner, coeffs):
+        return act
     gate_up = runtime.buffer("ffn_gate_up", (rows, 2 * inner))
     linear(x, w_gate_up, gate_up)
-    ops.clamped_swiglu(gate_up, bias, limit, gate_scale, act)
+    ops.clamped_swiglu(gate_up, coeffs, act)
     return act
 
 

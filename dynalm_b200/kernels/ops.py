@@ -36,7 +36,7 @@ _SIGNATURES = {
     },
     "activation": {"dl_silu_mul": [_I, _P, _P, _I, _I, _P], "dl_relu2": [_I, _P, _P, _L, _P],
                    "dl_gelu_tanh": [_I, _P, _P, _L, _P], "dl_xielu": [_I, _P, _P, _P, _L, _P],
-                   "dl_clamped_swiglu": [_I, _P, _P, _F, _F, _P, _I, _I, _P]},
+                   "dl_clamped_swiglu": [_I, _P, _P, _P, _I, _I, _P]},
     "norm_after_sum": {
         "dl_norm_after_sum": [_I, _I, _P, _P, _I, _L, _P, _F, _P, _F, _P, _I, _I, _P],
         "dl_cast_rows": [_I, _P, _P, _L, _P]},
@@ -1364,8 +1364,22 @@ SKINNY_MAX_ROWS = 64      # what the kernel takes
 SKINNY_FAST_ROWS = int(os.environ.get("DYNALM_SKINNY_ROWS", "16"))     # up to here the dispatchers use it (measured on B200)
 
 
-def _xielu_coeffs(mode: str, coeffs: Optional[torch.Tensor]) -> None:
-    if (mode == "xielu") != (coeffs is not None) or (coeffs is not None and (coeffs.dtype != torch.float32 or coeffs.numel() != 2)):
+CLAMPED_HEADER = 4        # numbers in front of the biases (csrc/common.cuh)
+
+
+def clamped_coeffs(limit: float, gate_scale: float, bias: Optional[torch.Tensor], inner: int, device) -> torch.Tensor:
+    """What a product's "swiglu" epilogue takes as `coeffs` for halves that are clamped: [limit, gate_scale, 0, 0 | a bias for
+    every gate feature | for every up feature], float32 (`bias` None: zeros)."""
+    head = torch.tensor([limit, gate_scale, 0.0, 0.0], dtype=torch.float32, device=device)
+    return torch.cat([head, bias.float() if bias is not None else torch.zeros(2 * inner, dtype=torch.float32, device=device)]).contiguous()
+
+
+def _epilogue_coeffs(mode: str, coeffs: Optional[torch.Tensor], features: int) -> None:
+    """xielu takes its two coefficients, swiglu those of clamped halves (clamped_coeffs) or none."""
+    if mode == "swiglu":
+        if coeffs is not None and (coeffs.dtype != torch.float32 or coeffs.numel() != CLAMPED_HEADER + features or coeffs.data_ptr() % 16):
+            raise InvalidArgument("swiglu with clamped halves goes with clamped_coeffs on the device")
+    elif (mode == "xielu") != (coeffs is not None) or (coeffs is not None and (coeffs.dtype != torch.float32 or coeffs.numel() != 2)):
         raise InvalidArgument("xielu goes with its two float32 coefficients on the device")
     _cuda(coeffs)
 
@@ -1375,9 +1389,10 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str =
     """Weight-streaming product for at most 64 rows, bfloat16 operands; see csrc/gemm_skinny.cu.
 
     mode "store": out [M, N] bfloat16 or float32, or float32 [parts, M, N] to split K over `parts`
-    blocks (the consumer adds the parts); mode "swiglu": w = [gate; up], out [M, N/2] bfloat16; mode "relu2":
+    blocks (the consumer adds the parts); mode "swiglu": w = [gate; up], out [M, N/2] bfloat16 (with `coeffs` of
+    clamped_coeffs its halves are clamped); mode "relu2":
     out [M, N] bfloat16 = max(x W^T, 0)^2; "gelu_tanh" and "xielu" (with `coeffs`, see ops.xielu) likewise."""
-    _xielu_coeffs(mode, coeffs)
+    _epilogue_coeffs(mode, coeffs, w.shape[0])
     _cuda(x, w, out)
     _rows_contiguous(x, "x")
     M, K = x.shape
@@ -1416,7 +1431,7 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str 
     x [M, K] and w [N, K] bfloat16; out [M, N] bfloat16 or float32, or with mode "swiglu"
     (w = [gate; up]) out [M, N/2] bfloat16, or with mode "relu2" out [M, N] bfloat16 = max(x W^T, 0)^2; "gelu_tanh" and
     "xielu" (with `coeffs`, see ops.xielu) likewise."""
-    _xielu_coeffs(mode, coeffs)
+    _epilogue_coeffs(mode, coeffs, w.shape[0])
     _cuda(x, w, out)
     _rows_contiguous(x, "x")
     M, K = x.shape
@@ -1470,7 +1485,7 @@ def gemm_stream(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str =
     out [M, N] bfloat16 or float32; float32 [parts, M, N] (contiguous): K is split over `parts` blocks and each
     leaves its partial sums; mode "swiglu" (w = [gate; up]): out [M, N/2] bfloat16; mode "relu2": out [M, N] bfloat16 =
     max(x W^T, 0)^2; "gelu_tanh" and "xielu" (with `coeffs`, see ops.xielu) likewise."""
-    _xielu_coeffs(mode, coeffs)
+    _epilogue_coeffs(mode, coeffs, w.shape[0])
     _cuda(x, w, out)
     _rows_contiguous(x, "x")
     M, K = x.shape
@@ -2436,13 +2451,13 @@ def normed_sum(a: torch.Tensor, wa: torch.Tensor, sa: float, b: torch.Tensor, wb
                                                   pb, stride_b, _p(wb), sb, eps, _p(out), rows, width, _stream()), "normed_sum")
 
 
-def clamped_swiglu(gate_up: torch.Tensor, bias: Optional[torch.Tensor], limit: float, gate_scale: float, out: torch.Tensor) -> None:
-    """With [g | u] = gate_up + bias (float32 [2 * inner], or None): out = min(g, limit) sigmoid(gate_scale min(g, limit))
-    (clamp(u, -limit, limit) + 1)."""
-    _cuda(gate_up, bias, out)
+def clamped_swiglu(gate_up: torch.Tensor, coeffs: torch.Tensor, out: torch.Tensor) -> None:
+    """With [g | u] = gate_up + bias: out = min(g, limit) sigmoid(gate_scale min(g, limit)) (clamp(u, -limit, limit) + 1);
+    limit, gate_scale and the biases in `coeffs` (clamped_coeffs)."""
+    _cuda(gate_up, coeffs, out)
     rows, inner = out.shape
     if gate_up.shape != (rows, 2 * inner) or gate_up.dtype != out.dtype or not gate_up.is_contiguous() or not out.is_contiguous() \
-            or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != 2 * inner)):
+            or coeffs.dtype != torch.float32 or coeffs.numel() != CLAMPED_HEADER + 2 * inner:
         raise InvalidArgument("clamped_swiglu: gate_up contiguous [rows, 2 * inner], out contiguous [rows, inner], one dtype")
-    _check(_fn("activation", "dl_clamped_swiglu")(dtype_code(out.dtype), _p(gate_up), _p(bias), limit, gate_scale, _p(out), rows,
-                                                   inner, _stream()), "clamped_swiglu")
+    _check(_fn("activation", "dl_clamped_swiglu")(dtype_code(out.dtype), _p(gate_up), _p(coeffs), _p(out), rows, inner, _stream()),
+           "clamped_swiglu")

@@ -81,8 +81,8 @@ class GatedDeltaMixer:
         two_gate = int(spec.get("gate_rank", 0)) > 0
         # one product, [inner vectors | q | k | v | gate | b | a], the pieces that are there; the convolution runs over q, k
         # and v. The inner vectors stand in front and are padded, as is the whole, so that rows and slices start on 16 bytes.
-        first = [tensors["decay_in"]] * self.by_channel + [tensors["gate_in"]] * two_gate
-        second = [tensors["decay_out"]] * self.by_channel + [tensors["gate_out"]] * two_gate
+        steps = (["decay"] if self.by_channel else []) + (["gate"] if two_gate else [])
+        first, second = [tensors[n + "_in"] for n in steps], [tensors[n + "_out"] for n in steps]
         mats = [self._padded(first)] if first else []
         self.inner_cols = mats[0].shape[0] if first else 0
         mats += [tensors[n] for n in ("q", "k", "v")]

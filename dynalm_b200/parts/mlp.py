@@ -40,13 +40,15 @@ class GatedMLP:
         self.activation = spec.get("activation", "silu")
         if self.activation not in ("silu", "gelu_tanh", "clamped_swiglu"):
             raise Unsupported(f"gated_mlp: activation '{self.activation}' has no kernel (silu, gelu_tanh and clamped_swiglu do)")
-        self.b_gate_up = None
         biases = [tensors.get("gate_bias"), tensors.get("up_bias")]
-        if any(b is not None for b in biases):
-            self.b_gate_up = torch.cat([b if b is not None else torch.zeros(spec.inner, dtype=torch.float32, device=runtime.device)
-                                        for b in biases]).contiguous()
         self.b_down = tensors.get("down_bias")
-        if self.activation != "clamped_swiglu" and (self.b_gate_up is not None or self.b_down is not None):
+        self.coeffs = None
+        if self.activation == "clamped_swiglu":
+            # limit, scale and biases lie together in memory, where the products' epilogues read them
+            zeros = torch.zeros(spec.inner, dtype=torch.float32, device=runtime.device)
+            self.coeffs = ops.clamped_coeffs(float(spec.limit), float(spec.gate_scale),
+                                             torch.cat([b if b is not None else zeros for b in biases]), spec.inner, runtime.device)
+        elif any(b is not None for b in biases + [self.b_down]):
             raise Unsupported(f"gated_mlp: biases go with clamped_swiglu, not with {self.activation}")
         self.spec = spec
         self.rt = runtime
@@ -62,7 +64,7 @@ class GatedMLP:
         if x.shape[0] <= ops.SKINNY_FAST_ROWS:
             ops.stream_ahead(self.w_down)              # taken by the gate | up product, read by the product after it
         if self.activation == "clamped_swiglu":
-            act = linear_clamped_swiglu(x, self.w_gate_up, self.b_gate_up, float(s.limit), float(s.gate_scale), rt, s.inner)
+            act = linear_clamped_swiglu(x, self.w_gate_up, self.coeffs, rt, s.inner)
             return linear_partial_biased(act, self.w_down, self.b_down, rt, "ffn_out")
         if self.activation == "gelu_tanh":
             act = linear_geglu(x, self.w_gate_up, rt, s.inner)

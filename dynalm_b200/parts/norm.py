@@ -101,8 +101,7 @@ class LayerNorm:
                 delta_scale: float = 1.0, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """out = norm(residual + delta_scale * delta); the sum is written back to `residual` unless `rows` picks a
         subset."""
-        ops.stream_layer_norm(residual, 1, self.weight, self.bias, self.eps, out, delta=delta, delta_scale=delta_scale,
-                              rows=rows)
+        ops.residual_norm(residual, out, "layer", self.weight, self.bias, self.eps, delta=delta, delta_scale=delta_scale, rows=rows)
         return out
 
     def forward_update(self, stream, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
