@@ -13,47 +13,59 @@
 // q, k and v come from the short convolution's output (columns q | k | v of a row), b, a and the output gate from the
 // projection's row. What a request keeps is S of every head, float32 [H][d][e], at the head of its state row.
 //
+// Tokens are taken in runs of four. With S the state in front of a run, G_t the product of the run's decays up to token t
+// and D_st that from behind token s up to t,
+//
+//   u_t = beta_t (v_t - S^T (G_t k_t) - sum_{s<t} u_s (D_st k_s . k_t)),   o_t = S^T (G_t q_t) + sum_{s<=t} u_s (D_st k_s . q_t)
+//   S <- G_4 S + sum_s (D_s4 k_s) u_s^T
+//
+// so all dot products of a run over S are independent of one another, and what one token does to the next is a triangle of
+// four numbers a column; the sixteen dot products in brackets are the same for every column.
+//
 // Block = (slice of the e columns, head, request), 256 threads: four warps that compute and four that fetch.
 // A column of S lies over P neighbouring lanes of a computing warp, lane p holding the R rows p R .. p R + R - 1 in
-// registers; the two dot products of a token are finished by shuffles among those lanes. A request's tokens are
-// walked in tiles of 16 held twice in shared memory: while the computing warps run a tile's tokens over their
-// registers, the fetching warps write the next tile (queries and keys made unit vectors, a warp per token; the
-// values of the block's columns; the two gates; k . q) and ask for the one after it, whose numbers then have a whole
-// tile's time to arrive in their registers: no token waits for global memory. Both dot products of a
-// token run over the state it found (S'^T q = g S^T q + u (k . q)), so one round of shuffles a token is enough.
+// registers; a run's eight dot products are finished by shuffles among those lanes. A request's tokens are walked in tiles
+// of 16 (of 8 for heads of more than 256) held twice in shared memory: while the computing warps run a tile's runs over
+// their registers, each fetching warp writes a run of the next tile (queries and keys made unit vectors and multiplied by
+// their decays; the run's dot products; write strengths; the values of the block's columns) and asks for the one after it,
+// whose numbers then have a whole tile's time to arrive in its registers: no token waits for global memory. Tokens past a
+// tile's end are zeros with a decay of 1 and change nothing.
 // A lane's rows are R + 4 floats apart in shared memory, so that the P lanes' 16-byte loads fall into different banks.
-//
-// With a decay per channel the state is scaled first, S' = g S, and both dot products run over S'; g lies beside k and q.
 //
 // dl_head_norm_gate: out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * w * act(gate[t, h, :]), act silu or sigmoid.
 #include "common.cuh"
 
 namespace dl {
 
-constexpr int DR_TT = 16;
+constexpr int DR_RUN = 4;                               // tokens of a run
 constexpr int DR_COMPUTE = 128;
 constexpr int DR_THREADS = 256;
 
 __device__ __forceinline__ float dr_softplus(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 
-template <int R, int P, bool CH>
+template <int R, int P>
 struct DrTile {
+  static constexpr int TT = R * P > 256 ? 8 : 16;       // tokens of a tile
+  static constexpr int RUNS = TT / DR_RUN;
   static constexpr int RS = R + 4;                      // floats between two lanes' rows
   static constexpr int TS = P * RS;                     // floats of one token's query (or key)
   static constexpr int COLS = DR_COMPUTE / P;
-  // q | k | v | g | beta | k.q | spare, and with a decay per channel (CH) the decays of every token in the place of a key
-  static constexpr int FLOATS = (CH ? 3 : 2) * DR_TT * TS + DR_TT * COLS + 4 * DR_TT;
-  static constexpr int DECAYS = FLOATS - DR_TT * TS;    // where those begin
+  // G_t k_t | G_t q_t | D_t4 k_t of every token, G_4 of every run, the triangles of every run (t-th row: against the keys
+  // s < t, against the query s <= t), write strengths, values
+  static constexpr int Q = TT * TS, KD = 2 * TT * TS, G = 3 * TT * TS;
+  static constexpr int TRI = G + RUNS * TS, BETA = TRI + RUNS * 2 * DR_RUN * DR_RUN, V = BETA + TT;
+  static constexpr int FLOATS = V + TT * COLS;
 };
 
-// What a fetching thread holds of one tile between asking for it and writing it to shared memory.
+// What a fetching thread holds of one tile between asking for it and writing it to shared memory: of its warp's run the
+// numbers lane, lane + 32, ... of every query, key and row of decays, and lane t < 4 the write strength (and step size) of
+// token t; as they lie in memory, so that nothing waits for a load before the tile is written.
 template <typename T, int R, int P, bool CH>
 struct DrRaw {
-  static constexpr int NT = DR_TT / 4;                  // tokens of a warp
-  static constexpr int NL = (R * P + 31) / 32;          // a lane's numbers of one query (or key)
-  static constexpr int NV = DR_TT * DrTile<R, P, CH>::COLS / (DR_THREADS - DR_COMPUTE);
-  float g[CH ? NT : 1][CH ? NL : 1];                    // decays per channel
-  T q[NT][NL], k[NT][NL], v[NV], b, a;                  // as they lie in memory: nothing waits for a load before the tile is written
+  static constexpr int NL = (R * P + 31) / 32;
+  static constexpr int NV = (DrTile<R, P>::TT * DrTile<R, P>::COLS + DR_COMPUTE - 1) / DR_COMPUTE;
+  float g[CH ? DR_RUN : 1][CH ? NL : 1];
+  T q[DR_RUN][NL], k[DR_RUN][NL], v[NV], b, a;
 };
 
 // The fetching warps ask for tile [first_row, first_row + tn) of the request's rows: every load is issued, none is
@@ -63,92 +75,144 @@ __device__ __forceinline__ void dr_ask(DrRaw<T, R, P, CH>& raw, const T* __restr
                                        int v_at, const T* __restrict__ proj, int proj_stride, int b_at, int a_at,
                                        const float* __restrict__ decay, int decay_stride, int first_row, int tn, int d, int e,
                                        int col0, int lt) {
-  using L = DrTile<R, P, CH>;
+  using L = DrTile<R, P>;
   using W = DrRaw<T, R, P, CH>;
-  const int lane = lt & 31, warp = lt >> 5;
+  const int lane = lt & 31, run0 = (lt >> 5) * DR_RUN;
   const T zero = from_float<T>(0.0f);
+  raw.b = zero;
+  raw.a = zero;
+  if (run0 < L::TT) {
 #pragma unroll
-  for (int s = 0; s < W::NT; ++s) {
-    const int tt = warp + 4 * s;
-    const T* urow = u + static_cast<size_t>(first_row + max(min(tt, tn - 1), 0)) * u_stride;
+    for (int t = 0; t < DR_RUN; ++t) {
+      const int tt = run0 + t;
+      const size_t row = static_cast<size_t>(first_row + max(min(tt, tn - 1), 0));
+      const T* urow = u + row * u_stride;
 #pragma unroll
-    for (int c = 0; c < W::NL; ++c) {
-      const int i = lane + 32 * c;
-      const bool ok = tt < tn && i < d;
-      raw.q[s][c] = ok ? urow[q_at + i] : zero;
-      raw.k[s][c] = ok ? urow[k_at + i] : zero;
-      if constexpr (CH) raw.g[s][c] = ok ? decay[static_cast<size_t>(first_row + tt) * decay_stride + i] : 0.0f;
+      for (int c = 0; c < W::NL; ++c) {
+        const int i = lane + 32 * c;
+        const bool ok = tt < tn && i < d;
+        raw.q[t][c] = ok ? urow[q_at + i] : zero;
+        raw.k[t][c] = ok ? urow[k_at + i] : zero;
+        if constexpr (CH) raw.g[t][c] = ok ? decay[row * decay_stride + i] : 1.0f;
+      }
+    }
+    if (lane < DR_RUN && run0 + lane < tn) {
+      const T* prow = proj + static_cast<size_t>(first_row + run0 + lane) * proj_stride;
+      raw.b = prow[b_at];
+      if constexpr (!CH) raw.a = prow[a_at];
     }
   }
 #pragma unroll
   for (int c = 0; c < W::NV; ++c) {
-    const int idx = lt + (DR_THREADS - DR_COMPUTE) * c;
+    const int idx = lt + DR_COMPUTE * c;
     const int tt = idx / L::COLS, col = col0 + idx % L::COLS;
     raw.v[c] = (tt < tn && col < e) ? u[static_cast<size_t>(first_row + tt) * u_stride + v_at + col] : zero;
   }
-  raw.b = zero;
-  raw.a = zero;
-  if (lt < tn) {
-    const T* prow = proj + static_cast<size_t>(first_row + lt) * proj_stride;
-    raw.b = prow[b_at];
-    if constexpr (!CH) raw.a = prow[a_at];
-  }
 }
 
-// ... and write it into one of the two buffers: queries and keys as unit vectors (a warp per token), k . q, the
-// values of the block's columns, the two gates.
+// ... and write it into one of the two buffers.
 template <typename T, int R, int P, bool CH>
 __device__ __forceinline__ void dr_put(const DrRaw<T, R, P, CH>& raw, float* buf, int tn, int d, float q_scale, float decay_rate,
                                        float bias, int lt) {
-  using L = DrTile<R, P, CH>;
+  using L = DrTile<R, P>;
   using W = DrRaw<T, R, P, CH>;
-  float* sq = buf;
-  float* sk = sq + DR_TT * L::TS;
-  float* sv = sk + DR_TT * L::TS;
-  float* sg = sv + DR_TT * L::COLS;
-  float* sbeta = sg + DR_TT;
-  float* skq = sbeta + DR_TT;
-  const int lane = lt & 31, warp = lt >> 5;
+  const int lane = lt & 31, run = lt >> 5, run0 = run * DR_RUN;
 #pragma unroll
-  for (int s = 0; s < W::NT; ++s) {
-    const int tt = warp + 4 * s;
-    float qq = 0.0f, kk = 0.0f, kq = 0.0f, qf[W::NL], kf[W::NL];
+  for (int c = 0; c < W::NV; ++c) {
+    const int idx = lt + DR_COMPUTE * c;
+    if (idx < L::TT * L::COLS) buf[L::V + idx] = to_float(raw.v[c]);
+  }
+  if (run0 >= L::TT) return;                            // (a whole warp)
+  float gs[DR_RUN];                                     // one decay a token
+  if constexpr (!CH) {
+    const float mine = lane < DR_RUN && run0 + lane < tn ? expf(-decay_rate * dr_softplus(to_float(raw.a) + bias)) : 1.0f;
 #pragma unroll
-    for (int c = 0; c < W::NL; ++c) {
-      qf[c] = to_float(raw.q[s][c]);
-      kf[c] = to_float(raw.k[s][c]);
-      qq = fmaf(qf[c], qf[c], qq);
-      kk = fmaf(kf[c], kf[c], kk);
-      kq = fmaf(kf[c], qf[c], kq);
+    for (int t = 0; t < DR_RUN; ++t) gs[t] = __shfl_sync(0xffffffffu, mine, t);
+  }
+  auto g_of = [&](int t, int c) {
+    if constexpr (CH) return raw.g[t][c];
+    else return gs[t];
+  };
+  // sums over the channels: 0..3 q.q, 4..7 k.k, 8..13 (D_st k_s).k_t for s < t, 14..23 (D_st k_s).q_t for s <= t
+  float sum[32];
+#pragma unroll
+  for (int i = 0; i < 32; ++i) sum[i] = 0.0f;
+#pragma unroll
+  for (int c = 0; c < W::NL; ++c) {
+    float q[DR_RUN], k[DR_RUN];
+#pragma unroll
+    for (int t = 0; t < DR_RUN; ++t) {
+      q[t] = to_float(raw.q[t][c]);
+      k[t] = to_float(raw.k[t][c]);
+      sum[t] = fmaf(q[t], q[t], sum[t]);
+      sum[4 + t] = fmaf(k[t], k[t], sum[4 + t]);
     }
+    int a = 8, b = 14;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {                  // three sums side by side
-      qq += __shfl_xor_sync(0xffffffffu, qq, o);
-      kk += __shfl_xor_sync(0xffffffffu, kk, o);
-      kq += __shfl_xor_sync(0xffffffffu, kq, o);
-    }
-    const float fq = q_scale / sqrtf(qq + 1e-6f), fk = 1.0f / sqrtf(kk + 1e-6f);
-    if (lane == 0 && tt < tn) skq[tt] = kq * fq * fk;   // the unit key times the scaled unit query
+    for (int s = 0; s < DR_RUN; ++s) {
+      float w = k[s];
 #pragma unroll
-    for (int c = 0; c < W::NL; ++c) {
-      const int i = lane + 32 * c;
-      if (tt < tn && i < d) {
-        const int at = tt * L::TS + (i / R) * L::RS + i % R;
-        sq[at] = qf[c] * fq;
-        sk[at] = kf[c] * fk;
-        if constexpr (CH) buf[L::DECAYS + at] = raw.g[s][c];
+      for (int t = s; t < DR_RUN; ++t) {
+        if (t > s) {
+          w *= g_of(t, c);
+          sum[a] = fmaf(w, k[t], sum[a]);
+          ++a;
+        }
+        sum[b] = fmaf(w, q[t], sum[b]);
+        ++b;
       }
     }
   }
+  // every round halves the sums a lane is in charge of: in the end lane i holds sum i over all lanes
 #pragma unroll
-  for (int c = 0; c < W::NV; ++c) {
-    const int idx = lt + (DR_THREADS - DR_COMPUTE) * c;
-    if (idx < tn * L::COLS) sv[idx] = to_float(raw.v[c]);
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? sum[i] : sum[i + o], keep = up ? sum[i + o] : sum[i];
+      sum[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
   }
-  if (lt < tn) {
-    sbeta[lt] = 1.0f / (1.0f + expf(-to_float(raw.b)));
-    if constexpr (!CH) sg[lt] = expf(-decay_rate * dr_softplus(to_float(raw.a) + bias));
+  const float f = lane < 8 ? (lane < 4 ? q_scale : 1.0f) / sqrtf(sum[0] + 1e-6f) : 0.0f;      // to unit length
+  {
+    const bool keys = lane < 14;
+    int s = 0, t = 0;
+    if (lane >= 8 && lane < 24) {                       // which pair of tokens this lane's sum is of
+      int n = keys ? lane - 8 : lane - 14, len = keys ? DR_RUN - 1 : DR_RUN;
+      while (n >= len) { n -= len; --len; ++s; }
+      t = s + n + (keys ? 1 : 0);
+    }
+    const float fs = __shfl_sync(0xffffffffu, f, 4 + s), ft = __shfl_sync(0xffffffffu, f, keys ? 4 + t : t);
+    if (lane >= 8 && lane < 24) buf[L::TRI + (run * 2 + (keys ? 0 : 1)) * DR_RUN * DR_RUN + t * DR_RUN + s] = sum[0] * fs * ft;
   }
+  float fq[DR_RUN], fk[DR_RUN];
+#pragma unroll
+  for (int t = 0; t < DR_RUN; ++t) {
+    fq[t] = __shfl_sync(0xffffffffu, f, t);
+    fk[t] = __shfl_sync(0xffffffffu, f, 4 + t);
+  }
+#pragma unroll
+  for (int c = 0; c < W::NL; ++c) {
+    const int i = lane + 32 * c;
+    if (i < d) {
+      const int at = (i / R) * L::RS + i % R;
+      float G = 1.0f;
+#pragma unroll
+      for (int t = 0; t < DR_RUN; ++t) {
+        G *= g_of(t, c);
+        buf[(run0 + t) * L::TS + at] = to_float(raw.k[t][c]) * fk[t] * G;
+        buf[L::Q + (run0 + t) * L::TS + at] = to_float(raw.q[t][c]) * fq[t] * G;
+      }
+      buf[L::G + run * L::TS + at] = G;
+      float D = 1.0f;
+#pragma unroll
+      for (int t = DR_RUN - 1; t >= 0; --t) {
+        buf[L::KD + (run0 + t) * L::TS + at] = to_float(raw.k[t][c]) * fk[t] * D;
+        D *= g_of(t, c);
+      }
+    }
+  }
+  if (lane < DR_RUN) buf[L::BETA + run0 + lane] = run0 + lane < tn ? 1.0f / (1.0f + expf(-to_float(raw.b))) : 0.0f;
 }
 
 template <typename T, int R, int P, bool CH>
@@ -158,26 +222,25 @@ delta_rule_kernel(const T* __restrict__ u, int u_stride, int q_col, int k_col, i
                   const float* __restrict__ a_log, const float* __restrict__ dt_bias, const float* __restrict__ decays,
                   int decay_stride, float* __restrict__ state, size_t state_stride, const int* __restrict__ q_start,
                   const int* __restrict__ state_slots, float* __restrict__ out, int H, int G, int d, int e) {
-  using L = DrTile<R, P, CH>;
+  using L = DrTile<R, P>;
   extern __shared__ __align__(16) float sm[];   // two tiles
   const int h = blockIdx.y, r = blockIdx.z;
   const int j = h / (H / G);
   const int tid = threadIdx.x;
   const int col0 = blockIdx.x * L::COLS;
   const int row0 = q_start[r], n = q_start[r + 1] - row0;
+  if (n <= 0) return;
   const float q_scale = rsqrtf(static_cast<float>(d));
   const float decay_rate = CH ? 0.0f : expf(a_log[h]), bias = CH ? 0.0f : dt_bias[h];
   const float* decay = CH ? decays + static_cast<size_t>(h) * d : nullptr;
   const int q_at = q_col + j * d, k_at = k_col + j * d, v_at = v_col + h * e, b_at = b_col + h, a_at = a_col + h;
 
-  // rows past d (a lane's share rounded up) stay zero in both tiles: the fetching warps never touch them
-  if (R * P != d) {
-    for (int idx = tid; idx < 2 * L::FLOATS; idx += DR_THREADS) sm[idx] = 0.0f;
-    __syncthreads();
-  }
+  // rows past d (a lane's share rounded up) and the empty halves of the triangles stay zero in both tiles
+  for (int idx = tid; idx < 2 * L::FLOATS; idx += DR_THREADS) sm[idx] = 0.0f;
+  __syncthreads();
 
   const bool computes = tid < DR_COMPUTE;
-  const int col = col0 + tid / P, part = tid % P;
+  const int part = tid % P, cl = tid / P, col = col0 + cl;
   const bool live = computes && col < e;
   float* S_g = state + static_cast<size_t>(ck_request(state_slots[r])) * state_stride + static_cast<size_t>(h) * d * e;
   float S[R];
@@ -190,83 +253,103 @@ delta_rule_kernel(const T* __restrict__ u, int u_stride, int q_col, int k_col, i
       S[i] = (live && row < d) ? S_g[static_cast<size_t>(row) * e + col] : 0.0f;
     }
   } else {
-    dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride, row0, min(DR_TT, n), d, e, col0, lt);
-    dr_put<T, R, P, CH>(raw, sm, min(DR_TT, n), d, q_scale, decay_rate, bias, lt);
-    if (n > DR_TT)
-      dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride, row0 + DR_TT,
-                      min(DR_TT, n - DR_TT), d, e, col0, lt);
+    dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride, row0,
+                        min(L::TT, n), d, e, col0, lt);
+    dr_put<T, R, P, CH>(raw, sm, min(L::TT, n), d, q_scale, decay_rate, bias, lt);
+    if (n > L::TT)
+      dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride,
+                          row0 + L::TT, min(L::TT, n - L::TT), d, e, col0, lt);
   }
   __syncthreads();
 
   int which = 0;
-  for (int t0 = 0; t0 < n; t0 += DR_TT, which ^= 1) {
-    const int tn = min(DR_TT, n - t0);
+  for (int t0 = 0; t0 < n; t0 += L::TT, which ^= 1) {
+    const int tn = min(L::TT, n - t0);
     if (!computes) {
       // the tile after this one was asked for a tile ago: write it, then ask for the one after it
-      if (t0 + DR_TT < n) {
-        dr_put<T, R, P, CH>(raw, sm + (which ^ 1) * L::FLOATS, min(DR_TT, n - t0 - DR_TT), d, q_scale, decay_rate, bias, lt);
-        if (t0 + 2 * DR_TT < n)
-          dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride, row0 + t0 + 2 * DR_TT,
-                          min(DR_TT, n - t0 - 2 * DR_TT), d, e, col0, lt);
+      if (t0 + L::TT < n) {
+        dr_put<T, R, P, CH>(raw, sm + (which ^ 1) * L::FLOATS, min(L::TT, n - t0 - L::TT), d, q_scale, decay_rate, bias, lt);
+        if (t0 + 2 * L::TT < n)
+          dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride,
+                              row0 + t0 + 2 * L::TT, min(L::TT, n - t0 - 2 * L::TT), d, e, col0, lt);
       }
     } else {
-      const float* sq = sm + which * L::FLOATS;
-      const float* sk = sq + DR_TT * L::TS;
-      const float* sv = sk + DR_TT * L::TS;
-      const float* sg = sv + DR_TT * L::COLS;
-      const float* sbeta = sg + DR_TT;
-      float* orow = out + static_cast<size_t>(row0 + t0) * (H * e) + h * e + col;
-      const float* skq = sbeta + DR_TT;
-      // Both dot products of a token run over the state the token found: with S' = g S + k u^T the read-out is
-      // S'^T q = g (S^T q) + u (k . q), and k . q is the same for every column (the fetching warps leave it beside
-      // the gates). So the path from token to token is one round of multiply-adds, one round of shuffles (both sums
-      // at once) and the update; the products g S do not wait for the shuffles.
-#pragma unroll 2
-      for (int tt = 0; tt < tn; ++tt) {
-        const float g = CH ? 1.0f : sg[tt];
-        const float beta = sbeta[tt], kq = skq[tt], v = sv[tt * L::COLS + tid / P];
-        if constexpr (CH) {
-          const float4* g4 = reinterpret_cast<const float4*>(sq + L::DECAYS + tt * L::TS + part * L::RS);
+      const float* buf = sm + which * L::FLOATS;
+      for (int run = 0; run * DR_RUN < tn; ++run) {
+        const float* kg = buf + run * DR_RUN * L::TS + part * L::RS;
+        float a[DR_RUN] = {0.0f, 0.0f, 0.0f, 0.0f}, o[DR_RUN] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-          for (int i = 0; i < R / 4; ++i) {
-            const float4 gv = g4[i];
-            S[4 * i] *= gv.x;
-            S[4 * i + 1] *= gv.y;
-            S[4 * i + 2] *= gv.z;
-            S[4 * i + 3] *= gv.w;
+        for (int i = 0; i < R; i += 4) {
+#pragma unroll
+          for (int t = 0; t < DR_RUN; ++t) {
+            const float4 kv = *reinterpret_cast<const float4*>(kg + t * L::TS + i);
+            const float4 qv = *reinterpret_cast<const float4*>(kg + L::Q + t * L::TS + i);
+            a[t] = fmaf(S[i], kv.x, a[t]);
+            o[t] = fmaf(S[i], qv.x, o[t]);
+            a[t] = fmaf(S[i + 1], kv.y, a[t]);
+            o[t] = fmaf(S[i + 1], qv.y, o[t]);
+            a[t] = fmaf(S[i + 2], kv.z, a[t]);
+            o[t] = fmaf(S[i + 2], qv.z, o[t]);
+            a[t] = fmaf(S[i + 3], kv.w, a[t]);
+            o[t] = fmaf(S[i + 3], qv.w, o[t]);
           }
         }
-        const float4* k4 = reinterpret_cast<const float4*>(sk + tt * L::TS + part * L::RS);
-        const float4* q4 = reinterpret_cast<const float4*>(sq + tt * L::TS + part * L::RS);
-        float kr[R];
-        float d0 = 0.0f, d1 = 0.0f, d2 = 0.0f, d3 = 0.0f, o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
 #pragma unroll
-        for (int i = 0; i < R / 4; ++i) {
-          const float4 kv = k4[i], qv = q4[i];
-          kr[4 * i] = kv.x; kr[4 * i + 1] = kv.y; kr[4 * i + 2] = kv.z; kr[4 * i + 3] = kv.w;
-          d0 = fmaf(S[4 * i], kv.x, d0);
-          d1 = fmaf(S[4 * i + 1], kv.y, d1);
-          d2 = fmaf(S[4 * i + 2], kv.z, d2);
-          d3 = fmaf(S[4 * i + 3], kv.w, d3);
-          o0 = fmaf(S[4 * i], qv.x, o0);
-          o1 = fmaf(S[4 * i + 1], qv.y, o1);
-          o2 = fmaf(S[4 * i + 2], qv.z, o2);
-          o3 = fmaf(S[4 * i + 3], qv.w, o3);
+        for (int x = P >> 1; x > 0; x >>= 1) {
+#pragma unroll
+          for (int t = 0; t < DR_RUN; ++t) a[t] += __shfl_xor_sync(0xffffffffu, a[t], x);
         }
-        float dot = (d0 + d1) + (d2 + d3), sq_dot = (o0 + o1) + (o2 + o3);
-        if constexpr (!CH) {
+        const float* tri = buf + L::TRI + run * 2 * DR_RUN * DR_RUN;
+        const float4 beta = *reinterpret_cast<const float4*>(buf + L::BETA + run * DR_RUN);
+        const float* v = buf + L::V + run * DR_RUN * L::COLS + cl;
+        const float4 t2 = *reinterpret_cast<const float4*>(tri + 2 * DR_RUN), t3 = *reinterpret_cast<const float4*>(tri + 3 * DR_RUN);
+        const float u0 = beta.x * (v[0] - a[0]);
+        const float u1 = beta.y * (v[L::COLS] - a[1] - tri[DR_RUN] * u0);
+        const float u2 = beta.z * (v[2 * L::COLS] - a[2] - t2.x * u0 - t2.y * u1);
+        const float u3 = beta.w * (v[3 * L::COLS] - a[3] - t3.x * u0 - t3.y * u1 - t3.z * u2);
 #pragma unroll
-          for (int i = 0; i < R; ++i) S[i] *= g;
+        for (int i = 0; i < R; i += 4) {
+          const float4 gv = *reinterpret_cast<const float4*>(buf + L::G + run * L::TS + part * L::RS + i);
+          const float4 k0 = *reinterpret_cast<const float4*>(kg + L::KD + i), k1 = *reinterpret_cast<const float4*>(kg + L::KD + L::TS + i);
+          const float4 k2 = *reinterpret_cast<const float4*>(kg + L::KD + 2 * L::TS + i), k3 = *reinterpret_cast<const float4*>(kg + L::KD + 3 * L::TS + i);
+          S[i] = fmaf(k3.x, u3, fmaf(k2.x, u2, fmaf(k1.x, u1, fmaf(k0.x, u0, gv.x * S[i]))));
+          S[i + 1] = fmaf(k3.y, u3, fmaf(k2.y, u2, fmaf(k1.y, u1, fmaf(k0.y, u0, gv.y * S[i + 1]))));
+          S[i + 2] = fmaf(k3.z, u3, fmaf(k2.z, u2, fmaf(k1.z, u1, fmaf(k0.z, u0, gv.z * S[i + 2]))));
+          S[i + 3] = fmaf(k3.w, u3, fmaf(k2.w, u2, fmaf(k1.w, u1, fmaf(k0.w, u0, gv.w * S[i + 3]))));
         }
+        // the four read-outs: two rounds share them out among the lanes (one token a lane), the rest finish the sums
+        int mine = 0;                                   // the token this lane writes
+        float own;
+        if constexpr (P >= 4) {
+          const bool hi = part & (P >> 1), lo = part & (P >> 2);
+          const float x0 = (hi ? o[2] : o[0]) + __shfl_xor_sync(0xffffffffu, hi ? o[0] : o[2], P >> 1);
+          const float x1 = (hi ? o[3] : o[1]) + __shfl_xor_sync(0xffffffffu, hi ? o[1] : o[3], P >> 1);
+          own = (lo ? x1 : x0) + __shfl_xor_sync(0xffffffffu, lo ? x0 : x1, P >> 2);
 #pragma unroll
-        for (int o = P >> 1; o > 0; o >>= 1) {
-          dot += __shfl_xor_sync(0xffffffffu, dot, o);
-          sq_dot += __shfl_xor_sync(0xffffffffu, sq_dot, o);
+          for (int x = P >> 3; x > 0; x >>= 1) own += __shfl_xor_sync(0xffffffffu, own, x);
+          mine = (hi ? 2 : 0) + (lo ? 1 : 0);
+        } else {
+#pragma unroll
+          for (int x = P >> 1; x > 0; x >>= 1) {
+#pragma unroll
+            for (int t = 0; t < DR_RUN; ++t) o[t] += __shfl_xor_sync(0xffffffffu, o[t], x);
+          }
         }
-        const float uval = beta * (v - g * dot);
+        float* orow = out + static_cast<size_t>(row0 + t0 + run * DR_RUN) * (H * e) + h * e + col;
+        const float* tq = tri + DR_RUN * DR_RUN;
+        if constexpr (P >= 4) {
+          if (live && (part & ((P >> 2) - 1)) == 0 && run * DR_RUN + mine < tn) {
+            const float4 w = *reinterpret_cast<const float4*>(tq + mine * DR_RUN);
+            orow[static_cast<size_t>(mine) * (H * e)] = fmaf(w.w, u3, fmaf(w.z, u2, fmaf(w.y, u1, fmaf(w.x, u0, own))));
+          }
+        } else if (live && part == 0) {
 #pragma unroll
-        for (int i = 0; i < R; ++i) S[i] = fmaf(kr[i], uval, S[i]);
-        if (live && part == 0) orow[static_cast<size_t>(tt) * (H * e)] = fmaf(uval, kq, g * sq_dot);
+          for (int t = 0; t < DR_RUN; ++t) {
+            const float4 w = *reinterpret_cast<const float4*>(tq + t * DR_RUN);
+            if (run * DR_RUN + t < tn)
+              orow[static_cast<size_t>(t) * (H * e)] = fmaf(w.w, u3, fmaf(w.z, u2, fmaf(w.y, u1, fmaf(w.x, u0, o[t]))));
+          }
+        }
       }
     }
     __syncthreads();                            // the tile has been read, the next one is whole
@@ -425,7 +508,7 @@ int delta_rule_launch(const void* u, int u_stride, int q_col, int k_col, int v_c
                       float* state, long long state_stride,
                       const int* q_start, const int* state_slots, float* out, int requests, int H, int G, int d, int e,
                       cudaStream_t stream) {
-  using L = DrTile<R, P, CH>;
+  using L = DrTile<R, P>;
   const size_t smem = static_cast<size_t>(2 * L::FLOATS) * sizeof(float);
   auto kernel = delta_rule_kernel<T, R, P, CH>;
   if (smem > 48 * 1024) {
@@ -449,16 +532,20 @@ int delta_rule_launch(const void* u, int u_stride, int q_col, int k_col, int v_c
 DL_EXPORT int dl_delta_rule(int dtype, const void* u, int u_stride, int q_col, int k_col, int v_col, const void* proj,
                             int proj_stride, int b_col, int a_col, const float* a_log, const float* dt_bias,
                             const float* decays, int decay_stride, float* state, long long state_stride, const int* q_start,
-                            const int* state_slots, float* out, int requests, int H, int G, int d, int e, cudaStream_t stream) {
+                            const int* state_slots, float* out, int requests, int H, int G, int d, int e, int sm_count,
+                            cudaStream_t stream) {
   if (requests <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || d <= 0 || e <= 0 || d > 512 || H > 65535 || requests > 65535 ||
       (dtype != 0 && dtype != 1))
     return DL_ERR_UNSUPPORTED;
-  // lanes per column: the fewest (a power of two up to 16) that leave a lane at most 16 rows, or up to 32 from d = 257 on.
-  // Short rows keep a token's chain of dependent multiply-adds short; the shuffles that finish a dot product grow
-  // by one step with every doubling.
+  // lanes per column: the fewest (a power of two up to 16) that leave a lane at most 16 rows (24 or 32 from d = 257 on).
+  // Blocks get fewer columns (and lanes fewer rows) while they leave a third of the SMs without one: a column over twice the lanes costs
+  // a round of shuffles a run.
   int P = 1;
-  while (P < 16 && (d + P - 1) / P > 16) P *= 2;
+  while (P < 16 && (d + P - 1) / P > (P == 1 ? 8 : 16)) P *= 2;
+  while (P >= 2 && P < 16 && d > 4 * P && (d + 2 * P - 1) / (2 * P) <= 8 &&
+         3ll * ((e * P + dl::DR_COMPUTE - 1) / dl::DR_COMPUTE) * H * requests < 2ll * sm_count)
+    P *= 2;
   const int need = (d + P - 1) / P;
   const int R = (need + 7) / 8 * 8;
 #define DL_DR_T(T, RR, PP, CH)                                                                                             \
@@ -474,9 +561,9 @@ DL_EXPORT int dl_delta_rule(int dtype, const void* u, int u_stride, int q_col, i
     if (decays != nullptr) DL_DR_T(dl::bf16, RR, PP, true);                                                                \
     DL_DR_T(dl::bf16, RR, PP, false);                                                                                      \
   }
-  DL_DR(8, 1); DL_DR(16, 1);                                   // d up to 16
-  DL_DR(16, 2); DL_DR(16, 4); DL_DR(16, 8); DL_DR(16, 16);     // 17 .. 32, .. 64, .. 128, .. 256
-  DL_DR(24, 16); DL_DR(32, 16);                                // 257 .. 512
+  DL_DR(8, 1); DL_DR(8, 2); DL_DR(8, 4); DL_DR(8, 8); DL_DR(8, 16);      // d up to 8, 16, 32, 64, 128
+  DL_DR(16, 2); DL_DR(16, 4); DL_DR(16, 8); DL_DR(16, 16);               // .. 32, .. 64, .. 128, .. 256
+  DL_DR(24, 16); DL_DR(32, 16);                                          // 257 .. 512
 #undef DL_DR
 #undef DL_DR_T
   return DL_ERR_UNSUPPORTED;

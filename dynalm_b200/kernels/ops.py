@@ -78,7 +78,8 @@ _SIGNATURES = {
         "dl_paged_attention_generic_masked": [_I, _P, _I, _P, _L, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F,
                                               _I, _I, _I, _P, _P, _I, _P]},
     "delta_rule": {
-        "dl_delta_rule": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+        "dl_delta_rule": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I, _I,
+                          _P],
         "dl_delta_rule_step": [_I, _P, _I, _I, _I, _I, _P, _I, _I, _I, _P, _P, _P, _I, _P, _L, _P, _P, _P, _I, _I, _I, _I, _I,
                                _P],
         "dl_delta_decay": [_P, _I, _P, _P, _I, _I, _I, _P],
@@ -1751,10 +1752,14 @@ def delta_rule(u: torch.Tensor, q_col: int, k_col: int, v_col: int, proj: torch.
     if by_channel and not single:
         _check(_fn("delta_rule", "dl_delta_decay")(_p(channel_decay), stride, _p(a_log), _p(dt_bias), u.shape[0], heads, dim,
                                                     _stream()), "delta_decay")
-    _check(_fn("delta_rule", "dl_delta_rule_step" if single else "dl_delta_rule")(
-        dtype_code(u.dtype), _p(u), u.stride(0), q_col, k_col, v_col, _p(proj), proj.stride(0), b_col, a_col, _p(a_log),
-        _p(dt_bias), _p(channel_decay), stride, _p(state), state.stride(0), _p(q_start), _p(state_slots), _p(out), requests,
-        heads, kv_heads, dim, vdim, _stream()), "delta_rule")
+    args = (dtype_code(u.dtype), _p(u), u.stride(0), q_col, k_col, v_col, _p(proj), proj.stride(0), b_col, a_col, _p(a_log),
+            _p(dt_bias), _p(channel_decay), stride, _p(state), state.stride(0), _p(q_start), _p(state_slots), _p(out), requests,
+            heads, kv_heads, dim, vdim)
+    if single:
+        _check(_fn("delta_rule", "dl_delta_rule_step")(*args, _stream()), "delta_rule")
+    else:
+        from .device import sm_count
+        _check(_fn("delta_rule", "dl_delta_rule")(*args, sm_count(), _stream()), "delta_rule")
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, gate_col: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
