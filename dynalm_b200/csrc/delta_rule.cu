@@ -23,14 +23,16 @@
 // four numbers a column; the sixteen dot products in brackets are the same for every column.
 //
 // Block = (slice of the e columns, head, request), 256 threads: four warps that compute and four that fetch.
-// A column of S lies over P neighbouring lanes of a computing warp, lane p holding the R rows p R .. p R + R - 1 in
-// registers; a run's eight dot products are finished by shuffles among those lanes. A request's tokens are walked in tiles
+// A computing lane holds R rows of FOUR columns of S in registers, so that a number read from shared memory serves four
+// multiply-adds (what a lane reads, not what banks deliver, limits shared memory here); P neighbouring lanes hold a column's
+// rows. A run's 8 x 4 dot products are finished by shuffles: two rounds hand every lane one of the four columns (its slot s
+// holds column s xor lane % 4 of the four, so that nothing has to be selected), the rest finish the sums; after the triangle
+// the lanes swap what they write into their columns. A request's tokens are walked in tiles
 // of 16 (of 8 for heads of more than 256) held twice in shared memory: while the computing warps run a tile's runs over
 // their registers, each fetching warp writes a run of the next tile (queries and keys made unit vectors and multiplied by
 // their decays; the run's dot products; write strengths; the values of the block's columns) and asks for the one after it,
 // whose numbers then have a whole tile's time to arrive in its registers: no token waits for global memory. Tokens past a
 // tile's end are zeros with a decay of 1 and change nothing.
-// A lane's rows are R + 4 floats apart in shared memory, so that the P lanes' 16-byte loads fall into different banks.
 //
 // dl_head_norm_gate: out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * w * act(gate[t, h, :]), act silu or sigmoid.
 #include "common.cuh"
@@ -38,6 +40,7 @@
 namespace dl {
 
 constexpr int DR_RUN = 4;                               // tokens of a run
+constexpr int DR_COLS = 4;                              // columns of a lane
 constexpr int DR_COMPUTE = 128;
 constexpr int DR_THREADS = 256;
 
@@ -45,11 +48,11 @@ __device__ __forceinline__ float dr_softplus(float v) { return v > 20.0f ? v : l
 
 template <int R, int P>
 struct DrTile {
-  static constexpr int TT = R * P > 256 ? 8 : 16;       // tokens of a tile
+  static constexpr int TT = R > 8 ? 8 : 16;             // tokens of a tile
   static constexpr int RUNS = TT / DR_RUN;
-  static constexpr int RS = R + 4;                      // floats between two lanes' rows
+  static constexpr int RS = R % 8 == 0 ? R + 4 : R;     // floats between two lanes' rows: 16-byte loads in different banks
   static constexpr int TS = P * RS;                     // floats of one token's query (or key)
-  static constexpr int COLS = DR_COMPUTE / P;
+  static constexpr int COLS = DR_COMPUTE / P * DR_COLS;
   // G_t k_t | G_t q_t | D_t4 k_t of every token, G_4 of every run, the triangles of every run (t-th row: against the keys
   // s < t, against the query s <= t), write strengths, values
   static constexpr int Q = TT * TS, KD = 2 * TT * TS, G = 3 * TT * TS;
@@ -67,6 +70,25 @@ struct DrRaw {
   float g[CH ? DR_RUN : 1][CH ? NL : 1];
   T q[DR_RUN][NL], k[DR_RUN][NL], v[NV], b, a;
 };
+
+// A lane's R rows of a vector in shared memory.
+template <int R>
+__device__ __forceinline__ void dr_rows(const float* p, float* x) {
+  if constexpr (R % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < R; i += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(p + i);
+      x[i] = v.x;
+      x[i + 1] = v.y;
+      x[i + 2] = v.z;
+      x[i + 3] = v.w;
+    }
+  } else {
+    const float2 v = *reinterpret_cast<const float2*>(p);
+    x[0] = v.x;
+    x[1] = v.y;
+  }
+}
 
 // The fetching warps ask for tile [first_row, first_row + tn) of the request's rows: every load is issued, none is
 // waited for. The tile is asked for one tile's time before it is written, so its numbers are there by then.
@@ -240,17 +262,22 @@ delta_rule_kernel(const T* __restrict__ u, int u_stride, int q_col, int k_col, i
   __syncthreads();
 
   const bool computes = tid < DR_COMPUTE;
-  const int part = tid % P, cl = tid / P, col = col0 + cl;
+  const int part = tid % P, four = tid / P * DR_COLS, mine = part & 3;
+  const int cl = four + mine, col = col0 + cl;          // the lane's own column of its four
   const bool live = computes && col < e;
   float* S_g = state + static_cast<size_t>(ck_request(state_slots[r])) * state_stride + static_cast<size_t>(h) * d * e;
-  float S[R];
+  float S[DR_COLS][R];
   DrRaw<T, R, P, CH> raw;
   const int lt = tid - DR_COMPUTE;
   if (computes) {
 #pragma unroll
-    for (int i = 0; i < R; ++i) {
-      const int row = part * R + i;
-      S[i] = (live && row < d) ? S_g[static_cast<size_t>(row) * e + col] : 0.0f;
+    for (int c = 0; c < DR_COLS; ++c) {
+      const int cc = col0 + four + (c ^ mine);
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int row = part * R + i;
+        S[c][i] = (cc < e && row < d) ? S_g[static_cast<size_t>(row) * e + cc] : 0.0f;
+      }
     }
   } else {
     dr_ask<T, R, P, CH>(raw, u, u_stride, q_at, k_at, v_at, proj, proj_stride, b_at, a_at, decay, decay_stride, row0,
@@ -277,78 +304,102 @@ delta_rule_kernel(const T* __restrict__ u, int u_stride, int q_col, int k_col, i
       const float* buf = sm + which * L::FLOATS;
       for (int run = 0; run * DR_RUN < tn; ++run) {
         const float* kg = buf + run * DR_RUN * L::TS + part * L::RS;
-        float a[DR_RUN] = {0.0f, 0.0f, 0.0f, 0.0f}, o[DR_RUN] = {0.0f, 0.0f, 0.0f, 0.0f};
+        float a[DR_RUN][DR_COLS], o[DR_RUN][DR_COLS];
 #pragma unroll
-        for (int i = 0; i < R; i += 4) {
+        for (int t = 0; t < DR_RUN; ++t) {
+          float kv[R], qv[R];
+          dr_rows<R>(kg + t * L::TS, kv);
+          dr_rows<R>(kg + L::Q + t * L::TS, qv);
 #pragma unroll
-          for (int t = 0; t < DR_RUN; ++t) {
-            const float4 kv = *reinterpret_cast<const float4*>(kg + t * L::TS + i);
-            const float4 qv = *reinterpret_cast<const float4*>(kg + L::Q + t * L::TS + i);
-            a[t] = fmaf(S[i], kv.x, a[t]);
-            o[t] = fmaf(S[i], qv.x, o[t]);
-            a[t] = fmaf(S[i + 1], kv.y, a[t]);
-            o[t] = fmaf(S[i + 1], qv.y, o[t]);
-            a[t] = fmaf(S[i + 2], kv.z, a[t]);
-            o[t] = fmaf(S[i + 2], qv.z, o[t]);
-            a[t] = fmaf(S[i + 3], kv.w, a[t]);
-            o[t] = fmaf(S[i + 3], qv.w, o[t]);
+          for (int c = 0; c < DR_COLS; ++c) {
+            a[t][c] = S[c][0] * kv[0];
+            o[t][c] = S[c][0] * qv[0];
+          }
+#pragma unroll
+          for (int i = 1; i < R; ++i) {
+#pragma unroll
+            for (int c = 0; c < DR_COLS; ++c) {
+              a[t][c] = fmaf(S[c][i], kv[i], a[t][c]);
+              o[t][c] = fmaf(S[c][i], qv[i], o[t][c]);
+            }
           }
         }
+        // every lane its own column: slots 1 and 3, then slot 2 go to the lanes whose own columns they are
 #pragma unroll
-        for (int x = P >> 1; x > 0; x >>= 1) {
+        for (int t = 0; t < DR_RUN; ++t) {
 #pragma unroll
-          for (int t = 0; t < DR_RUN; ++t) a[t] += __shfl_xor_sync(0xffffffffu, a[t], x);
+          for (int c = 0; c < DR_COLS; c += 2) {
+            a[t][c] += __shfl_xor_sync(0xffffffffu, a[t][c + 1], 1);
+            o[t][c] += __shfl_xor_sync(0xffffffffu, o[t][c + 1], 1);
+          }
+        }
+        float as[DR_RUN], os[DR_RUN];
+#pragma unroll
+        for (int t = 0; t < DR_RUN; ++t) {
+          as[t] = a[t][0] + __shfl_xor_sync(0xffffffffu, a[t][2], 2);
+          os[t] = o[t][0] + __shfl_xor_sync(0xffffffffu, o[t][2], 2);
+        }
+#pragma unroll
+        for (int x = P >> 1; x > 2; x >>= 1) {
+#pragma unroll
+          for (int t = 0; t < DR_RUN; ++t) as[t] += __shfl_xor_sync(0xffffffffu, as[t], x);
         }
         const float* tri = buf + L::TRI + run * 2 * DR_RUN * DR_RUN;
         const float4 beta = *reinterpret_cast<const float4*>(buf + L::BETA + run * DR_RUN);
         const float* v = buf + L::V + run * DR_RUN * L::COLS + cl;
         const float4 t2 = *reinterpret_cast<const float4*>(tri + 2 * DR_RUN), t3 = *reinterpret_cast<const float4*>(tri + 3 * DR_RUN);
-        const float u0 = beta.x * (v[0] - a[0]);
-        const float u1 = beta.y * (v[L::COLS] - a[1] - tri[DR_RUN] * u0);
-        const float u2 = beta.z * (v[2 * L::COLS] - a[2] - t2.x * u0 - t2.y * u1);
-        const float u3 = beta.w * (v[3 * L::COLS] - a[3] - t3.x * u0 - t3.y * u1 - t3.z * u2);
+        float w[DR_RUN][DR_COLS];                       // what every token writes into the lane's columns; slot 0: its own
+        w[0][0] = beta.x * (v[0] - as[0]);
+        w[1][0] = beta.y * (v[L::COLS] - as[1] - tri[DR_RUN] * w[0][0]);
+        w[2][0] = beta.z * (v[2 * L::COLS] - as[2] - t2.x * w[0][0] - t2.y * w[1][0]);
+        w[3][0] = beta.w * (v[3 * L::COLS] - as[3] - t3.x * w[0][0] - t3.y * w[1][0] - t3.z * w[2][0]);
 #pragma unroll
-        for (int i = 0; i < R; i += 4) {
-          const float4 gv = *reinterpret_cast<const float4*>(buf + L::G + run * L::TS + part * L::RS + i);
-          const float4 k0 = *reinterpret_cast<const float4*>(kg + L::KD + i), k1 = *reinterpret_cast<const float4*>(kg + L::KD + L::TS + i);
-          const float4 k2 = *reinterpret_cast<const float4*>(kg + L::KD + 2 * L::TS + i), k3 = *reinterpret_cast<const float4*>(kg + L::KD + 3 * L::TS + i);
-          S[i] = fmaf(k3.x, u3, fmaf(k2.x, u2, fmaf(k1.x, u1, fmaf(k0.x, u0, gv.x * S[i]))));
-          S[i + 1] = fmaf(k3.y, u3, fmaf(k2.y, u2, fmaf(k1.y, u1, fmaf(k0.y, u0, gv.y * S[i + 1]))));
-          S[i + 2] = fmaf(k3.z, u3, fmaf(k2.z, u2, fmaf(k1.z, u1, fmaf(k0.z, u0, gv.z * S[i + 2]))));
-          S[i + 3] = fmaf(k3.w, u3, fmaf(k2.w, u2, fmaf(k1.w, u1, fmaf(k0.w, u0, gv.w * S[i + 3]))));
+        for (int t = 0; t < DR_RUN; ++t) {
+#pragma unroll
+          for (int c = 1; c < DR_COLS; ++c) w[t][c] = __shfl_xor_sync(0xffffffffu, w[t][0], c);
         }
-        // the four read-outs: two rounds share them out among the lanes (one token a lane), the rest finish the sums
-        int mine = 0;                                   // the token this lane writes
-        float own;
-        if constexpr (P >= 4) {
-          const bool hi = part & (P >> 1), lo = part & (P >> 2);
-          const float x0 = (hi ? o[2] : o[0]) + __shfl_xor_sync(0xffffffffu, hi ? o[0] : o[2], P >> 1);
-          const float x1 = (hi ? o[3] : o[1]) + __shfl_xor_sync(0xffffffffu, hi ? o[1] : o[3], P >> 1);
-          own = (lo ? x1 : x0) + __shfl_xor_sync(0xffffffffu, lo ? x0 : x1, P >> 2);
+        {
+          float gv[R], kv[DR_RUN][R];
+          dr_rows<R>(buf + L::G + run * L::TS + part * L::RS, gv);
 #pragma unroll
-          for (int x = P >> 3; x > 0; x >>= 1) own += __shfl_xor_sync(0xffffffffu, own, x);
-          mine = (hi ? 2 : 0) + (lo ? 1 : 0);
-        } else {
+          for (int t = 0; t < DR_RUN; ++t) dr_rows<R>(kg + L::KD + t * L::TS, kv[t]);
 #pragma unroll
-          for (int x = P >> 1; x > 0; x >>= 1) {
+          for (int i = 0; i < R; ++i) {
 #pragma unroll
-            for (int t = 0; t < DR_RUN; ++t) o[t] += __shfl_xor_sync(0xffffffffu, o[t], x);
+            for (int c = 0; c < DR_COLS; ++c) S[c][i] *= gv[i];
+#pragma unroll
+            for (int t = 0; t < DR_RUN; ++t) {
+#pragma unroll
+              for (int c = 0; c < DR_COLS; ++c) S[c][i] = fmaf(kv[t][i], w[t][c], S[c][i]);
+            }
           }
         }
-        float* orow = out + static_cast<size_t>(row0 + t0 + run * DR_RUN) * (H * e) + h * e + col;
+        // the four read-outs of the lane's column: up to two rounds share them out among its lanes, the rest finish the sums
         const float* tq = tri + DR_RUN * DR_RUN;
-        if constexpr (P >= 4) {
-          if (live && (part & ((P >> 2) - 1)) == 0 && run * DR_RUN + mine < tn) {
-            const float4 w = *reinterpret_cast<const float4*>(tq + mine * DR_RUN);
-            orow[static_cast<size_t>(mine) * (H * e)] = fmaf(w.w, u3, fmaf(w.z, u2, fmaf(w.y, u1, fmaf(w.x, u0, own))));
+        float* orow = out + static_cast<size_t>(row0 + t0 + run * DR_RUN) * (H * e) + h * e + col;
+        auto write = [&](int t, float sum) {
+          if (run * DR_RUN + t < tn) {
+            const float4 f = *reinterpret_cast<const float4*>(tq + t * DR_RUN);
+            orow[static_cast<size_t>(t) * (H * e)] = fmaf(f.w, w[3][0], fmaf(f.z, w[2][0], fmaf(f.y, w[1][0], fmaf(f.x, w[0][0], sum))));
           }
-        } else if (live && part == 0) {
+        };
+        if constexpr (P >= 8) {
+          const bool hi = part & (P >> 1);
+          float x0 = (hi ? os[2] : os[0]) + __shfl_xor_sync(0xffffffffu, hi ? os[0] : os[2], P >> 1);
+          float x1 = (hi ? os[3] : os[1]) + __shfl_xor_sync(0xffffffffu, hi ? os[1] : os[3], P >> 1);
+          if constexpr (P >= 16) {
+            const bool lo = part & (P >> 2);
+            float y = (lo ? x1 : x0) + __shfl_xor_sync(0xffffffffu, lo ? x0 : x1, P >> 2);
 #pragma unroll
-          for (int t = 0; t < DR_RUN; ++t) {
-            const float4 w = *reinterpret_cast<const float4*>(tq + t * DR_RUN);
-            if (run * DR_RUN + t < tn)
-              orow[static_cast<size_t>(t) * (H * e)] = fmaf(w.w, u3, fmaf(w.z, u2, fmaf(w.y, u1, fmaf(w.x, u0, o[t]))));
+            for (int x = P >> 3; x > 2; x >>= 1) y += __shfl_xor_sync(0xffffffffu, y, x);
+            if (live && (part & ((P >> 2) - 1)) < 4) write((hi ? 2 : 0) + (lo ? 1 : 0), y);
+          } else if (live) {
+            write(hi ? 2 : 0, x0);
+            write(hi ? 3 : 1, x1);
           }
+        } else if (live) {
+#pragma unroll
+          for (int t = 0; t < DR_RUN; ++t) write(t, os[t]);
         }
       }
     }
@@ -356,9 +407,13 @@ delta_rule_kernel(const T* __restrict__ u, int u_stride, int q_col, int k_col, i
   }
   if (computes) {
 #pragma unroll
-    for (int i = 0; i < R; ++i) {
-      const int row = part * R + i;
-      if (live && row < d) S_g[static_cast<size_t>(row) * e + col] = S[i];
+    for (int c = 0; c < DR_COLS; ++c) {
+      const int cc = col0 + four + (c ^ mine);
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        const int row = part * R + i;
+        if (cc < e && row < d) S_g[static_cast<size_t>(row) * e + cc] = S[c][i];
+      }
     }
   }
 }
@@ -538,16 +593,16 @@ DL_EXPORT int dl_delta_rule(int dtype, const void* u, int u_stride, int q_col, i
   if (H <= 0 || G <= 0 || H % G != 0 || d <= 0 || e <= 0 || d > 512 || H > 65535 || requests > 65535 ||
       (dtype != 0 && dtype != 1))
     return DL_ERR_UNSUPPORTED;
-  // lanes per column: the fewest (a power of two up to 16) that leave a lane at most 16 rows (24 or 32 from d = 257 on).
-  // Blocks get fewer columns (and lanes fewer rows) while they leave a third of the SMs without one: a column over twice the lanes costs
-  // a round of shuffles a run.
-  int P = 1;
-  while (P < 16 && (d + P - 1) / P > (P == 1 ? 8 : 16)) P *= 2;
-  while (P >= 2 && P < 16 && d > 4 * P && (d + 2 * P - 1) / (2 * P) <= 8 &&
-         3ll * ((e * P + dl::DR_COMPUTE - 1) / dl::DR_COMPUTE) * H * requests < 2ll * sm_count)
-    P *= 2;
-  const int need = (d + P - 1) / P;
-  const int R = (need + 7) / 8 * 8;
+  // four rows a lane up to d = 128 (on 4 to 32 lanes), more on 32 lanes beyond; two rows on 32 lanes where four would leave
+  // SMs without a block
+  int P = 4, R = 4;
+  while (P < 32 && P * R < d) P *= 2;
+  while (P * R < d) R += 4;
+  const int cols = dl::DR_COMPUTE / P * dl::DR_COLS;
+  if (P == 16 && 3ll * ((e + cols - 1) / cols) * H * requests < 2ll * sm_count) {
+    P = 32;
+    R = 2;
+  }
 #define DL_DR_T(T, RR, PP, CH)                                                                                             \
   return dl::delta_rule_launch<T, RR, PP, CH>(u, u_stride, q_col, k_col, v_col, proj, proj_stride, b_col, a_col, a_log,    \
                                               dt_bias, decays, decay_stride, state, state_stride, q_start, state_slots,    \
@@ -561,9 +616,8 @@ DL_EXPORT int dl_delta_rule(int dtype, const void* u, int u_stride, int q_col, i
     if (decays != nullptr) DL_DR_T(dl::bf16, RR, PP, true);                                                                \
     DL_DR_T(dl::bf16, RR, PP, false);                                                                                      \
   }
-  DL_DR(8, 1); DL_DR(8, 2); DL_DR(8, 4); DL_DR(8, 8); DL_DR(8, 16);      // d up to 8, 16, 32, 64, 128
-  DL_DR(16, 2); DL_DR(16, 4); DL_DR(16, 8); DL_DR(16, 16);               // .. 32, .. 64, .. 128, .. 256
-  DL_DR(24, 16); DL_DR(32, 16);                                          // 257 .. 512
+  DL_DR(4, 4); DL_DR(4, 8); DL_DR(4, 16); DL_DR(4, 32); DL_DR(2, 32);      // d up to 16, 32, 64, 128; 33 .. 64
+  DL_DR(8, 32); DL_DR(12, 32); DL_DR(16, 32);                              // d up to 256, 384, 512
 #undef DL_DR
 #undef DL_DR_T
   return DL_ERR_UNSUPPORTED;
