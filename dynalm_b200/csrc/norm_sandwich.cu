@@ -98,8 +98,13 @@ normed_sum_kernel(const TA* __restrict__ a, int parts_a, size_t stride_a, const 
   for (int n = 0; n < N; ++n) {
     const int c = threadIdx.x * V + n * step;
     if (c < width) {
+      float va[V], vb[V];
 #pragma unroll
-      for (int i = 0; i < V; ++i) x[n][i] = x[n][i] * ra * wa[c + i] + y[n][i] * rb * wb[c + i];
+      for (int i = 0; i < V; ++i) va[i] = vb[i] = 0.0f;
+      ns_add<float, V>(wa + c, va);
+      ns_add<float, V>(wb + c, vb);
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[n][i] = x[n][i] * ra * va[i] + y[n][i] * rb * vb[i];
       if constexpr (V == 4) {
         *reinterpret_cast<float4*>(out + base + c) = make_float4(x[n][0], x[n][1], x[n][2], x[n][3]);
       } else {
@@ -166,7 +171,8 @@ DL_EXPORT int dl_normed_sum(int dtype_a, const void* a, int parts_a, long long s
   if (rows <= 0 || width <= 0) return 0;
   if ((dtype_a != 0 && dtype_a != 1) || (dtype_b != 0 && dtype_b != 1) || parts_a < 1 || parts_b < 1) return DL_ERR_UNSUPPORTED;
   const bool wide = width % 4 == 0 && stride_a % 4 == 0 && stride_b % 4 == 0 &&
-                    ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+                    ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(out) |
+                      reinterpret_cast<uintptr_t>(wa) | reinterpret_cast<uintptr_t>(wb)) & 15) == 0;
   const size_t pa = static_cast<size_t>(stride_a), pb = static_cast<size_t>(stride_b);
 #define DL_NS(TA, TB) return dl::launch_normed_sum<TA, TB>(a, parts_a, pa, wa, sa, b, parts_b, pb, wb, sb, eps, out, rows, width, wide, stream)
   if (dtype_a == 0 && dtype_b == 0) DL_NS(float, float);

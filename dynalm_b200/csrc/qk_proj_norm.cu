@@ -178,30 +178,38 @@ qk_norm_turn_vec_kernel(T* __restrict__ proj, int stride, const float* __restric
                         const double* __restrict__ freq, int rot, float mag, const int* __restrict__ positions,
                         const int* __restrict__ row_slot, const int* __restrict__ block_table, int max_blocks,
                         T* __restrict__ k_cache, size_t k_row, T* __restrict__ v_cache, size_t v_row, int H, int G, int d, int e,
-                        int page_size, int values_are_keys, int TG) {
+                        int page_size, int values_are_keys, int tg_shift) {
   constexpr int V = PerVec<T>::n;
   constexpr int MAX_PAIRS = 128;
-  __shared__ float cos_s[MAX_PAIRS], sin_s[MAX_PAIRS];
+  __shared__ __align__(16) float cos_s[MAX_PAIRS], sin_s[MAX_PAIRS];
   const int row = blockIdx.x, tid = threadIdx.x;
+  T* base = proj + static_cast<size_t>(row) * stride;
+  const int TG = 1 << tg_shift, tg_mask = TG - 1, per_head = d / V, half = rot / 2, half_lanes = half / V, own_values = values_are_keys ? 0 : G * e / V;
+  const int turned = (H + G) * TG, total = turned + own_values;
+  // where the 16 bytes of place i begin in the row (heads, then values), -1: an idle lane
+  auto source = [&](int i) {
+    if (i < turned) return (i & tg_mask) < per_head ? (i >> tg_shift) * d + (i & tg_mask) * V : -1;
+    return i < total ? (H + G) * d + (i - turned) * V : -1;
+  };
+  Vec16 raw;
+  raw.raw = make_uint4(0u, 0u, 0u, 0u);
+  int at = source(tid);
+  if (at >= 0) raw = *reinterpret_cast<const Vec16*>(base + at);      // asked for before the angles are worked out
   const int pos = positions[row];
   const int* table = block_table + static_cast<size_t>(ck_request(row_slot[row])) * max_blocks;
   const int page = ck_page_store(table, pos / page_size, max_blocks);
   const size_t slot = static_cast<size_t>(page < 0 ? 0 : page) * page_size + pos % page_size;
-  T* base = proj + static_cast<size_t>(row) * stride;
-  const int half = rot / 2;
   for (int i = tid; i < half; i += blockDim.x) qk_angle(pos, freq[i], mag, cos_s[i], sin_s[i]);
   __syncthreads();
-  const int per_head = d / V, half_lanes = half / V, own_values = values_are_keys ? 0 : G * e / V;
-  const int turned = (H + G) * TG, total = turned + own_values;
   // whole warps walk the heads, so that the shuffles below find their lanes
   for (int i = tid; i < (total + 31) / 32 * 32; i += blockDim.x) {
-    const int head = i / TG, l = i % TG;
-    const bool is_head = i < turned;
-    const bool live = is_head && l < per_head;
-    Vec16 raw;
-    raw.raw = make_uint4(0u, 0u, 0u, 0u);
-    T* src = base + static_cast<size_t>(head) * d + l * V;
-    if (live) raw = *reinterpret_cast<const Vec16*>(src);
+    if (i != tid) {
+      at = source(i);
+      raw.raw = make_uint4(0u, 0u, 0u, 0u);
+      if (at >= 0) raw = *reinterpret_cast<const Vec16*>(base + at);
+    }
+    const int head = i >> tg_shift, l = i & tg_mask;
+    const bool is_head = i < turned, live = is_head && at >= 0;
     float x[V];
     unpack<T>(raw, x);
     float ss = 0.0f;
@@ -209,31 +217,42 @@ qk_norm_turn_vec_kernel(T* __restrict__ proj, int stride, const float* __restric
     for (int j = 0; j < V; ++j) ss = fmaf(x[j], x[j], ss);
     for (int o = TG >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const float r = 1.0f / sqrtf(ss / static_cast<float>(d) + eps);
-    const float* w = head < H ? wq : wk;
     if (live) {
+      const float4* w = reinterpret_cast<const float4*>((head < H ? wq : wk) + l * V);
 #pragma unroll
-      for (int j = 0; j < V; ++j) x[j] *= r * w[l * V + j];
+      for (int j = 0; j < V; j += 4) {
+        const float4 f = w[j / 4];
+        x[j] *= r * f.x;
+        x[j + 1] *= r * f.y;
+        x[j + 2] *= r * f.z;
+        x[j + 3] *= r * f.w;
+      }
     }
     const bool first = l < half_lanes, pair = l < 2 * half_lanes;
     const int lane = tid & 31, partner = pair ? (first ? lane + half_lanes : lane - half_lanes) : lane;
     const int a0 = pair ? (first ? l : l - half_lanes) * V : 0;
 #pragma unroll
-    for (int j = 0; j < V; ++j) {
-      const float y = __shfl_sync(0xffffffffu, x[j], partner);
+    for (int j = 0; j < V; j += 4) {
+      float y[4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n) y[n] = __shfl_sync(0xffffffffu, x[j + n], partner);
       if (pair && live) {
-        const float c = cos_s[a0 + j], s = sin_s[a0 + j];
-        x[j] = first ? x[j] * c - y * s : x[j] * c + y * s;
+        const float4 c = *reinterpret_cast<const float4*>(cos_s + a0 + j), s = *reinterpret_cast<const float4*>(sin_s + a0 + j);
+        const float f = first ? -1.0f : 1.0f;           // (u cos - v sin, v cos + u sin)
+        x[j] = fmaf(x[j], c.x, f * y[0] * s.x);
+        x[j + 1] = fmaf(x[j + 1], c.y, f * y[1] * s.y);
+        x[j + 2] = fmaf(x[j + 2], c.z, f * y[2] * s.z);
+        x[j + 3] = fmaf(x[j + 3], c.w, f * y[3] * s.w);
       }
     }
     if (live && head < H) {
-      *reinterpret_cast<Vec16*>(src) = pack<T>(x);
+      *reinterpret_cast<Vec16*>(base + at) = pack<T>(x);
     } else if (live && page >= 0) {
-      const size_t at = static_cast<size_t>(head - H) * d + l * V;
-      *reinterpret_cast<Vec16*>(k_cache + slot * k_row + at) = pack<T>(x);
-      if (values_are_keys) *reinterpret_cast<Vec16*>(v_cache + slot * v_row + at) = raw;
-    } else if (!is_head && i < total && page >= 0) {
-      const size_t at = static_cast<size_t>(i - turned) * V;
-      *reinterpret_cast<Vec16*>(v_cache + slot * v_row + at) = *reinterpret_cast<const Vec16*>(base + static_cast<size_t>(H + G) * d + at);
+      const size_t to = static_cast<size_t>(head - H) * d + l * V;
+      *reinterpret_cast<Vec16*>(k_cache + slot * k_row + to) = pack<T>(x);
+      if (values_are_keys) *reinterpret_cast<Vec16*>(v_cache + slot * v_row + to) = raw;
+    } else if (!is_head && at >= 0 && page >= 0) {
+      *reinterpret_cast<Vec16*>(v_cache + slot * v_row + static_cast<size_t>(i - turned) * V) = raw;
     }
   }
 }
@@ -361,18 +380,22 @@ DL_EXPORT int dl_qk_norm_turn_cache(int dtype, void* proj, int stride, const flo
       wq == nullptr || wk == nullptr || (rot > 0 && freq == nullptr) || (values_are_keys && d != e) || (dtype != 0 && dtype != 1))
     return DL_ERR_UNSUPPORTED;
   const int V = dtype == 0 ? 4 : 8;
-  int TG = 1;
-  while (TG * V < d) TG *= 2;
-  const uintptr_t bases = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
+  int TG = 1, tg_shift = 0;
+  while (TG * V < d) {
+    TG *= 2;
+    ++tg_shift;
+  }
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |
+                          reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wk);
   if (d % V == 0 && e % V == 0 && TG <= 32 && (rot / 2) % V == 0 && stride % V == 0 && k_row % V == 0 && v_row % V == 0 && (bases & 15) == 0) {
     const int lanes = (H + G) * TG + (values_are_keys ? 0 : G * e / V);
-    const int threads = lanes <= 64 ? 64 : lanes <= 128 ? 128 : lanes <= 256 ? 256 : 512;
+    const int threads = lanes <= 64 ? 64 : lanes <= 128 ? 128 : rows >= 256 || lanes <= 256 ? 256 : 512;   // many rows: more blocks an SM
 #define DL_QK(T)                                                                                                            \
   dl::qk_norm_turn_vec_kernel<T><<<rows, threads, 0, stream>>>(static_cast<T*>(proj), stride, wq, wk, eps, freq, rot, mag,  \
                                                                positions, row_slot, block_table, max_blocks,                \
                                                                static_cast<T*>(k_cache), static_cast<size_t>(k_row),        \
                                                                static_cast<T*>(v_cache), static_cast<size_t>(v_row), H, G,  \
-                                                               d, e, page_size, values_are_keys, TG)
+                                                               d, e, page_size, values_are_keys, tg_shift)
     if (dtype == 0) DL_QK(float);
     else DL_QK(dl::bf16);
 #undef DL_QK
